@@ -26,7 +26,9 @@ pages that lie wholly before that are returned when the length is published and 
 table entries are cleared.  Work already put on the stream may still read them; whoever
 takes them next writes them in work that is put on the stream later.  Such a sequence
 holds about `window / 64 + 2` pages however long it grows.  A need with a `chunk` does the
-same with the pages that lie wholly before the chunk of the next position.
+same with the pages that lie wholly before the chunk of the next position.  A need with
+`keep_first` keeps the pages of that many first positions as long as the sequence lives; the
+pages given back are those between them and the window.
 """
 from __future__ import annotations
 
@@ -81,13 +83,14 @@ class _KVGroup:
             self.values = torch.empty(shape, dtype=dtype, device=device)
         self.pool = FreeList(pages, "cache page")
         self.table = np.zeros((slots, pages_per_sequence), dtype=np.int32)
+        self.kept_pages = pages_for(need.keep_first)  # the first pages of a sequence, never given back while it lives
         self.held: Dict[int, List[int]] = {}          # the pages a sequence holds, oldest first
-        self.released: Dict[int, int] = {}            # how many older pages it has given back already (a window's doing)
+        self.released: Dict[int, int] = {}            # how many pages behind the kept ones it has given back already (a window's doing)
 
     def tokens_read(self, length: int) -> int:
         if self.need.chunk:
             return length - length // self.need.chunk * self.need.chunk
-        return min(length, self.need.window) if self.need.window else length
+        return min(length, self.need.window + self.need.keep_first) if self.need.window else length
 
     def first_kept(self, length: int) -> int:
         """The oldest position that a query at position `length` (the next one) can still read."""
@@ -124,7 +127,7 @@ class SequenceCache:
         # keeps no keys and values at all (state of fixed size only).
         kv_needs = [need for need, _ in groups.values() if need.kind in ("kv", "rows")]
         bounded = all(need.window or need.chunk for need in kv_needs)
-        self.widest_window = max((need.window or need.chunk for need in kv_needs), default=0) if bounded else None
+        self.widest_window = max(((need.window or need.chunk) + pages_for(need.keep_first) * PAGE_TOKENS for need in kv_needs), default=0) if bounded else None
         # ... but its page table is addressed by position, so a sequence is given at most 64 times the pages of the whole cache
         # (1,024 at least), not the 2^31 positions that a design without a position limit would allow.
         self.pages_per_sequence = (min(pages_for(max_sequence_tokens), max(64 * self.n_pages, 1024)) if bounded
@@ -198,14 +201,14 @@ class SequenceCache:
             if not (group.need.window or group.need.chunk):
                 continue
             # The next query sits at position `new_length` and sees keys from `new_length - window + 1` (or its chunk's first) on.
-            keep_from = group.first_kept(new_length) // PAGE_TOKENS
-            gone = keep_from - group.released[slot]
+            keep_from, kept = group.first_kept(new_length) // PAGE_TOKENS, group.kept_pages
+            gone = keep_from - kept - group.released[slot]
             if gone > 0:
                 held = group.held[slot]
-                group.pool.give_back(held[:gone])
-                del held[:gone]
-                group.table[slot, group.released[slot] : keep_from] = 0
-                group.released[slot] = keep_from
+                group.pool.give_back(held[kept : kept + gone])
+                del held[kept : kept + gone]
+                group.table[slot, kept + group.released[slot] : keep_from] = 0
+                group.released[slot] = keep_from - kept
 
     def page_rows(self, group: str, slots, pages: int) -> np.ndarray:
         """Page numbers `[len(slots), pages]` of the given sequences (host memory)."""
@@ -252,5 +255,5 @@ class SequenceCache:
                     raise AssertionError("a sequence is longer than the pages it holds")
                 if group.released[slot] and not (group.need.window or group.need.chunk):
                     raise AssertionError("a group without a window gave pages back early")
-                if group.released[slot] * PAGE_TOKENS > group.first_kept(self.lengths[slot]):
+                if group.released[slot] and (group.kept_pages + group.released[slot]) * PAGE_TOKENS > group.first_kept(self.lengths[slot]):
                     raise AssertionError("a page inside the window was given back")

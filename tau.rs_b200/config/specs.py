@@ -17,7 +17,9 @@ from typing import Optional, Tuple
 class NormSpec:
     """`kind == "rms_norm"`: `x / sqrt(mean(x^2) + eps) * w`.  `kind == "layer_norm"`: `(x - mean) / sqrt(variance + eps) * w + b`,
     the bias being the tensor `<weight's name><bias_suffix>`.  With `groups` > 1 an RMS norm cuts the row into that many equal
-    consecutive pieces and divides each by its own root mean square (on a residual stream kept in 32-bit)."""
+    consecutive pieces and divides each by its own root mean square (on a residual stream kept in 32-bit).  `kind == "dynamic_tanh"`:
+    `tanh(alpha * x) * w + b` with `alpha` the one number `<weight's name>.alpha`, no statistic at all (`eps` is not used), on a residual
+    stream kept in 32-bit."""
 
     width: int
     eps: float
@@ -53,7 +55,9 @@ class AttentionSpec:
 
 @dataclass(frozen=True)
 class SwiGLUSpec:
-    """`down(act(gate(x)) * up(x))` with `act` = `activation` ("silu" or "relu").  The three tensors are `<prefix>.<name><weight_suffix>`."""
+    """`down(act(gate(x)) * up(x))` with `act` = `activation` ("silu" or "relu"), or with `activation == "clamped"` `down(g sigmoid(1.702 g) (u + 1))`,
+    `g = min(gate(x), limit)` and `u` = `up(x)` held between -limit and limit.  The three tensors are `<prefix>.<name><weight_suffix>`.
+    `wide_result`: the last product leaves in 32-bit whatever the run's dtype."""
 
     hidden: int
     intermediate: int
@@ -63,6 +67,8 @@ class SwiGLUSpec:
     down_name: str = "down_proj"
     weight_suffix: str = ".weight"
     activation: str = "silu"
+    limit: float = 0.0
+    wide_result: bool = False
 
 
 @dataclass(frozen=True)
@@ -156,8 +162,12 @@ class LinearRecurrenceSpec:
     `gating == "decay"`: `a_t` is the head's constant of `decays`, `b_t = 1`, and q, k, v pass through `activation`.
     `gating == "exponential"`: a log input gate and a log forget gate per head and token (both soft-capped at `gate_cap`),
     a running maximum that keeps the exponentials in range, a normaliser state, and queries scaled by `query_scale`.
-    `norm_groups` says over what the output is divided by its root mean square before the weight and the sigmoid gate:
-    `"head"` (each head alone) or `"all"` (the concatenated heads)."""
+    `gating == "forget"`: `S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T` with the forget gate `f = l + (1 - l) sigmoid(W_f h + b_f)` per head and
+    key channel, `l` a lower bound per channel (`lower`); there is no key, and the queries pass SiLU.
+    `norm_groups` says over what the output is divided by its root mean square before the weight and the gate:
+    `"head"` (each head alone) or `"all"` (the concatenated heads).  `norm_weight`: `"full"` (one weight per head and value channel),
+    `"head"` (one per value channel, shared by the heads) or None.  `gate_activation`: the output gate is `"sigmoid"` or `"silu"` of one
+    more projection, or absent (None).  `position`: queries and keys are turned by it; `key_scale` multiplies the keys."""
 
     hidden: int
     n_heads: int
@@ -171,6 +181,10 @@ class LinearRecurrenceSpec:
     query_scale: float = 1.0
     activation: Optional[str] = None
     kind: str = "linear_recurrence"
+    position: Optional["ScaledRotationSpec"] = None
+    key_scale: float = 1.0
+    norm_weight: Optional[str] = "full"
+    gate_activation: Optional[str] = "sigmoid"
 
 
 @dataclass(frozen=True)
@@ -206,7 +220,13 @@ class MaskedAttentionSpec:
     one r2 per head (`r1`, `r2`).  `weights == "sigmoid"`: no softmax; a visible key weighs `sigmoid(score + pb[head])` (`pb`, one
     number per head), not normalised over the keys.  `gate`: `"head"` multiplies each head's result by the sigmoid of one number per
     head, `"element"` every element by the sigmoid of its own (`g`, a projection of the mixer's input).  `own_keys=False`: the
-    layer has no key and value tensors and reads the keys and values that another layer of the same sizes cached."""
+    layer has no key and value tensors and reads the keys and values that another layer of the same sizes cached.
+
+    `keep_first`: the sequence's first that many positions stay visible (and cached) however far they lie before the window.  `talk`:
+    the heads' scores are mixed before the softmax, `score_h <- sum_g talk[h, g] score_g` (`talk` [heads, heads]).  `value_mix`:
+    `"first"` hands the layer's values on to the later layers of the step; `"mix"` caches `(1 - share) v + share * first` with the
+    values `first` of the same token that the `"first"` layer handed on (`vmix`, one number; a `"first"` layer has the tensor too and
+    does not use it)."""
 
     hidden: int
     n_heads: int
@@ -228,6 +248,9 @@ class MaskedAttentionSpec:
     weights: str = "softmax"
     gate: Optional[str] = None
     own_keys: bool = True
+    keep_first: int = 0
+    talk: bool = False
+    value_mix: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -331,7 +354,8 @@ class RoutedExpertsSpec:
 
 @dataclass(frozen=True)
 class BlockSpec:
-    """One layer: its weight-name prefix, its two parts and the norm before each.  `residual_scale` (parallel blocks): what the two
+    """One layer: its weight-name prefix, its two parts (the feed-forward may be None in parallel and `"pre_norm_stream"` blocks) and the
+    norm before each.  `residual_scale` (parallel blocks): what the two
     parts return is multiplied by it as it joins the residual stream."""
 
     prefix: str
@@ -433,3 +457,5 @@ class ModelSpec:
     embedding_scale: float = 1.0
     # The logits are the head's product times this.
     logit_scale: float = 1.0
+    # With a cap c > 0 the logits l leave as c * tanh(l / c).
+    logit_cap: float = 0.0

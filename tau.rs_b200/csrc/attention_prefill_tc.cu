@@ -17,6 +17,13 @@
 // (in the exponent's base-2 scale, one `lg2.approx` a score); sigmoid weights `sigmoid(score + offset[head])` replace the softmax (no
 // maximum, no sum, no rescaling: every probability stands alone, one `tanh.approx` each); and a gate per (token, head) multiplies the row as it leaves.
 //
+// The extended form also keeps the sequence's first `keep_first` positions visible beside a window: an item then walks the pages that
+// hold them first, and goes on at its window's first page.
+// A third form (`kSegments`) is for scores mixed over the heads, score_h = sum_g talk[h, g] q_g . k: the caller's queries are mixed
+// beforehand, one piece of D elements for each key head, and S = sum over the key heads j of Q_j K_j^T accumulates in tensor memory
+// piece by piece.  The Q tile is then `n_kv_heads` pieces wide, a stage of the key ring holds one key head's tile, and one block has an
+// SM to itself.
+//
 // The accumulator O is rescaled only when a row's maximum has grown by more than 2^8 since the last rescale, so most
 // tiles do not touch it; the final division by the row sum makes the result exact either way.  The score products run
 // one tile ahead of the softmax (two score buffers in tensor memory), so the tensor cores work on tile i + 1 and on the
@@ -53,6 +60,7 @@ constexpr int kKeyBytes = BN * D * 2;   // a key tile, or a value tile
 #define TAU_ATTN_KEY_STAGES 2
 #endif
 constexpr int kKeyStages = TAU_ATTN_KEY_STAGES;   // key tiles in flight: a key tile is free as soon as its scores are done
+constexpr int kMostKeyStages = kKeyStages > 4 ? kKeyStages : 4;   // the segmented form has as many as fit, up to this
 constexpr int kValueStages = 2;                   // value tiles in flight: free when the second product of their tile is done
 // Shared memory: Q, the key ring, the value ring, then the barriers; nothing is spent on aligning the tiles (dynamic
 // shared memory starts at a multiple of 1,024 bytes, which the kernel checks before it does anything else), so that
@@ -255,9 +263,9 @@ struct Shared {
     float bias[4][96];              // per softmax warp: the distance bias of a tile's 32 rows and 64 keys by distance (95 values)
     uint64_t q_full;                // the Q tile of an item has landed
     uint64_t q_free;                // the last scores of an item are done: the place of its Q tile may be written
-    uint64_t k_full[kKeyStages];    // a key tile has landed
+    uint64_t k_full[kMostKeyStages];    // a key tile has landed
     uint64_t v_full[kValueStages];  // a value tile has landed
-    uint64_t k_free[kKeyStages];    // the first product that read a key tile has finished
+    uint64_t k_free[kMostKeyStages];    // the first product that read a key tile has finished
     uint64_t v_free[kValueStages];  // the second product that read a value tile has finished
     uint64_t s_full[2];             // scores of a tile are in their buffer of tensor memory
     uint64_t s_free[2];             // the softmax has read that buffer
@@ -272,9 +280,10 @@ struct Shared {
     int abort_flag;
 };
 
-// The tiles of an item: which keys its rows see.
+// The tiles of an item: which keys its rows see.  Tiles are numbered from 0; the first `kept_tiles` are the sequence's first pages.
 struct Span {
-    int last_position, first_tile, n_tiles;
+    int last_position, first_tile, n_tiles, kept_tiles;
+    __device__ __forceinline__ int page(int tile) const { return tile < kept_tiles ? tile : first_tile + tile - kept_tiles; }
 };
 // The oldest key that a query at `position` sees: the window's last position, or the first of the query's own chunk (chunks of
 // `chunk` positions counted from position 0), or 0.  Never decreases with the position.
@@ -283,28 +292,33 @@ __device__ __forceinline__ int first_seen(int position, int window, int chunk) {
     if (chunk > 0) return position / chunk * chunk;
     return 0;
 }
-__device__ __forceinline__ Span span_of(const Item& item, int window, int chunk) {
+__device__ __forceinline__ Span span_of(const Item& item, int window, int chunk, int keep_first) {
     Span span;
     span.last_position = item.position0 + item.rows_here - 1;   // of the last real row
     const int first_key = first_seen(item.position0, window, chunk);
     span.first_tile = first_key / BN;
-    span.n_tiles = item.rows_here > 0 ? span.last_position / BN - span.first_tile + 1 : 0;
+    span.kept_tiles = min((keep_first + BN - 1) / BN, span.first_tile);
+    span.n_tiles = item.rows_here > 0 ? span.kept_tiles + span.last_position / BN - span.first_tile + 1 : 0;
     return span;
 }
 
-template <bool kExtended>
+template <bool kExtended, bool kSegments>
 __global__ void __launch_bounds__(kThreads, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                             const __grid_constant__ CUtensorMap v_map, const __grid_constant__ CUtensorMap out_map, bf16* __restrict__ out,
                             const int* __restrict__ cu_seqlens, const int* __restrict__ seq_start, const int* __restrict__ page_rows,
                             int page_stride, int n_seqs, int n_tokens, int n_heads, int n_kv_heads, float scale, int window, int chunk, int sink,
                             float out_scale, long long out_stride, int n_items, int* __restrict__ schedule, const float* __restrict__ distance,
-                            int sigmoid_weights, const float* __restrict__ head_offset, const bf16* __restrict__ head_gate, long long gate_stride) {
+                            int sigmoid_weights, const float* __restrict__ head_offset, const bf16* __restrict__ head_gate, long long gate_stride,
+                            int keep_first_keys, int stages_of_keys) {
+    const int keep_first = kExtended ? keep_first_keys : 0;
+    const int segments = kSegments ? n_kv_heads : 1;                                        // pieces of a query, each against one key head
+    const uint32_t key_stages = kSegments ? static_cast<uint32_t>(stages_of_keys) : kKeyStages;
     extern __shared__ uint8_t shared_raw[];
     uint8_t* tiles = shared_raw;                                   // the swizzled tiles need 1,024-byte alignment
     uint8_t* q_tile = tiles;                                       // kHalves slices of [128 rows x 128 bytes]
-    uint8_t* key_tiles = tiles + kQBytes;                          // kKeyStages key tiles
-    uint8_t* value_tiles = key_tiles + kKeyStages * kKeyBytes;     // kValueStages value tiles
+    uint8_t* key_tiles = tiles + segments * kQBytes;               // key_stages key tiles
+    uint8_t* value_tiles = key_tiles + key_stages * kKeyBytes;     // kValueStages value tiles
     Shared* shared = reinterpret_cast<Shared*>(value_tiles + kValueStages * kKeyBytes);
     if ((smem_address(shared_raw) & 1023u) != 0u) {   // never seen; the same for every thread, before anything is set up
         if (threadIdx.x == 0) atomicExch(&attention_tc_error, 2);
@@ -322,7 +336,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     if (threadIdx.x == 0) {
         barrier_init(&shared->q_full, 1);
         barrier_init(&shared->q_free, 1);
-        for (int s = 0; s < kKeyStages; ++s) {
+        for (int s = 0; s < kMostKeyStages; ++s) {
             barrier_init(&shared->k_full[s], 1);
             barrier_init(&shared->k_free[s], 1);
         }
@@ -417,27 +431,30 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
             bool alive = publish(0, number);
             for (uint32_t k = 0; alive && number >= 0; ++k) {
                 const Item item = shared->item[k & 1];
-                const Span span = span_of(item, window, chunk);
+                const Span span = span_of(item, window, chunk, keep_first);
                 int next = -1;
                 if (span.n_tiles > 0) {
                     const int kv_head = item.head / (n_heads / n_kv_heads);
                     const int* pages = page_rows + static_cast<size_t>(item.seq) * page_stride;
                     if (n > 0 && !barrier_wait(&shared->q_free, (n - 1) & 1u, abort_flag)) break;
-                    barrier_expect_bytes(&shared->q_full, kQBytes);
-                    for (int half = 0; half < kHalves; ++half)
-                        tma_load_2d(q_tile + half * (BM * 128), &q_map, item.head * D + half * 64, item.row, &shared->q_full);
+                    barrier_expect_bytes(&shared->q_full, segments * kQBytes);
+                    for (int slice = 0; slice < segments * kHalves; ++slice)
+                        tma_load_2d(q_tile + slice * (BM * 128), &q_map, item.head * segments * D + slice * 64, item.row, &shared->q_full);
                     // The place of key tile i is free when the scores of the tile kKeyStages before it are done, which is
                     // earlier than the place of value tile i (free when the second product of the tile kValueStages
                     // before it is done): keys are asked for ahead of values, in the order in which their places come free.
                     auto load_keys = [&](int i) {
-                        const int s = kt % kKeyStages;
-                        const uint32_t use = kt / kKeyStages;
-                        if (use > 0 && !barrier_wait(&shared->k_free[s], (use - 1) & 1u, abort_flag)) return false;
-                        const int row = (pages[span.first_tile + i] * n_kv_heads + kv_head) * BN;
-                        barrier_expect_bytes(&shared->k_full[s], kKeyBytes);
-                        for (int half = 0; half < kHalves; ++half)
-                            tma_load_2d(key_tiles + s * kKeyBytes + half * (BN * 128), &k_map, half * 64, row, &shared->k_full[s]);
-                        ++kt;
+                        const int page = pages[span.page(i)];
+                        for (int segment = 0; segment < segments; ++segment) {      // (segmented: the tile of every key head, one after the other)
+                            const int s = kt % key_stages;
+                            const uint32_t use = kt / key_stages;
+                            if (use > 0 && !barrier_wait(&shared->k_free[s], (use - 1) & 1u, abort_flag)) return false;
+                            const int row = (page * n_kv_heads + (kSegments ? segment : kv_head)) * BN;
+                            barrier_expect_bytes(&shared->k_full[s], kKeyBytes);
+                            for (int half = 0; half < kHalves; ++half)
+                                tma_load_2d(key_tiles + s * kKeyBytes + half * (BN * 128), &k_map, half * 64, row, &shared->k_full[s]);
+                            ++kt;
+                        }
                         return true;
                     };
                     auto load_values = [&](int i) {
@@ -445,7 +462,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                         const uint32_t use = vt / kValueStages;
                         if (use > 0 && !barrier_wait(&shared->v_free[s], (use - 1) & 1u, abort_flag)) return false;
                         if (i == 0 && n > 0 && !send_rows()) return false;   // the item before this one leaves first
-                        const int row = (pages[span.first_tile + i] * n_kv_heads + kv_head) * BN;
+                        const int row = (pages[span.page(i)] * n_kv_heads + kv_head) * BN;
                         barrier_expect_bytes(&shared->v_full[s], kKeyBytes);
                         for (int half = 0; half < kHalves; ++half)
                             tma_load_2d(value_tiles + s * kKeyBytes + half * (BN * 128), &v_map, half * 64, row, &shared->v_full[s]);
@@ -455,7 +472,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     // Completion order of the products: scores 0, scores 1, second product 0, scores 2, second product 1, ...; a
                     // load is issued when the product that frees its place is the next to finish, so no wait blocks a later load
                     // whose place is free already: keys run kAhead tiles ahead of values.
-                    constexpr int kAhead = kKeyStages - kValueStages + 1;
+                    // (Segmented: a tile's key heads take turns in the ring, and one tile ahead is as far as the scores run.)
+                    constexpr int kAhead = kSegments ? 1 : kKeyStages - kValueStages + 1;
                     for (int i = 0; i < span.n_tiles + kAhead && alive; ++i) {
                         // The next item is taken when this one has a few tiles left: late, so that blocks which are done
                         // early find the items that remain, but early enough for the answer to be here at this item's end.
@@ -479,25 +497,29 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         if (lane == 0) {
             const uint32_t score_descriptor = instruction_descriptor(BN, false), value_descriptor = instruction_descriptor(D, true);
             const uint32_t q_address = smem_address(q_tile);
-            uint32_t t = 0, n = 0;   // tiles and items with work so far
+            uint32_t t = 0, n = 0, kt = 0;   // tiles, items with work and key tiles so far
             // Scores run one tile ahead of the softmax: while the four warps work on tile i, the products of tile i + 1
             // fill the other score buffer, and the second product of tile i follows as soon as its probabilities are there.
             auto issue_scores = [&](uint32_t tile, bool last_of_item) {
-                const int s = tile % kKeyStages;
-                const uint32_t key_address = smem_address(key_tiles + s * kKeyBytes);
-                if (!barrier_wait(&shared->k_full[s], (tile / kKeyStages) & 1u, abort_flag)) return false;
                 // The buffer also held the probabilities of the tile two before; their product was issued before this one and
                 // the tensor core takes products in the order of issue, so only the softmax's read needs waiting for.
-                if (tile >= 2 && !barrier_wait(&shared->s_free[tile & 1], ((tile >> 1) - 1) & 1u, abort_flag)) return false;
-                tensor_fence_after_sync();
+                if (kSegments && tile >= 2 && !barrier_wait(&shared->s_free[tile & 1], ((tile >> 1) - 1) & 1u, abort_flag)) return false;
+                for (int segment = 0; segment < segments; ++segment) {
+                    const int s = kt % key_stages;
+                    const uint32_t key_address = smem_address(key_tiles + s * kKeyBytes), piece_address = q_address + segment * kQBytes;
+                    if (!barrier_wait(&shared->k_full[s], (kt / key_stages) & 1u, abort_flag)) return false;
+                    if (!kSegments && tile >= 2 && !barrier_wait(&shared->s_free[tile & 1], ((tile >> 1) - 1) & 1u, abort_flag)) return false;
+                    tensor_fence_after_sync();
 #pragma unroll
-                for (int k = 0; k < D / 16; ++k) {
-                    const uint32_t offset = (k / 4) * 128 * BM + (k % 4) * 32;          // slice of 64 d, then 16 d inside it
-                    const uint32_t key_offset = (k / 4) * 128 * BN + (k % 4) * 32;
-                    mma_issue(tensor_base + (tile & 1) * BN, k_major_descriptor(q_address + offset),
-                              k_major_descriptor(key_address + key_offset), score_descriptor, k > 0 ? 1u : 0u);
+                    for (int k = 0; k < D / 16; ++k) {
+                        const uint32_t offset = (k / 4) * 128 * BM + (k % 4) * 32;          // slice of 64 d, then 16 d inside it
+                        const uint32_t key_offset = (k / 4) * 128 * BN + (k % 4) * 32;
+                        mma_issue(tensor_base + (tile & 1) * BN, k_major_descriptor(piece_address + offset),
+                                  k_major_descriptor(key_address + key_offset), score_descriptor, (segment > 0 || k > 0) ? 1u : 0u);
+                    }
+                    mma_commit(&shared->k_free[s]);
+                    ++kt;
                 }
-                mma_commit(&shared->k_free[s]);
                 mma_commit(&shared->s_full[tile & 1]);
                 if (last_of_item) mma_commit(&shared->q_free);
                 return true;
@@ -508,7 +530,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 const Item item = shared->item[k & 1];
                 barrier_arrive(&shared->item_free[k & 1]);
                 if (item.seq < 0) break;
-                const int n_tiles = span_of(item, window, chunk).n_tiles;
+                const int n_tiles = span_of(item, window, chunk, keep_first).n_tiles;
                 if (n_tiles == 0) continue;
                 alive = barrier_wait(&shared->q_full, n & 1u, abort_flag) && issue_scores(t, n_tiles == 1);
                 for (int i = 0; i < n_tiles && alive; ++i) {
@@ -545,7 +567,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
             // The item stays in its place until this warp is done with it (the producer writes the item after the next
             // there, when its own work on the next is over), so the epilogue reads it again and the loop carries less.
             const volatile Item* item_place = &shared->item[k & 1];
-            int n_tiles, first_tile, last_position, position0;
+            int n_tiles, first_tile, kept_tiles, last_position, position0;
             float far = 0.0f, reach = 0.0f, offset_log2 = 0.0f;     // the head's distance numbers and its offset (extended form)
             if (kExtended) {
                 const int head = item_place->head;
@@ -563,8 +585,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     if (item.seq < 0) break;
                     continue;
                 }
-                const Span span = span_of(item, window, chunk);
-                n_tiles = span.n_tiles, first_tile = span.first_tile, last_position = span.last_position, position0 = item.position0;
+                const Span span = span_of(item, window, chunk, keep_first);
+                n_tiles = span.n_tiles, first_tile = span.first_tile, kept_tiles = span.kept_tiles, last_position = span.last_position, position0 = item.position0;
             }
             const int position = position0 + row;
             float used_max = -INFINITY, sum = 0.0f;                   // the maximum that O and `sum` are scaled by
@@ -588,7 +610,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 tensor_fence_before_sync();
                 __syncwarp();
                 if (lane == 0) barrier_arrive(&shared->s_free[tile & 1]);
-                const int key0 = (first_tile + i) * BN;
+                const int key0 = (kExtended && i < kept_tiles ? i : first_tile + i - (kExtended ? kept_tiles : 0)) * BN;
                 if (key0 + BN - 1 > last_position) {
                     // Rows of the page beyond the last position hold whatever an earlier sequence left there.  Their
                     // probabilities are zero, but zero times a stale NaN is not: clear those value rows before the product.
@@ -604,8 +626,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 // window's edge: keys [lowest, highest] of the tile are visible to a row), or none.
                 const int warp_first = position0 + warp * 32, warp_last = warp_first + 31;    // positions of the warp's rows
                 const bool bounded = window > 0 || chunk > 0;
-                const bool all_seen = key0 + BN - 1 <= warp_first && (!bounded || key0 >= first_seen(warp_last, window, chunk));
-                const bool none_seen = key0 > warp_last || (bounded && key0 + BN - 1 < first_seen(warp_first, window, chunk));
+                const bool all_seen = key0 + BN - 1 <= warp_first && (!bounded || key0 >= first_seen(warp_last, window, chunk) || (kExtended && key0 + BN <= keep_first));
+                const bool none_seen = key0 > warp_last || (bounded && key0 + BN - 1 < first_seen(warp_first, window, chunk) && (!kExtended || key0 >= keep_first));
                 if (biased && !none_seen) {
                     // score * scale * log2(e) - r1 * log2(1 + r2 * distance).  The warp's 32 rows and the tile's 64 keys lie 95 different
                     // distances apart: the lanes compute the bias once for each (three to a lane) and every row reads its 64 from
@@ -626,8 +648,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     const int highest = position - key0;
                     if (bounded) {
                         const int lowest = first_seen(position, window, chunk) - key0;
+                        const int kept = kExtended ? keep_first - key0 : 0;      // keys of the tile before this one are kept
 #pragma unroll
-                        for (int j = 0; j < BN; ++j) score[j] = (j <= highest && j >= lowest) ? score[j] : -INFINITY;
+                        for (int j = 0; j < BN; ++j) score[j] = (j <= highest && (j >= lowest || (kExtended && j < kept))) ? score[j] : -INFINITY;
                     } else {
 #pragma unroll
                         for (int j = 0; j < BN; ++j) score[j] = j <= highest ? score[j] : -INFINITY;
@@ -843,30 +866,65 @@ TAU_EXPORT int tau_attention_prefill_tc_status() {
     return flag;
 }
 
+// Key tiles in flight of the segmented form for that many key heads, 0 where its tiles do not fit an SM's shared memory.
+namespace {
+constexpr int kMostShared = 227 * 1024;
+int segmented_bytes(int n_kv_heads, int key_stages) { return n_kv_heads * kQBytes + (key_stages + kValueStages) * kKeyBytes + static_cast<int>(sizeof(Shared)); }
+int segmented_key_stages(int n_kv_heads) {
+    if (n_kv_heads <= 0 || n_kv_heads > 1024) return 0;
+    for (int stages = kMostKeyStages; stages >= 2; --stages)
+        if (segmented_bytes(n_kv_heads, stages) <= kMostShared) return stages;
+    return 0;
+}
+}  // namespace
+
+TAU_EXPORT int tau_attention_prefill_tc_segments_fit(int n_kv_heads) { return segmented_key_stages(n_kv_heads) > 0; }
+
+// `segmented`: queries are [n_tokens, n_heads * n_kv_heads * D], a piece for each key head, and a score is the sum over the key heads.
+// `keep_first`: the sequence's first that many positions stay visible beside a window.
 // `n_pages`: pages of the cache layer (keys and values are `[n_pages, n_kv_heads, 64, D]`).  `schedule`: two integers at
 // zero, which the kernel uses and puts back to zero; launches that share them must follow one another on one stream.
 TAU_EXPORT int tau_attention_prefill_tc(const void* queries, const void* keys, const void* values, void* out, const int* cu_seqlens,
                                         const int* seq_start, const int* page_rows, int page_stride, int page_tokens, long long n_pages,
                                         int n_seqs, int n_tokens, int n_heads, int n_kv_heads, float scale, int window, int chunk, int sink,
                                         float out_scale, long long out_stride, int* schedule, const float* distance, int sigmoid_weights,
-                                        const float* head_offset, const void* head_gate, long long gate_stride, void* stream) {
+                                        const float* head_offset, const void* head_gate, long long gate_stride, int keep_first, int segmented,
+                                        void* stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (sigmoid_weights && sink) return cudaErrorInvalidValue;
     if (!queries || !keys || !values || !out || !cu_seqlens || !seq_start || !page_rows || !schedule || n_heads <= 0 || n_kv_heads <= 0 ||
-        n_heads % n_kv_heads != 0 || page_tokens != BN || window < 0 || chunk < 0 || (window > 0 && chunk > 0) || n_pages <= 0 ||
+        n_heads % n_kv_heads != 0 || page_tokens != BN || window < 0 || chunk < 0 || (window > 0 && chunk > 0) || n_pages <= 0 || keep_first < 0 ||
         out_stride < static_cast<long long>(n_heads) * D || out_stride % 8 != 0 || (reinterpret_cast<uintptr_t>(out) & 15u) != 0)
         return cudaErrorInvalidValue;   // the copy engine and the 16-byte stores want output rows that start on 16 bytes
+    const int segments = segmented ? n_kv_heads : 1;
     CUtensorMap q_map, k_map, v_map, out_map;
     const long long cache_rows = n_pages * n_kv_heads * BN;
     if (cache_rows > 0x7fffffffLL) return cudaErrorInvalidValue;   // a tile's row is a 32-bit coordinate of the copy
-    if (!make_map(&q_map, queries, n_tokens, static_cast<long long>(n_heads) * D, BM) || !make_map(&k_map, keys, cache_rows, D, BN) ||
+    if (!make_map(&q_map, queries, n_tokens, static_cast<long long>(n_heads) * D * segments, BM) || !make_map(&k_map, keys, cache_rows, D, BN) ||
         !make_map(&v_map, values, cache_rows, D, BN) || !make_map(&out_map, out, n_tokens, static_cast<long long>(n_heads) * D, BM, out_stride))
         return cudaErrorInvalidValue;
+    if (segmented) {
+        const int key_stages = segmented_key_stages(n_kv_heads);
+        if (key_stages == 0) return cudaErrorInvalidValue;
+        const int bytes = segmented_bytes(n_kv_heads, key_stages);
+        const cudaError_t status = cudaFuncSetAttribute(attention_prefill_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMostShared);
+        if (status != cudaSuccess) return static_cast<int>(status);
+        int device = 0, sms = 0;
+        if (cudaGetDevice(&device) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) != cudaSuccess || sms <= 0)
+            return cudaErrorInvalidValue;
+        const long long items = (static_cast<long long>((n_tokens + BM - 1) / BM) + n_seqs) * n_heads, fit = bytes + 1024 <= kMostShared / 2 ? 2LL * sms : sms;
+        if (items > 0x7fffffffLL) return cudaErrorInvalidValue;
+        tau_launch(attention_prefill_tc_kernel<true, true>, dim3(static_cast<unsigned>(items < fit ? items : fit)), dim3(kThreads), bytes, static_cast<cudaStream_t>(stream),
+                   q_map, k_map, v_map, out_map, static_cast<bf16*>(out), cu_seqlens, seq_start, page_rows, page_stride, n_seqs, n_tokens, n_heads, n_kv_heads, scale,
+                   window, chunk, sink, out_scale, out_stride, static_cast<int>(items), schedule, distance, sigmoid_weights, head_offset,
+                   static_cast<const bf16*>(head_gate), gate_stride, keep_first, key_stages);
+        return tau_launch_status();
+    }
     const int shared_bytes = kQBytes + (kKeyStages + kValueStages) * kKeyBytes + static_cast<int>(sizeof(Shared));
     static int places = 0;   // blocks that the device holds at once
     if (!places) {
-        cudaError_t status = cudaFuncSetAttribute(attention_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, shared_bytes);
-        if (status == cudaSuccess) status = cudaFuncSetAttribute(attention_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, shared_bytes);
+        cudaError_t status = cudaFuncSetAttribute(attention_prefill_tc_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, shared_bytes);
+        if (status == cudaSuccess) status = cudaFuncSetAttribute(attention_prefill_tc_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, shared_bytes);
         if (status != cudaSuccess) return static_cast<int>(status);
         // Two blocks to an SM: the kernel is compiled for that many (registers), tensor memory holds the columns of two,
         // and a block's shared memory (plus the kilobyte that the system keeps for each) fits twice.
@@ -881,10 +939,10 @@ TAU_EXPORT int tau_attention_prefill_tc(const void* queries, const void* keys, c
     const long long items = (static_cast<long long>((n_tokens + BM - 1) / BM) + n_seqs) * n_heads;   // every sequence may leave a ragged tile
     if (items > 0x7fffffffLL) return cudaErrorInvalidValue;
     const int blocks = static_cast<int>(items < places ? items : places);
-    const bool extended = distance || sigmoid_weights || head_offset || head_gate;
-    tau_launch(extended ? attention_prefill_tc_kernel<true> : attention_prefill_tc_kernel<false>, dim3(blocks), dim3(kThreads), shared_bytes,
+    const bool extended = distance || sigmoid_weights || head_offset || head_gate || keep_first;
+    tau_launch(extended ? attention_prefill_tc_kernel<true, false> : attention_prefill_tc_kernel<false, false>, dim3(blocks), dim3(kThreads), shared_bytes,
                static_cast<cudaStream_t>(stream), q_map, k_map, v_map, out_map, static_cast<bf16*>(out), cu_seqlens, seq_start, page_rows, page_stride, n_seqs,
                n_tokens, n_heads, n_kv_heads, scale, window, chunk, sink, out_scale, out_stride, static_cast<int>(items), schedule, distance, sigmoid_weights,
-               head_offset, static_cast<const bf16*>(head_gate), gate_stride);
+               head_offset, static_cast<const bf16*>(head_gate), gate_stride, keep_first, kKeyStages);
     return tau_launch_status();
 }

@@ -51,6 +51,22 @@ __device__ __forceinline__ float block_sum(float value, float* scratch) {
     return scratch[32];
 }
 
+// What a gated product makes of a gate value and its up value: silu(gate) * up, or with `limit` > 0 the clamped form
+// g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = up held between -limit and limit.  For results that are rounded to bfloat16:
+// the fast exponential and quotient lose nothing then.
+constexpr float kClampedGateSlope = 1.702f;
+__device__ __forceinline__ float gated_value(float gate, float up, float limit) {
+    const bool clamped = limit > 0.0f;
+    const float g = clamped ? fminf(gate, limit) : gate;
+    const float u = clamped ? fminf(fmaxf(up, -limit), limit) + 1.0f : up;
+    return __fdividef(g, 1.0f + __expf(clamped ? -kClampedGateSlope * g : -g)) * u;
+}
+// The same to 32-bit accuracy.
+__device__ __forceinline__ float clamped_gate_exact(float gate, float up, float limit) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.0f + expf(-kClampedGateSlope * g)) * (u + 1.0f);
+}
+
 static inline int tau_launch_status() { return static_cast<int>(cudaGetLastError()); }
 
 // Programmatic dependent launch.  Every kernel of this library starts with `grid_dependents_launch()` (the next

@@ -51,11 +51,12 @@ __device__ __forceinline__ void copy_async_16(void* destination, const void* sou
 __device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// `Gated`: a block's 16 rows are 8 gate rows followed by their 8 up rows; it writes silu(gate) * up to `out[M, N / 2]`.
+// `Gated`: a block's 16 rows are 8 gate rows followed by their 8 up rows; it writes silu(gate) * up (or, with `gate_limit` > 0, the
+// clamped form) to `out[M, N / 2]`.
 template <int NB, typename TOut, bool Gated, int kWarps>
 __global__ void __launch_bounds__(kWarps * 32, TAU_SKINNY_MIN_BLOCKS)
 gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, const float* __restrict__ bias, TOut* __restrict__ out,
-                   int M, int N, int K, long long x_stride, long long w_stride, long long out_stride) {
+                   int M, int N, int K, long long x_stride, long long w_stride, long long out_stride, float gate_limit) {
     grid_dependents_launch();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int g = lane >> 2, t = lane & 3;
@@ -151,7 +152,7 @@ gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, const
             const float mine = round_through<bf16>(sum);
             const float other = __shfl_xor_sync(0xffffffffu, mine, 8);
             if (r < 8 && token < M && feature < N)
-                out[static_cast<size_t>(token) * out_stride + (row0 >> 1) + r] = from_float<TOut>(mine / (1.0f + expf(-mine)) * other);
+                out[static_cast<size_t>(token) * out_stride + (row0 >> 1) + r] = from_float<TOut>(gated_value(mine, other, gate_limit));
         } else if (token < M && feature < N) {
             out[static_cast<size_t>(token) * out_stride + feature] = from_float<TOut>(sum);
         }
@@ -160,7 +161,7 @@ gemm_skinny_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, const
 
 template <int NB, typename TOut, bool Gated, int kWarps>
 int launch_with(const void* x, const void* w, const float* bias, void* out, int M, int N, int K, long long x_stride, long long w_stride,
-                long long out_stride, cudaStream_t stream, int* resident_blocks) {
+                long long out_stride, float gate_limit, cudaStream_t stream, int* resident_blocks) {
     constexpr int bytes = ring_bytes(kWarps);
     static int resident = 0;   // blocks of this kernel that the device holds at once
     if (!resident) {
@@ -179,7 +180,7 @@ int launch_with(const void* x, const void* w, const float* bias, void* out, int 
     }
     const unsigned blocks = (N + kRows - 1) / kRows;
     tau_launch(gemm_skinny_kernel<NB, TOut, Gated, kWarps>, dim3(blocks), dim3(kWarps * 32), bytes, stream, static_cast<const bf16*>(x),
-               static_cast<const bf16*>(w), bias, static_cast<TOut*>(out), M, N, K, x_stride, w_stride, out_stride);
+               static_cast<const bf16*>(w), bias, static_cast<TOut*>(out), M, N, K, x_stride, w_stride, out_stride, gate_limit);
     return tau_launch_status();
 }
 
@@ -187,22 +188,22 @@ int launch_with(const void* x, const void* w, const float* bias, void* out, int 
 // resident) do not, the 12-warp form runs instead.
 template <int NB, typename TOut, bool Gated>
 int launch_typed(const void* x, const void* w, const float* bias, void* out, int M, int N, int K, long long x_stride, long long w_stride,
-                 long long out_stride, cudaStream_t stream) {
+                 long long out_stride, float gate_limit, cudaStream_t stream) {
     int wide = 0, narrow = 0;
-    int status = launch_with<NB, TOut, Gated, 16>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, stream, &wide);
-    if (status == 0) status = launch_with<NB, TOut, Gated, 12>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, stream, &narrow);
+    int status = launch_with<NB, TOut, Gated, 16>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, stream, &wide);
+    if (status == 0) status = launch_with<NB, TOut, Gated, 12>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, stream, &narrow);
     if (status != 0) return status;
     const int blocks = (N + kRows - 1) / kRows;
     if (blocks > wide && blocks <= narrow)
-        return launch_with<NB, TOut, Gated, 12>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, stream, nullptr);
-    return launch_with<NB, TOut, Gated, 16>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, stream, nullptr);
+        return launch_with<NB, TOut, Gated, 12>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, stream, nullptr);
+    return launch_with<NB, TOut, Gated, 16>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, stream, nullptr);
 }
 
 template <int NB, bool Gated>
 int launch(int out_dtype, const void* x, const void* w, const float* bias, void* out, int M, int N, int K, long long x_stride,
-           long long w_stride, long long out_stride, cudaStream_t stream) {
-    if (out_dtype == TAU_BF16) return launch_typed<NB, bf16, Gated>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, stream);
-    return launch_typed<NB, float, Gated>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, stream);
+           long long w_stride, long long out_stride, float gate_limit, cudaStream_t stream) {
+    if (out_dtype == TAU_BF16) return launch_typed<NB, bf16, Gated>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, stream);
+    return launch_typed<NB, float, Gated>(x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, stream);
 }
 
 }  // namespace
@@ -211,7 +212,7 @@ TAU_EXPORT int tau_gemm_skinny_max_rows() { return 32; }
 
 // bfloat16 inputs; `out_dtype` bfloat16 or float32.  Strides in elements.
 TAU_EXPORT int tau_gemm_skinny(int out_dtype, const void* x, const void* w, const float* bias, void* out, int M, int N, int K,
-                               long long x_stride, long long w_stride, long long out_stride, int gated, void* stream) {
+                               long long x_stride, long long w_stride, long long out_stride, int gated, float gate_limit, void* stream) {
     if (M <= 0 || N <= 0) return 0;
     if (!x || !w || !out || K <= 0 || M > 32 || (K & 7) || (x_stride & 7) || (w_stride & 7) ||
         (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15) ||
@@ -219,11 +220,11 @@ TAU_EXPORT int tau_gemm_skinny(int out_dtype, const void* x, const void* w, cons
         return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     if (gated) {
-        if (M <= 8) return launch<1, true>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, s);
-        if (M <= 16) return launch<2, true>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, s);
-        return launch<4, true>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, s);
+        if (M <= 8) return launch<1, true>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, s);
+        if (M <= 16) return launch<2, true>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, s);
+        return launch<4, true>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, s);
     }
-    if (M <= 8) return launch<1, false>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, s);
-    if (M <= 16) return launch<2, false>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, s);
-    return launch<4, false>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, s);
+    if (M <= 8) return launch<1, false>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, s);
+    if (M <= 16) return launch<2, false>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, s);
+    return launch<4, false>(out_dtype, x, w, bias, out, M, N, K, x_stride, w_stride, out_stride, gate_limit, s);
 }

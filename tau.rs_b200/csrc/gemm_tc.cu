@@ -177,12 +177,13 @@ struct Shared {
 };
 
 // `Gated`: the weight's rows come in groups of 16, 8 gate rows followed by their 8 up rows; the epilogue writes
-// silu(gate) * up, so `out` has N / 2 columns (crates/cuda-kernels/src/kernels/silu_and_mul.cu:51-76 as an epilogue).
+// silu(gate) * up, so `out` has N / 2 columns (crates/cuda-kernels/src/kernels/silu_and_mul.cu:51-76 as an epilogue), or, with
+// `gate_limit` > 0, the clamped form of `gated_value` below.
 template <int BN, typename TOut, bool Gated>
 __global__ void __launch_bounds__(kThreads, BN <= 128 ? 2 : 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap weight_map, const __grid_constant__ CUtensorMap input_map,
                const float* __restrict__ bias, TOut* __restrict__ out, int M, int N, int K, long long out_stride, int stages,
-               int splits, float* __restrict__ workspace, int* __restrict__ tickets, int clustered) {
+               int splits, float* __restrict__ workspace, int* __restrict__ tickets, int clustered, float gate_limit) {
     extern __shared__ uint8_t shared_raw[];
     Shared* shared = reinterpret_cast<Shared*>(shared_raw);
     uint8_t* tiles = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(shared_raw) + sizeof(Shared) + 1023) & ~uintptr_t(1023));
@@ -316,7 +317,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap weight_map, const __grid_cons
                     const float other = __shfl_xor_sync(0xffffffffu, mine, 8);
                     if ((lane & 8) == 0 && feature < N && token < M)
                         out[static_cast<size_t>(token) * out_stride + (feature >> 4) * 8 + (feature & 7)] =
-                            from_float<TOut>(__fdividef(mine, 1.0f + __expf(-mine)) * other);   // the result is rounded to bfloat16: the fast forms lose nothing
+                            from_float<TOut>(gated_value(mine, other, gate_limit));
                 } else if (feature < N && token < M) {
                     out[static_cast<size_t>(token) * out_stride + feature] = from_float<TOut>(value + offset);
                 }
@@ -413,7 +414,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap weight_map, const __grid_cons
                             const int feature = feature4 + i;
                             if ((group & 2) == 0 && feature < N && token < M)
                                 out[static_cast<size_t>(token) * out_stride + (feature >> 4) * 8 + (feature & 7)] =
-                                    from_float<TOut>(__fdividef(mine, 1.0f + __expf(-mine)) * other);
+                                    from_float<TOut>(gated_value(mine, other, gate_limit));
                         }
                     } else if (token < M) {
 #pragma unroll
@@ -468,7 +469,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap weight_map, const __grid_cons
                         const int feature = feature4 + i;
                         if ((group & 2) == 0 && feature < N)
                             out[static_cast<size_t>(token) * out_stride + (feature >> 4) * 8 + (feature & 7)] =
-                                from_float<TOut>(__fdividef(mine, 1.0f + __expf(-mine)) * other);
+                                from_float<TOut>(gated_value(mine, other, gate_limit));
                     }
                 } else {
 #pragma unroll
@@ -560,7 +561,7 @@ template <typename TOut, bool Gated>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap weight_map, const __grid_constant__ CUtensorMap input_map,
                     const float* __restrict__ bias, TOut* __restrict__ out, int M, int N, int K, long long out_stride, int stages,
-                    int vector_stores) {
+                    int vector_stores, float gate_limit) {
     extern __shared__ uint8_t shared_raw[];
     Shared* shared = reinterpret_cast<Shared*>(shared_raw);
     uint8_t* tiles = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(shared_raw) + sizeof(Shared) + 1023) & ~uintptr_t(1023));
@@ -686,7 +687,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap weight_map, const __grid
 #pragma unroll
                     for (int j = 0; j < 8; ++j) {
                         const float gate = round_through<bf16>(value[16 * group + j]), up = round_through<bf16>(value[16 * group + 8 + j]);
-                        result[j] = __fdividef(gate, 1.0f + __expf(-gate)) * up;   // the result is rounded to bfloat16: the fast forms lose nothing
+                        result[j] = gated_value(gate, up, gate_limit);
                     }
 #pragma unroll
                     for (int j = 0; j < 4; ++j) packed[4 * group + j] = pack_pair(result[2 * j], result[2 * j + 1]);
@@ -855,6 +856,7 @@ struct SplitPlan {
     long long workspace_floats;
     int* tickets;            // 4096 ints, zero between launches
     int cluster;             // 0: the ranges of a tile meet in the workspace even where a cluster could be formed
+    float gate_limit;        // of a gated product: 0 for silu(gate) * up, else the clamped form's limit
 };
 
 template <int BN, typename TOut, bool Gated>
@@ -931,19 +933,19 @@ int launch(const CUtensorMap& weight_map, const CUtensorMap& input_map, const fl
             const int cluster_bytes = shared_for(whole, &cluster_stages);
             if (cluster_stages * stage_bytes >= BN * BM * 4) {   // the partial tile lies over the stages
                 tau_launch_clusters(splits, gemm_tc_kernel<BN, TOut, Gated>, dim3(blocks), dim3(kThreads), cluster_bytes, stream, weight_map, input_map,
-                                    bias, static_cast<TOut*>(out), M, N, K, out_stride, cluster_stages, splits, plan.workspace, plan.tickets, 1);
+                                    bias, static_cast<TOut*>(out), M, N, K, out_stride, cluster_stages, splits, plan.workspace, plan.tickets, 1, plan.gate_limit);
                 return tau_launch_status();
             }
         }
     }
     tau_launch(gemm_tc_kernel<BN, TOut, Gated>, dim3(blocks), dim3(kThreads), shared_bytes, stream, weight_map, input_map, bias, static_cast<TOut*>(out), M, N, K,
-               out_stride, stages, splits, plan.workspace, plan.tickets, 0);
+               out_stride, stages, splits, plan.workspace, plan.tickets, 0, plan.gate_limit);
     return tau_launch_status();
 }
 
 template <typename TOut, bool Gated>
 int launch_pair(const CUtensorMap& weight_map, const CUtensorMap& input_map, const float* bias, void* out, int M, int N, int K,
-                long long out_stride, cudaStream_t stream) {
+                long long out_stride, float gate_limit, cudaStream_t stream) {
     constexpr int stage_bytes = (kPairHalf + BM) * BK * 2;
     int stages = (200 * 1024) / stage_bytes;
     if (stages > 8) stages = 8;
@@ -960,14 +962,14 @@ int launch_pair(const CUtensorMap& weight_map, const CUtensorMap& input_map, con
     const int group = Gated ? 16 : (sizeof(TOut) == 2 ? 8 : 4);
     const int vector_stores = (reinterpret_cast<uintptr_t>(out) % 16 == 0) && (out_stride * sizeof(TOut)) % 16 == 0 && N % group == 0;
     tau_launch_clusters(2, gemm_tc_pair_kernel<TOut, Gated>, dim3(2 * pairs), dim3(kThreads), shared_bytes, stream, weight_map, input_map, bias,
-                        static_cast<TOut*>(out), M, N, K, out_stride, stages, vector_stores);
+                        static_cast<TOut*>(out), M, N, K, out_stride, stages, vector_stores, gate_limit);
     return tau_launch_status();
 }
 
 template <typename TOut, bool Gated>
 int dispatch(const CUtensorMap& weight_map, const CUtensorMap& input_map, int box, const float* bias, void* out, int M, int N, int K,
              long long out_stride, const SplitPlan& plan, cudaStream_t stream) {
-    if (box == kPairHalf + 1) return launch_pair<TOut, Gated>(weight_map, input_map, bias, out, M, N, K, out_stride, stream);
+    if (box == kPairHalf + 1) return launch_pair<TOut, Gated>(weight_map, input_map, bias, out, M, N, K, out_stride, plan.gate_limit, stream);
     switch (box) {
         case 16: return launch<16, TOut, Gated>(weight_map, input_map, bias, out, M, N, K, out_stride, plan, stream);
         case 32: return launch<32, TOut, Gated>(weight_map, input_map, bias, out, M, N, K, out_stride, plan, stream);
@@ -988,19 +990,20 @@ TAU_EXPORT int tau_gemm_tc_status() {
 }
 
 // bfloat16 inputs; `out_dtype` bfloat16 or float32.  Strides in elements.  `token_box` = 0 picks the token tile from M.
-// `gated`: rows of `w` are groups of 8 gate rows and their 8 up rows; `out` is `[M, N / 2]` = silu(gate) * up.
+// `gated`: rows of `w` are groups of 8 gate rows and their 8 up rows; `out` is `[M, N / 2]` = silu(gate) * up, or with `gate_limit` L > 0
+// g sigmoid(1.702 g) (u + 1) with g = min(gate, L), u = min(max(up, -L), L).
 // `workspace` (`workspace_floats` floats) and `tickets` (4096 ints, zero, left at zero) allow cutting along K; `splits` = 0
 // lets the launcher choose, 1 forbids it, more asks for exactly that many ranges (refused if they do not fit).
 // `cluster`: 0 keeps the ranges of a tile from meeting in a cluster's shared memory (they meet in the workspace).
 // `pair`: 1 runs 256 x 256 tiles on pairs of SMs (only with the 256-token tile), 0 never, -1 where the 256-token tile is chosen.
 TAU_EXPORT int tau_gemm_tc(int out_dtype, const void* x, const void* w, const float* bias, void* out, int M, int N, int K,
                            long long x_stride, long long w_stride, long long out_stride, int token_box, int gated, int splits,
-                           void* workspace, long long workspace_floats, void* tickets, int pair, int cluster, void* stream) {
+                           void* workspace, long long workspace_floats, void* tickets, int pair, int cluster, float gate_limit, void* stream) {
     if (M <= 0 || N <= 0) return 0;
     if (!x || !w || !out || K <= 0 || (K & 7) || (x_stride & 7) || (w_stride & 7) || (reinterpret_cast<uintptr_t>(x) & 15) ||
         (reinterpret_cast<uintptr_t>(w) & 15) || (out_dtype != TAU_BF16 && out_dtype != TAU_F32) || splits < 0)
         return cudaErrorInvalidValue;
-    const SplitPlan plan{splits, static_cast<float*>(workspace), workspace_floats, static_cast<int*>(tickets), cluster};
+    const SplitPlan plan{splits, static_cast<float*>(workspace), workspace_floats, static_cast<int*>(tickets), cluster, gated ? gate_limit : 0.0f};
     int box = token_box;
     if (box == 0) box = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
     if (box != 16 && box != 32 && box != 64 && box != 128 && box != 192 && box != 256) return cudaErrorInvalidValue;
@@ -1088,7 +1091,7 @@ TAU_EXPORT int tau_gemm_tc_groups(int out_dtype, const void* x, const void* w, v
         result = tau_gemm_tc(out_dtype, static_cast<const bf16*>(x) + static_cast<size_t>(begin) * x_stride,
                              static_cast<const bf16*>(w) + static_cast<size_t>(group) * w_group, nullptr,
                              static_cast<char*>(out) + static_cast<size_t>(begin) * out_stride * out_bytes, rows, N, K, x_stride, w_stride,
-                             out_stride, 0, gated, spread ? 1 : 0, workspace, workspace_floats, tickets, -1, 1,
+                             out_stride, 0, gated, spread ? 1 : 0, workspace, workspace_floats, tickets, -1, 1, 0.0f,
                              spread ? static_cast<void*>(group_streams[launched % kGroupStreams]) : stream);
         ++launched;
     }

@@ -82,13 +82,13 @@ _CLASS_OF = {
     "gemm_skinny": "product", "gemm_tc": "product", "attention_prepare": "attention", "attention": "attention",
     "attention_decode": "attention", "attention_prefill": "attention", "attention_prefill_tc": "attention", "argmax": "selection",
     "sample_gumbel": "selection", "store_words_host": "selection", "random_normal": "other",
-    "stream_add_norm": "norm", "normed_pair_sum": "norm", "gated_group_norm": "norm", "gemm_simt_batched": "product", "linear_recurrence": "recurrence",
+    "stream_add_norm": "norm", "stream_add_tanh": "norm", "soft_cap": "other", "normed_pair_sum": "norm", "gated_group_norm": "norm", "gemm_simt_batched": "product", "linear_recurrence": "recurrence",
     "latent_prepare": "attention", "latent_attention": "attention", "latent_expand": "attention", "moe_route": "routing", "moe_gate_up": "experts", "moe_down": "experts", "gemm_tc_groups": "experts", "moe_sort": "routing", "moe_gather": "routing",
     "moe_combine": "routing", "diff_prepare": "attention", "diff_attention": "attention", "diff_combine": "attention", "causal_taps": "norm", "gated_add_norm": "norm",
     "side_gate": "activation", "unit_add_mix": "norm", "norm_rows": "norm", "relu_squared": "activation",
     "short_conv": "recurrence", "delta_prepare": "recurrence", "delta_rule": "recurrence", "selective_scan": "recurrence",
-    "masked_prepare": "attention", "masked_attention": "attention", "gated_rows": "attention",
-    "token_shift": "recurrence", "tanh": "activation", "channel_decay": "recurrence", "wkv": "recurrence",
+    "masked_prepare": "attention", "masked_attention": "attention", "talking_decode": "attention", "gated_rows": "attention",
+    "token_shift": "recurrence", "tanh": "activation", "channel_decay": "recurrence", "wkv": "recurrence", "forget_gates": "recurrence", "turn_heads": "recurrence",
 }
 _timing = None     # while timing: [last event, [(class, event after the launch), ...]]
 
@@ -244,6 +244,47 @@ def stream_add_norm(stream, branches, weight, eps: float, out, rows=None, update
                                        ctypes.c_int(groups), ctypes.c_float(branch_scale), _stream()), "stream_add_norm")
 
 
+def stream_add_tanh(stream, branches, alpha, weight, bias, out, rows=None, update: bool = True, branch_scale: float = 1.0) -> None:
+    """What `stream_add_norm` does with an element-wise tanh in the norm's place: `sum = stream[r] + branch_scale * (a[r] + b[r])` in 32-bit;
+    with `update` the sum replaces `stream[r]`; `out[i] = tanh(alpha * sum) * weight + bias`, rounded once to the output's dtype.  `alpha` is
+    one float32 number on the device."""
+    if branches is None:
+        branches = ()
+    elif not isinstance(branches, (tuple, list)):
+        branches = (branches,)
+    branches = tuple(branch for branch in branches if branch is not None)
+    _require(len(branches) <= 2, "at most two branches join the stream at once")
+    _on_device(stream, alpha, weight, bias, out, rows, *branches)
+    width = stream.shape[-1]
+    _f32_vector(alpha, 1, "alpha")
+    _f32_vector(weight, width, "the norm weight")
+    _f32_vector(bias, width, "the norm bias")
+    _require(stream.dtype == torch.float32 and stream.is_contiguous() and out.is_contiguous() and out.shape[-1] == width,
+             "the stream must be contiguous float32 and the output as wide")
+    for branch in branches:
+        _require(branch.shape == stream.shape and branch.is_contiguous(), "a branch must match the stream")
+    _require(not (update and rows is not None), "rows are gathered from a stream that is left as it is")
+    if rows is not None:
+        _int_vector(rows, "row numbers")
+    count = out.numel() // width
+    _require(count == (rows.shape[0] if rows is not None else stream.numel() // width), "output row count does not match")
+    first = branches[0] if branches else None
+    second = branches[1] if len(branches) > 1 else None
+    library = build.load_library("stream32.cu")
+    _check(library.tau_stream_add_tanh(_code(out), _pointer(stream), _pointer(first), ctypes.c_int(_code(first) if first is not None else 0),
+                                       _pointer(second), ctypes.c_int(_code(second) if second is not None else 0), _pointer(rows), _pointer(alpha),
+                                       _pointer(weight), _pointer(bias), _pointer(out), ctypes.c_int(count), ctypes.c_int(width),
+                                       ctypes.c_int(1 if update else 0), ctypes.c_float(branch_scale), _stream()), "stream_add_tanh")
+
+
+def soft_cap(values, cap: float) -> None:
+    """`values = cap * tanh(values / cap)` in place, float32."""
+    _on_device(values)
+    _require(values.dtype == torch.float32 and values.is_contiguous() and cap > 0.0, "the values must be contiguous float32 and the cap positive")
+    library = build.load_library("stream32.cu")
+    _check(library.tau_soft_cap(_pointer(values), ctypes.c_longlong(values.numel()), ctypes.c_float(cap), _stream()), "soft_cap")
+
+
 def normed_pair_sum(left, right, left_weight, right_weight, eps: float, left_scale: float, right_scale: float, out) -> None:
     """`out = left_scale * left / rms(left) * left_weight + right_scale * right / rms(right) * right_weight`, each root mean square
     over the whole row (eps inside the root); everything float32 [rows, width]."""
@@ -262,7 +303,7 @@ def normed_pair_sum(left, right, left_weight, right_weight, eps: float, left_sca
 def gated_group_norm(values, weight, gate, out, groups: int, eps: float, normalize: bool, silu_gate: bool = False) -> None:
     """`values` [rows, width] in 32-bit; with `normalize` each of the `groups` equal parts of a row is divided by its root
     mean square (eps inside the root); then times `weight` (float32 [width] or None), times `sigmoid(gate)` or, with `silu_gate`,
-    `gate * sigmoid(gate)` (the output's dtype, [rows, width], rows any distance apart, or None); rounded once to the output's
+    `gate * sigmoid(gate)` (float32 or bfloat16 [rows, width], rows any distance apart, or None); rounded once to the output's
     dtype.  The output's rows may lie any distance apart too (a column range of a wider tensor)."""
     _on_device(values, weight, gate, out)
     rows, width = values.shape
@@ -271,16 +312,17 @@ def gated_group_norm(values, weight, gate, out, groups: int, eps: float, normali
     _require(groups > 0 and width % groups == 0, "the groups must divide the width")
     _f32_vector(weight, width, "the weight")
     if gate is not None:
-        _require(gate.dtype == out.dtype and gate.shape == values.shape and gate.stride(1) == 1, "the gate must have the output's dtype and shape")
+        _require(gate.shape == values.shape and gate.stride(1) == 1, "the gate must have the values' shape")
     library = build.load_library("stream32.cu")
-    _check(library.tau_gated_group_norm(_code(out), _pointer(values), _pointer(weight), _pointer(gate),
+    _check(library.tau_gated_group_norm(_code(out), _pointer(values), _pointer(weight), _pointer(gate), ctypes.c_int(0 if gate is None else _code(gate)),
                                         ctypes.c_longlong(0 if gate is None else gate.stride(0)), _pointer(out), ctypes.c_longlong(out.stride(0)), ctypes.c_int(rows),
                                         ctypes.c_int(groups), ctypes.c_int(width // groups), ctypes.c_float(eps), ctypes.c_int(1 if normalize else 0),
                                         ctypes.c_int(1 if silu_gate else 0), _stream()), "gated_group_norm")
 
 
-def silu_mul(stacked, out, relu: bool = False) -> None:
-    """`out[r, c] = silu(stacked[r, c]) * stacked[r, width + c]`; with `relu` the activation is `max(z, 0)` instead."""
+def silu_mul(stacked, out, relu: bool = False, limit: float = 0.0) -> None:
+    """`out[r, c] = silu(stacked[r, c]) * stacked[r, width + c]`; with `relu` the activation is `max(z, 0)` instead; with `limit` L > 0 the
+    result is `g sigmoid(1.702 g) (u + 1)`, `g = min(stacked[r, c], L)` and `u = stacked[r, width + c]` held between -L and L."""
     _on_device(stacked, out)
     width = out.shape[-1]
     _require(stacked.shape[-1] == 2 * width and stacked.shape[0] == out.shape[0] and stacked.dtype == out.dtype,
@@ -288,7 +330,7 @@ def silu_mul(stacked, out, relu: bool = False) -> None:
     _require(stacked.is_contiguous() and out.is_contiguous(), "tensors must be contiguous")
     library = build.load_library("elementwise.cu")
     _check(library.tau_silu_mul(_code(out), _pointer(stacked), _pointer(out), ctypes.c_longlong(out.shape[0]), ctypes.c_int(width),
-                                ctypes.c_int(1 if relu else 0), _stream()), "silu_mul")
+                                ctypes.c_int(1 if relu else 0), ctypes.c_float(limit), _stream()), "silu_mul")
 
 
 # ---------------------------------------------------------------------------- products
@@ -344,10 +386,11 @@ def _skinny_fits(values, weight, out) -> bool:
             and weight.data_ptr() % 16 == 0)
 
 
-def gemm_skinny(values, weight, bias, out, gated: bool = False) -> None:
+def gemm_skinny(values, weight, bias, out, gated: bool = False, gate_limit: float = 0.0) -> None:
     """bfloat16 product for at most 32 activation rows, bound by streaming `weight` once.
 
-    `gated`: the weight's rows are groups of 8 gate rows and their 8 up rows; `out` is `[M, N / 2]` = silu(gate) * up.
+    `gated`: the weight's rows are groups of 8 gate rows and their 8 up rows; `out` is `[M, N / 2]` = silu(gate) * up, or with
+    `gate_limit` > 0 the clamped form (`silu_mul`'s `limit`).
     """
     _on_device(values, weight, bias, out)
     rows, depth = values.shape
@@ -362,7 +405,7 @@ def gemm_skinny(values, weight, bias, out, gated: bool = False) -> None:
     _check(library.tau_gemm_skinny(_code(out), _pointer(values), _pointer(weight), _pointer(bias), _pointer(out), ctypes.c_int(rows),
                                    ctypes.c_int(features), ctypes.c_int(depth), ctypes.c_longlong(values.stride(0)),
                                    ctypes.c_longlong(weight.stride(0)), ctypes.c_longlong(out.stride(0)), ctypes.c_int(1 if gated else 0),
-                                   _stream()), "gemm_skinny")
+                                   ctypes.c_float(gate_limit), _stream()), "gemm_skinny")
 
 
 def _tc_fits(values, weight, out) -> bool:
@@ -398,10 +441,12 @@ def _tc_workspace_for(device):
     return entry
 
 
-def gemm_tc(values, weight, bias, out, token_box: int = 0, gated: bool = False, splits: int = 0, pair: int = -1, cluster: bool = True) -> None:
+def gemm_tc(values, weight, bias, out, token_box: int = 0, gated: bool = False, splits: int = 0, pair: int = -1, cluster: bool = True,
+            gate_limit: float = 0.0) -> None:
     """bfloat16 product on the tcgen05 tensor cores (TMA-fed, accumulator in tensor memory); any M and N, K % 8 == 0.
 
-    `gated`: the weight's rows are groups of 8 gate rows and their 8 up rows; `out` is `[M, N / 2]` = silu(gate) * up.
+    `gated`: the weight's rows are groups of 8 gate rows and their 8 up rows; `out` is `[M, N / 2]` = silu(gate) * up, or with
+    `gate_limit` > 0 the clamped form (`silu_mul`'s `limit`).
     `splits`: K ranges that the product is cut into (0: chosen from the sizes, for products with few tiles).
     `cluster`: False makes the K ranges of a tile meet in a workspace in global memory even where they could meet in the
     shared memory of a thread-block cluster.
@@ -422,7 +467,8 @@ def gemm_tc(values, weight, bias, out, token_box: int = 0, gated: bool = False, 
                                ctypes.c_int(features), ctypes.c_int(depth), ctypes.c_longlong(values.stride(0)),
                                ctypes.c_longlong(weight.stride(0)), ctypes.c_longlong(out.stride(0)), ctypes.c_int(token_box),
                                ctypes.c_int(1 if gated else 0), ctypes.c_int(splits), _pointer(workspace),
-                               ctypes.c_longlong(workspace.numel()), _pointer(tickets), ctypes.c_int(pair), ctypes.c_int(1 if cluster else 0), _stream()), "gemm_tc")
+                               ctypes.c_longlong(workspace.numel()), _pointer(tickets), ctypes.c_int(pair), ctypes.c_int(1 if cluster else 0),
+                               ctypes.c_float(gate_limit), _stream()), "gemm_tc")
 
 
 def gemm_tc_groups(values, weights, out, bounds, gated: bool = False) -> None:
@@ -478,13 +524,13 @@ def gated_fits(in_features: int, out_features: int, dtype) -> bool:
     return _prefer_optimized and dtype == torch.bfloat16 and in_features % 8 == 0 and out_features % GATE_GROUP == 0
 
 
-def linear_gated(values, weight, out) -> None:
+def linear_gated(values, weight, out, limit: float = 0.0) -> None:
     """`out = silu(values @ gate.T) * (values @ up.T)` in one product; `weight` holds groups of 8 gate rows followed by
-    their 8 up rows (see `parts.linear.StackedLinear(interleave=...)`)."""
+    their 8 up rows (see `parts.linear.StackedLinear(interleave=...)`).  `limit` > 0: the clamped form of `silu_mul` instead."""
     if _skinny_fits(values, weight, out) and _skinny_wins(values, weight):
-        return gemm_skinny(values, weight, None, out, gated=True)
+        return gemm_skinny(values, weight, None, out, gated=True, gate_limit=limit)
     _require(_tc_fits(values, weight, out), "the gated product needs bfloat16, K % 8 == 0 and 16-byte aligned rows")
-    gemm_tc(values, weight, None, out, gated=True)
+    gemm_tc(values, weight, None, out, gated=True, gate_limit=limit)
 
 
 def linear(values, weight, bias, out) -> None:
@@ -699,14 +745,17 @@ _prefill_schedule = {}   # (device, stream) -> the two counters by which the blo
 
 def attention_prefill_tc(queries, keys, values, out, cu_seqlens, seq_start, page_rows, n_heads: int, n_kv_heads: int, head_dim: int,
                          scale: float, window: int, chunk: int = 0, sink: bool = False, out_scale: float = 1.0, distance=None, sigmoid_weights: bool = False,
-                         head_offset=None, head_gate=None) -> None:
+                         head_offset=None, head_gate=None, keep_first: int = 0, segmented: bool = False) -> None:
     """The same as `attention_prefill` on the tcgen05 tensor cores (accumulators in tensor memory); head sizes 64 and 128.
     Beyond it: with `chunk` a query sees only the keys of its own chunk of `chunk` positions (counted from position 0 of the
     sequence) instead of a window; with `sink` the softmax's denominator has one added; the result is multiplied by `out_scale`;
     `out` may be a column range of a wider tensor whose rows start on 16-byte borders.  `distance` (float32 [n_heads, 2] = (r1, r2)):
     `r1 * ln(1 + r2 * (i - j))` is taken off the score of key j for the query at i.  `sigmoid_weights`: every visible key weighs
     `sigmoid(score + head_offset[head])` (float32 [n_heads] or None) instead of its share of a softmax.  `head_gate` (bfloat16
-    [tokens, n_heads], rows any distance apart): a head's result is multiplied by the sigmoid of its number."""
+    [tokens, n_heads], rows any distance apart): a head's result is multiplied by the sigmoid of its number.  `keep_first`: the
+    sequence's first that many positions stay visible beside a window.  `segmented`: a query has a piece of `head_dim` elements for each
+    key head (`queries` [tokens, n_heads * n_kv_heads * head_dim]) and a score is the sum over the key heads; where
+    `attention_prefill_tc_segments_fit`."""
     _on_device(queries, keys, values, out, cu_seqlens, seq_start, page_rows, distance, head_offset, head_gate)
     if distance is not None:
         _require(distance.dtype == torch.float32 and distance.shape == (n_heads, 2) and distance.is_contiguous(), "the distance numbers must be float32 [heads, 2]")
@@ -718,12 +767,13 @@ def attention_prefill_tc(queries, keys, values, out, cu_seqlens, seq_start, page
     n_seqs = seq_start.numel()
     _require(head_dim in (64, 128), "the tensor-core prefill kernel serves head sizes 64 and 128")
     _require(queries.dtype == torch.bfloat16 == out.dtype == keys.dtype == values.dtype, "the tensor-core prefill kernel is bfloat16 only")
-    _require(queries.shape == (tokens, n_heads * head_dim) and out.shape == queries.shape and queries.is_contiguous() and out.stride(1) == 1
+    _require(queries.shape == (tokens, n_heads * head_dim * (n_kv_heads if segmented else 1)) and out.shape == (tokens, n_heads * head_dim) and queries.is_contiguous() and out.stride(1) == 1
              and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0, "queries and output must be [tokens, n_heads * head_dim], output rows on 16-byte borders")
     _require(n_heads % n_kv_heads == 0, "n_heads must be a multiple of n_kv_heads")
     _require(keys.shape[1:] == (n_kv_heads, PAGE_TOKENS, head_dim) and keys.is_contiguous() and values.is_contiguous()
              and values.shape == keys.shape, "cache pages must be [pages, n_kv_heads, 64, head_dim]")
     _require(not (window and chunk), "a window or a chunk, not both")
+    _require(keep_first >= 0 and (not keep_first or window), "first positions are kept beside a window")
     _int_vector(cu_seqlens, "cu_seqlens")
     _int_vector(seq_start, "seq_start")
     _require(cu_seqlens.numel() == n_seqs + 1 and page_rows.dtype == torch.int32 and page_rows.dim() == 2 and page_rows.is_contiguous()
@@ -739,7 +789,13 @@ def attention_prefill_tc(queries, keys, values, out, cu_seqlens, seq_start, page
         ctypes.c_int(tokens), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_float(scale), ctypes.c_int(window), ctypes.c_int(chunk),
         ctypes.c_int(1 if sink else 0), ctypes.c_float(out_scale), ctypes.c_longlong(out.stride(0)), _pointer(schedule), _pointer(distance),
         ctypes.c_int(1 if sigmoid_weights else 0), _pointer(head_offset), _pointer(head_gate), ctypes.c_longlong(0 if head_gate is None else head_gate.stride(0)),
-        _stream()), "attention_prefill_tc")
+        ctypes.c_int(keep_first), ctypes.c_int(1 if segmented else 0), _stream()), "attention_prefill_tc")
+
+
+def attention_prefill_tc_segments_fit(head_dim: int, n_kv_heads: int) -> bool:
+    """Whether the segmented form of `attention_prefill_tc` serves that many key heads."""
+    library = build.load_library("attention_prefill_tc.cu", (f"TAU_HEAD_DIM={head_dim}",))
+    return bool(library.tau_attention_prefill_tc_segments_fit(ctypes.c_int(n_kv_heads)))
 
 
 def attention_prefill_tc_status(head_dim: int) -> int:
@@ -1272,7 +1328,7 @@ MASKED_STAGED_WARPS = 4      # query heads of a key/value head that one block of
 
 def masked_prepare(projected, q_weight, k_weight, eps: float, frequency, rotary_dim: int, magnitude: float, queries, rows, positions, token_seq,
                    page_rows, n_heads: int, n_kv_heads: int, dim: int, vdim: int, write_rows: bool = True, value_pages=None,
-                   temperature=None) -> None:
+                   temperature=None, talk=None, first_values=None, value_share=None) -> None:
     """`projected` [tokens, >= n_heads * dim + n_kv_heads * (dim + vdim)] holds queries, keys and values side by side.  With weights
     (float32 [n_heads * dim] and [n_kv_heads * dim]) the queries, and the keys, are divided by the root mean square over their
     whole projection (eps inside the root) and multiplied by the weight.  In every head element `i` of the first `rotary_dim` is
@@ -1281,14 +1337,25 @@ def masked_prepare(projected, q_weight, k_weight, eps: float, frequency, rotary_
     [pages, 64, n_kv_heads * (dim + vdim)] as [keys of all heads | values], or, with `value_pages`, to pages of ordinary heads:
     keys to `rows` [pages, n_kv_heads, 64, dim], values to `value_pages` [pages, n_kv_heads, 64, vdim].  Without `write_rows` the
     projection need hold the queries alone.  `temperature` = (coef, every): the query at position p is multiplied by
-    `1 + coef * ln(floor((p + 1) / every) + 1)`."""
-    _on_device(projected, q_weight, k_weight, frequency, queries, rows, positions, token_seq, page_rows, value_pages)
+    `1 + coef * ln(floor((p + 1) / every) + 1)`.  `talk` (float32 [n_heads, n_heads]): instead of its own query every head gets the
+    queries of all heads weighed by its row of `talk` and added up per key head, `queries` being [tokens, n_heads, n_kv_heads * dim];
+    against the keys of all key heads side by side (`masked_attention`'s `shared_keys`) they give the mixed scores.  `first_values`
+    ([tokens, n_kv_heads * vdim], rows any distance apart) and `value_share` (one float32 number on the device): the values that are
+    cached are `(1 - share) * v + share * first`."""
+    _on_device(projected, q_weight, k_weight, frequency, queries, rows, positions, token_seq, page_rows, value_pages, talk, first_values, value_share)
     tokens = projected.shape[0]
     row_width = n_kv_heads * (dim + vdim)
     _require(projected.shape[1] >= n_heads * dim + (row_width if write_rows else 0) and projected.stride(1) == 1, "the projection is too narrow")
     coef, every = (0.0, 0) if temperature is None else (float(temperature[0]), int(temperature[1]))
     _require(every >= 0, "the temperature's period must be positive")
-    _require(queries.shape == (tokens, n_heads, dim) and queries.is_contiguous() and queries.dtype == projected.dtype, "queries must be [tokens, n_heads, dim]")
+    _require(queries.shape == (tokens, n_heads, dim if talk is None else n_kv_heads * dim) and queries.is_contiguous() and queries.dtype == projected.dtype,
+             "queries must be [tokens, n_heads, dim], or with talk [tokens, n_heads, n_kv_heads * dim]")
+    _f32_vector(talk, n_heads * n_heads, "the heads' mixing weights")
+    if first_values is not None:
+        _require(first_values.shape == (tokens, n_kv_heads * vdim) and first_values.stride(1) == 1 and first_values.dtype == projected.dtype,
+                 "the first values must be [tokens, n_kv_heads * vdim] in the projection's dtype")
+        _require(value_share is not None, "the share of the first values is needed")
+        _f32_vector(value_share, 1, "the share of the first values")
     _f32_vector(q_weight, n_heads * dim, "the query norm weight")
     _f32_vector(k_weight, n_kv_heads * dim, "the key norm weight")
     _require(rotary_dim % 2 == 0 and 0 <= rotary_dim <= dim, "rotary_dim must be even and at most dim")
@@ -1305,7 +1372,8 @@ def masked_prepare(projected, q_weight, k_weight, eps: float, frequency, rotary_
         _pointer(frequency if rotary_dim else None), ctypes.c_int(rotary_dim), ctypes.c_float(magnitude), _pointer(queries), _pointer(rows if write_rows else None),
         _pointer(value_pages if write_rows else None), _pointer(positions), _pointer(token_seq), _pointer(page_rows), ctypes.c_int(page_rows.shape[1] if write_rows else 0), ctypes.c_int(PAGE_TOKENS),
         ctypes.c_int(tokens), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(dim), ctypes.c_int(vdim), ctypes.c_int(1 if write_rows else 0),
-        ctypes.c_float(coef), ctypes.c_int(every), _stream()), "masked_prepare")
+        ctypes.c_float(coef), ctypes.c_int(every), _pointer(talk), _pointer(first_values), ctypes.c_longlong(0 if first_values is None else first_values.stride(0)),
+        _pointer(value_share), _stream()), "masked_prepare")
 
 
 def _require_masked_pages(rows, value_pages, dtype, n_kv_heads: int, dim: int, vdim: int) -> None:
@@ -1318,7 +1386,7 @@ def _require_masked_pages(rows, value_pages, dtype, n_kv_heads: int, dim: int, v
 
 def masked_attention(queries, rows, out, step, page_rows, n_kv_heads: int, vdim: int, scale: float, window: int = 0, chunk: int = 0, sink: bool = False,
                      out_scale: float = 1.0, value_pages=None, staged: bool = False, distance=None, sigmoid_weights: bool = False, head_offset=None,
-                     gate=None, gate_per_head: bool = False, splits: int = 1) -> None:
+                     gate=None, gate_per_head: bool = False, splits: int = 1, keep_first: int = 0, shared_keys: bool = False) -> None:
     """Causal softmax attention of every token over the cached rows of its sequence: within `window` positions (if not 0), or
     within the token's own chunk of `chunk` positions counted from position 0 (if not 0); with `sink` the softmax's denominator has
     one added.  `out` [tokens, n_heads * vdim] (rows any distance apart) receives the result times `out_scale`.  Scores, weights
@@ -1329,9 +1397,14 @@ def masked_attention(queries, rows, out, step, page_rows, n_kv_heads: int, vdim:
     softmax every visible key weighs `sigmoid(score + head_offset[head])` (float32 [n_heads] or None), not normalised.  `gate`
     ([tokens, n_heads] with `gate_per_head`, else [tokens, n_heads * vdim]; the queries' dtype; rows any distance apart): the result
     is multiplied by its sigmoid.  `splits` > 1 (with `staged`): every token's context is cut into that many ranges that as many
-    blocks walk, and a second launch joins them."""
+    blocks walk, and a second launch joins them.  `keep_first`: the sequence's first that many positions stay visible however far they
+    lie before the window.  `shared_keys`: a query has `n_kv_heads * dim` elements and asks the keys of all key heads side by side."""
     _on_device(queries, rows, out, page_rows, value_pages, distance, head_offset, gate)
     tokens, n_heads, dim = queries.shape
+    if shared_keys:
+        _require(dim % n_kv_heads == 0, "a query against all key heads has a piece for each")
+        dim //= n_kv_heads
+    _require(keep_first >= 0, "the kept first positions cannot be negative")
     if distance is not None:
         _require(distance.dtype == torch.float32 and distance.shape == (n_heads, 2) and distance.is_contiguous(), "the distance numbers must be float32 [heads, 2]")
     _f32_vector(head_offset, n_heads, "the heads' offsets")
@@ -1354,7 +1427,43 @@ def masked_attention(queries, rows, out, step, page_rows, n_kv_heads: int, vdim:
         ctypes.c_int(dim), ctypes.c_int(vdim), ctypes.c_float(scale), ctypes.c_int(window), ctypes.c_int(chunk), ctypes.c_int(1 if sink else 0),
         ctypes.c_float(out_scale), ctypes.c_int(1 if staged else 0), _pointer(distance), ctypes.c_int(1 if sigmoid_weights else 0), _pointer(head_offset),
         _pointer(gate), ctypes.c_longlong(0 if gate is None else gate.stride(0)), ctypes.c_int(1 if gate_per_head else 0), ctypes.c_int(splits), _pointer(partial),
-        _stream()), "masked_attention", 2 if splits > 1 else 1)
+        ctypes.c_int(keep_first), ctypes.c_int(1 if shared_keys else 0), _stream()), "masked_attention", 2 if splits > 1 else 1)
+
+
+_talking_fits = {}
+
+
+def talking_decode_fits(dtype, n_heads: int, n_kv_heads: int, dim: int, vdim: int) -> bool:
+    """Whether `talking_decode` serves these sizes (else: `masked_attention` with mixed queries)."""
+    key = (dtype, n_heads, n_kv_heads, dim, vdim)
+    if key not in _talking_fits:
+        library = build.load_library("masked_attention.cu")
+        _talking_fits[key] = bool(library.tau_talking_decode_fits(*(ctypes.c_int(value) for value in (_DTYPE_CODE[dtype], n_heads, n_kv_heads, dim, vdim))))
+    return _talking_fits[key]
+
+
+def talking_decode(queries, rows, talk, out, step, page_rows, n_kv_heads: int, vdim: int, scale: float, window: int = 0, keep_first: int = 0,
+                   out_scale: float = 1.0, value_pages=None, splits: int = 1) -> None:
+    """Causal softmax attention of single tokens whose scores are mixed over the heads first: `score_h <- sum_g talk[h, g] score_g` (`talk`
+    float32 [n_heads, n_heads]), over the last `window` positions (0: all) and the sequence's first `keep_first`.  `queries` [tokens,
+    n_heads, dim]; the cache in either layout of `masked_prepare`; `out` [tokens, n_heads * vdim], rows any distance apart.  `splits` > 1:
+    that many ranges of every token's keys, which a second launch joins."""
+    _on_device(queries, rows, talk, out, page_rows, value_pages)
+    tokens, n_heads, dim = queries.shape
+    _f32_vector(talk, n_heads * n_heads, "the heads' mixing weights")
+    _require(queries.is_contiguous() and out.shape == (tokens, n_heads * vdim) and out.stride(1) == 1 and out.dtype == queries.dtype == rows.dtype,
+             "queries must be [tokens, n_heads, dim] and the output [tokens, n_heads * vdim]")
+    _require_masked_pages(rows, value_pages, queries.dtype, n_kv_heads, dim, vdim)
+    _require(rows.data_ptr() % 16 == 0 and (value_pages is None or value_pages.data_ptr() % 16 == 0), "cache pages must start on 16-byte borders")
+    _require(page_rows.dtype == torch.int32 and page_rows.dim() == 2 and page_rows.is_contiguous(), "page rows must be int32 [sequences, stride]")
+    splits = max(1, min(int(splits), 64))
+    partial = torch.empty((tokens, n_heads, splits, vdim + 2), dtype=torch.float32, device=queries.device) if splits > 1 else None
+    library = build.load_library("masked_attention.cu")
+    _check(library.tau_talking_decode(
+        _code(queries), _pointer(queries), _pointer(rows), _pointer(value_pages), _pointer(talk), _pointer(out), ctypes.c_longlong(out.stride(0)), _pointer(step.positions),
+        _pointer(step.token_seq), _pointer(page_rows), ctypes.c_int(page_rows.shape[1]), ctypes.c_int(PAGE_TOKENS), ctypes.c_int(tokens), ctypes.c_int(n_heads),
+        ctypes.c_int(n_kv_heads), ctypes.c_int(dim), ctypes.c_int(vdim), ctypes.c_float(scale), ctypes.c_int(window), ctypes.c_int(keep_first), ctypes.c_float(out_scale),
+        ctypes.c_int(splits), _pointer(partial), _stream()), "talking_decode", 2 if splits > 1 else 1)
 
 
 def gated_rows(values, gate, out) -> None:
@@ -1407,15 +1516,31 @@ def channel_decay(values, offset) -> None:
     _check(library.tau_channel_decay(_pointer(values), _pointer(offset), ctypes.c_longlong(rows), ctypes.c_int(width), _stream()), "channel_decay")
 
 
-def wkv(r, k, v, w, bonus, state, cu_seqlens, seq_slot, out, n_heads: int, key_dim: int, value_dim: int) -> None:
-    """Per (sequence, head) over the sequence's new tokens: `o = (S + diag(bonus) k v^T)^T r`, then `S <- diag(w) S + k v^T`.
-    `r`, `k`, `w` float32 [tokens, n_heads * key_dim], `v` and `out` float32 [tokens, n_heads * value_dim], `bonus` float32
-    [n_heads, key_dim], `state` float32 [slots, n_heads * value_dim * key_dim], updated in place."""
-    _on_device(r, k, v, w, bonus, state, cu_seqlens, seq_slot, out)
+WALK_FORMS = {"bonus": 0, "forget_writes": 1, "constant_decay": 2}
+
+
+def wkv(r, k, v, w, per_head, state, cu_seqlens, seq_slot, out, n_heads: int, key_dim: int, value_dim: int, form: str = "bonus") -> None:
+    """The walk over a matrix state `S` (key_dim x value_dim) per (sequence, head), over the sequence's new tokens.  `form`:
+    `"bonus"`: `o = (S + diag(bonus) k v^T)^T r`, then `S <- diag(w) S + k v^T` (`per_head` float32 [n_heads, key_dim], the bonus);
+    `"forget_writes"`: `S <- diag(w) S + (1 - w) v^T`, then `o = S^T r` (no `k`, no `per_head`);
+    `"constant_decay"`: `S <- d S + k v^T`, then `o = S^T r` (no `w`; `per_head` float32 [n_heads], the decays).
+    `r`, `k`, `w` float32 [tokens, n_heads * key_dim] (rows one distance apart), `v` float32 [tokens, n_heads * value_dim] (rows any
+    distance apart), `out` the same and contiguous, `state` float32 [slots, n_heads * value_dim * key_dim], updated in place."""
+    _require(form in WALK_FORMS, f"unknown form {form!r}")
+    _on_device(r, k, v, w, per_head, state, cu_seqlens, seq_slot, out)
+    _require((k is not None) == (form != "forget_writes") and (w is not None) == (form != "constant_decay") and (per_head is not None) == (form != "forget_writes"),
+             "the form says which of k, w and per_head there are")
     tokens = r.shape[0]
     for tensor, width, what in ((r, key_dim, "r"), (k, key_dim, "k"), (w, key_dim, "w"), (v, value_dim, "v"), (out, value_dim, "the output")):
-        _require(tensor.dtype == torch.float32 and tensor.shape == (tokens, n_heads * width) and tensor.is_contiguous(), f"{what} must be contiguous float32 [tokens, heads * width]")
-    _require(bonus.dtype == torch.float32 and bonus.shape == (n_heads, key_dim) and bonus.is_contiguous(), "the bonus must be float32 [heads, key_dim]")
+        if tensor is not None:
+            _require(tensor.dtype == torch.float32 and tensor.shape == (tokens, n_heads * width) and tensor.stride(1) == 1, f"{what} must be float32 [tokens, heads * width]")
+    for tensor in (k, w):
+        _require(tensor is None or tensor.stride(0) == r.stride(0), "rows of r, k and w must lie equally far apart")
+    _require(out.is_contiguous(), "the output must be contiguous")
+    if form == "bonus":
+        _require(per_head.dtype == torch.float32 and per_head.shape == (n_heads, key_dim) and per_head.is_contiguous(), "the bonus must be float32 [heads, key_dim]")
+    elif form == "constant_decay":
+        _f32_vector(per_head, n_heads, "the decays")
     _require(state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and state.shape[1] == n_heads * value_dim * key_dim,
              f"the state must be float32 [slots, {n_heads * value_dim * key_dim}]")
     _require(1 <= key_dim <= WKV_MAX_KEY_DIM, f"key_dim must lie between 1 and {WKV_MAX_KEY_DIM}")
@@ -1424,8 +1549,38 @@ def wkv(r, k, v, w, bonus, state, cu_seqlens, seq_slot, out, n_heads: int, key_d
     n_seqs = seq_slot.numel()
     _require(cu_seqlens.numel() == n_seqs + 1, "one run per sequence")
     library = build.load_library("wkv.cu", (f"TAU_KEY_DIM={key_dim}",))
-    _check(library.tau_wkv(_pointer(r), _pointer(k), _pointer(v), _pointer(w), _pointer(bonus), _pointer(state), ctypes.c_longlong(state.stride(0)),
-                           _pointer(cu_seqlens), _pointer(seq_slot), _pointer(out), ctypes.c_int(n_seqs), ctypes.c_int(n_heads), ctypes.c_int(value_dim), _stream()), "wkv")
+    _check(library.tau_wkv(ctypes.c_int(WALK_FORMS[form]), _pointer(r), _pointer(k), _pointer(v), _pointer(w), ctypes.c_longlong(r.stride(0)), ctypes.c_longlong(v.stride(0)),
+                           _pointer(per_head), _pointer(state), ctypes.c_longlong(state.stride(0)), _pointer(cu_seqlens), _pointer(seq_slot), _pointer(out), ctypes.c_int(n_seqs),
+                           ctypes.c_int(n_heads), ctypes.c_int(value_dim), _stream()), "wkv")
+
+
+def forget_gates(rows, query_offset: int, gate_offset: int, lower) -> None:
+    """In place on float32 `rows` [tokens, width] (rows any distance apart): the columns from `query_offset` on pass SiLU, those from
+    `gate_offset` on become `l + (1 - l) sigmoid(x)` with `lower` float32 [count] the bounds l; `count` columns each."""
+    _on_device(rows, lower)
+    count = lower.numel()
+    _f32_vector(lower, count, "the lower bounds")
+    _require(rows.dtype == torch.float32 and rows.dim() == 2 and rows.stride(1) == 1 and query_offset + count <= rows.shape[1] and gate_offset + count <= rows.shape[1],
+             "rows must be float32 and hold the queries and the gates")
+    library = build.load_library("walk_prepare.cu")
+    _check(library.tau_forget_gates(_pointer(rows), ctypes.c_longlong(rows.stride(0)), ctypes.c_int(query_offset), ctypes.c_int(gate_offset), _pointer(lower),
+                                    ctypes.c_longlong(rows.shape[0]), ctypes.c_int(count), _stream()), "forget_gates")
+
+
+def turn_heads(rows, positions, frequency, rotary_dim: int, n_heads: int, dim: int, scaled_from: int, scale: float) -> None:
+    """In place on the first `n_heads * dim` columns of float32 `rows` (rows any distance apart): in every head element `i` of the first
+    `rotary_dim` is turned together with element `i + rotary_dim / 2` by `position * frequency[i]`; the heads from number `scaled_from`
+    on are multiplied by `scale`."""
+    _on_device(rows, positions, frequency)
+    _require(rows.dtype == torch.float32 and rows.dim() == 2 and rows.stride(1) == 1 and rows.shape[1] >= n_heads * dim, "rows must be float32 and hold the heads")
+    _require(rotary_dim % 2 == 0 and 0 <= rotary_dim <= dim, "rotary_dim must be even and at most dim")
+    if rotary_dim:
+        _f32_vector(frequency, rotary_dim // 2, "the rotation's frequencies")
+    _int_vector(positions, "positions")
+    library = build.load_library("walk_prepare.cu")
+    _check(library.tau_turn_heads(_pointer(rows), ctypes.c_longlong(rows.stride(0)), _pointer(positions), _pointer(frequency if rotary_dim else None), ctypes.c_int(rotary_dim),
+                                  ctypes.c_longlong(rows.shape[0]), ctypes.c_int(n_heads), ctypes.c_int(dim), ctypes.c_int(scaled_from), ctypes.c_float(scale), _stream()),
+           "turn_heads")
 
 
 # ---------------------------------------------------------------------------- routed experts

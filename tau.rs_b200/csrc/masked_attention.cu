@@ -3,7 +3,13 @@
 //   * key and value sizes may differ (`dim`, `vdim`); one cached row per position holds [kv_heads x key | kv_heads x value], or keys
 //     and values lie in pages of their own in the layout of ordinary heads, [pages, kv_heads, positions of a page, dim or vdim];
 //   * a query at position i sees key j <= i if j > i - window (`window` > 0), or if j lies in i's chunk, floor(j / chunk) ==
-//     floor(i / chunk) (`chunk` > 0; chunks are counted from position 0 of the sequence), or always (both 0);
+//     floor(i / chunk) (`chunk` > 0; chunks are counted from position 0 of the sequence), or always (both 0); the sequence's first
+//     `keep_first` positions stay visible however far back they lie;
+//   * `talk` ([heads, heads]): the scores of all heads are mixed before the softmax, score_h <- sum_g talk[h, g] score_g.  A score is linear
+//     in its query, so for runs of tokens prepare mixes the queries instead: head h asks every key head j with the query
+//     sum over the heads g of j's group of talk[h, g] q_g, one query of kv_heads * dim elements against the position's keys of all key
+//     heads side by side (`shared_keys`).  Single tokens take the kernel at the end of this file, which mixes the scores themselves;
+//   * prepare may mix the values with another layer's of the same token, v <- (1 - share) v + share first;
 //   * `sink`: the denominator of the softmax has exp(0) added (a key with score 0 and no value);
 //   * the result is multiplied by `out_scale` before its one rounding; output rows may lie any distance apart;
 //   * `distance` (two numbers r1, r2 per head): r1 * ln(1 + r2 * (i - j)) is taken off the score of key j for the query at i;
@@ -23,7 +29,23 @@
 namespace {
 
 constexpr int kWarps = 8;
+constexpr int kMaxShared = 200 * 1024;      // dynamic shared memory that a block of these kernels may ask for
 constexpr int kMaxOwned = 16;     // value columns per lane: vdim <= 512
+
+// The keys that a query sees, numbered 0 .. count - 1: the kept first positions that lie before its window (or chunk), then the window's.
+struct Visible {
+    int first, kept, count;
+    __device__ __forceinline__ int key(int number) const { return number < kept ? number : first + number - kept; }
+};
+__device__ __forceinline__ Visible visible_keys(int position, int window, int chunk, int keep_first) {
+    Visible seen;
+    seen.first = 0;
+    if (window > 0 && position - window + 1 > 0) seen.first = position - window + 1;
+    if (chunk > 0) seen.first = position / chunk * chunk;
+    seen.kept = keep_first < seen.first ? keep_first : seen.first;
+    seen.count = seen.kept + position - seen.first + 1;
+    return seen;
+}
 
 // grid: tokens; block kWarps * 32.  projected row: [heads * dim | kv_heads * dim | kv_heads * vdim] from its first column on.
 // Dynamic shared memory: rotary / 2 float2 (cosine, sine).
@@ -32,10 +54,11 @@ __global__ void __launch_bounds__(kWarps * 32)
 masked_prepare_kernel(const T* __restrict__ projected, long long projected_stride, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                       float eps, const float* __restrict__ frequency, int rotary, float magnitude, T* __restrict__ queries, T* __restrict__ rows,
                       T* __restrict__ value_pages, const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ page_rows, int page_stride,
-                      int page_tokens, int heads, int kv_heads, int dim, int vdim, int write_rows, float temperature_coef, int temperature_every) {
+                      int page_tokens, int heads, int kv_heads, int dim, int vdim, int write_rows, float temperature_coef, int temperature_every,
+                      const float* __restrict__ talk, const T* __restrict__ first_values, long long first_stride, const float* __restrict__ value_share) {
     grid_dependents_launch();
     grid_dependency_wait();
-    extern __shared__ float2 turns[];
+    extern __shared__ float2 turns[];       // then, with `talk`, heads * dim floats: the turned queries
     __shared__ float scratch[33];
     const int token = blockIdx.x;
     const int position = positions[token];
@@ -84,6 +107,7 @@ masked_prepare_kernel(const T* __restrict__ projected, long long projected_strid
     }
     // Items: within each head, the `half` rotated pairs, then the dim - rotary elements that pass.
     const int per_head = half + (dim - rotary);
+    float* turned = reinterpret_cast<float*>(turns + half);
     const int q_items = heads * per_head, items = q_items + (write_rows ? kv_heads * per_head : 0);
     for (int item = threadIdx.x; item < items; item += blockDim.x) {
         const bool is_query = item < q_items;
@@ -101,18 +125,44 @@ masked_prepare_kernel(const T* __restrict__ projected, long long projected_strid
                 w *= weight[head * dim + second];
             }
             const float2 turn = turns[within];
-            target[first] = from_float<T>(u * turn.x - w * turn.y);
-            target[second] = from_float<T>(w * turn.x + u * turn.y);
+            const float a = u * turn.x - w * turn.y, b = w * turn.x + u * turn.y;
+            if (talk && is_query) {
+                turned[head * dim + first] = a;
+                turned[head * dim + second] = b;
+            } else {
+                target[first] = from_float<T>(a);
+                target[second] = from_float<T>(b);
+            }
         } else {
             const int column = rotary + (within - half);
             float u = to_float(from[column]) * inverse;
             if (weight) u *= weight[head * dim + column];
-            target[column] = from_float<T>(u);
+            if (talk && is_query) turned[head * dim + column] = u;
+            else target[column] = from_float<T>(u);
         }
     }
     if (write_rows) {
         const T* values = source + q_width + k_width;
-        for (int column = threadIdx.x; column < kv_heads * vdim; column += blockDim.x) value_row[(column / vdim) * value_head_stride + column % vdim] = values[column];
+        const T* first = first_values ? first_values + static_cast<size_t>(token) * first_stride : nullptr;
+        const float share = first ? *value_share : 0.0f;
+        for (int column = threadIdx.x; column < kv_heads * vdim; column += blockDim.x) {
+            T value = values[column];
+            if (first) value = from_float<T>((1.0f - share) * to_float(value) + share * to_float(first[column]));
+            value_row[(column / vdim) * value_head_stride + column % vdim] = value;
+        }
+    }
+    if (talk) {      // head h's query for key head j: the queries of j's group, weighed by row h of `talk`; rounded once
+        __syncthreads();
+        const int group_size = heads / kv_heads, wide = kv_heads * dim;
+        T* mixed = queries + static_cast<size_t>(token) * heads * wide;
+        for (int index = threadIdx.x; index < heads * wide; index += blockDim.x) {
+            const int head = index / wide, within = index % wide, group = within / dim, column = within % dim;
+            const float* from = turned + group * group_size * dim + column;
+            const float* weight = talk + head * heads + group * group_size;
+            float sum = 0.0f;
+            for (int g = 0; g < group_size; ++g) sum = fmaf(weight[g], from[g * dim], sum);
+            mixed[index] = from_float<T>(sum);
+        }
     }
 }
 
@@ -123,16 +173,18 @@ masked_attention_kernel(const T* __restrict__ queries, const T* __restrict__ row
                         const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ page_rows, int page_stride,
                         int page_tokens, int heads, int kv_heads, int dim, int vdim, float scale, int window, int chunk, int sink, float out_scale,
                         const float* __restrict__ distance, int sigmoid_weights, const float* __restrict__ head_offset, const T* __restrict__ gate,
-                        long long gate_stride, int gate_per_head) {
+                        long long gate_stride, int gate_per_head, int keep_first, int shared_keys) {
     grid_dependents_launch();
     grid_dependency_wait();
     extern __shared__ float shared[];
     const int token = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int head = blockIdx.y * kWarps + warp;
     if (head >= heads) return;
-    float* query = shared + static_cast<size_t>(warp) * dim;
-    const T* q_source = queries + (static_cast<size_t>(token) * heads + head) * dim;
-    for (int column = lane; column < dim; column += 32) query[column] = to_float(q_source[column]) * scale;
+    // With `shared_keys` a query is `segments` pieces of `dim` elements, one for each key head of the position.
+    const int segments = shared_keys ? kv_heads : 1, query_width = segments * dim;
+    float* query = shared + static_cast<size_t>(warp) * query_width;
+    const T* q_source = queries + (static_cast<size_t>(token) * heads + head) * query_width;
+    for (int column = lane; column < query_width; column += 32) query[column] = to_float(q_source[column]) * scale;
     __syncwarp();
     const int position = positions[token];
     const int* pages = page_rows + static_cast<size_t>(token_seq[token]) * page_stride;
@@ -141,25 +193,25 @@ masked_attention_kernel(const T* __restrict__ queries, const T* __restrict__ row
     const T* keys;
     const T* values;
     long long key_page, key_row, value_page, value_row;
+    const int key_group = shared_keys ? 0 : group;
+    const long long key_segment = value_pages ? static_cast<long long>(page_tokens) * dim : dim;      // from one key head's key to the next one's
     if (value_pages) {      // [pages, kv_heads, page_tokens, dim or vdim]
         key_row = dim, value_row = vdim, key_page = static_cast<long long>(kv_heads) * page_tokens * dim, value_page = static_cast<long long>(kv_heads) * page_tokens * vdim;
-        keys = rows + static_cast<long long>(group) * page_tokens * dim, values = value_pages + static_cast<long long>(group) * page_tokens * vdim;
+        keys = rows + static_cast<long long>(key_group) * page_tokens * dim, values = value_pages + static_cast<long long>(group) * page_tokens * vdim;
     } else {                // [pages, page_tokens, keys of all heads | values of all heads]
         key_row = value_row = kv_heads * (dim + vdim), key_page = value_page = key_row * page_tokens;
-        keys = rows + group * dim, values = rows + kv_heads * dim + group * vdim;
+        keys = rows + key_group * dim, values = rows + kv_heads * dim + group * vdim;
     }
-    int first_key = 0;
-    if (window > 0 && position - window + 1 > 0) first_key = position - window + 1;
-    if (chunk > 0) first_key = position / chunk * chunk;
+    const Visible seen = visible_keys(position, window, chunk, keep_first);
     float top = sink ? 0.0f : -INFINITY, sum = sink ? 1.0f : 0.0f;       // the sink: a weight of exp(0 - top) that carries no value
     const float far = distance ? distance[2 * head] : 0.0f, reach = distance ? distance[2 * head + 1] : 0.0f;
     const float offset = head_offset ? head_offset[head] : 0.0f;
     float acc[kMaxOwned];
 #pragma unroll
     for (int i = 0; i < kMaxOwned; ++i) acc[i] = 0.0f;
-    for (int base = first_key; base <= position; base += 32) {
-        const int key = base + lane;
-        const bool valid = key <= position;
+    for (int base = 0; base < seen.count; base += 32) {
+        const bool valid = base + lane < seen.count;
+        const int key = seen.key(base + lane);
         long long value_index = 0;
         float score = -INFINITY;
         if (valid) {
@@ -167,12 +219,15 @@ masked_attention_kernel(const T* __restrict__ queries, const T* __restrict__ row
             value_index = page * value_page + within_page * value_row;
             const T* k = keys + page * key_page + within_page * key_row;
             float a = 0.0f, b = 0.0f;
-            int column = 0;
-            for (; column + 1 < dim; column += 2) {
-                a = fmaf(query[column], to_float(k[column]), a);
-                b = fmaf(query[column + 1], to_float(k[column + 1]), b);
+            for (int segment = 0; segment < segments; ++segment, k += key_segment) {
+                const float* part = query + segment * dim;
+                int column = 0;
+                for (; column + 1 < dim; column += 2) {
+                    a = fmaf(part[column], to_float(k[column]), a);
+                    b = fmaf(part[column + 1], to_float(k[column + 1]), b);
+                }
+                if (column < dim) a = fmaf(part[column], to_float(k[column]), a);
             }
-            if (column < dim) a = fmaf(query[column], to_float(k[column]), a);
             score = a + b;
             if (distance) score -= far * log1pf(reach * static_cast<float>(position - key));
         }
@@ -188,7 +243,7 @@ masked_attention_kernel(const T* __restrict__ queries, const T* __restrict__ row
 #pragma unroll
             for (int i = 0; i < kMaxOwned; ++i) acc[i] *= keep;
         }
-        const int count = position - base + 1 < 32 ? position - base + 1 : 32;
+        const int count = seen.count - base < 32 ? seen.count - base : 32;
         for (int j = 0; j < count; ++j) {
             const float w = __shfl_sync(0xffffffffu, p, j);
             const T* v = values + __shfl_sync(0xffffffffu, value_index, j);
@@ -251,7 +306,7 @@ masked_attention_staged_kernel(const T* __restrict__ queries, const T* __restric
                                long long out_stride, const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ page_rows,
                                int page_stride, int page_tokens, int heads, int kv_heads, int dim, int vdim, float scale, int window, int chunk, int sink,
                                float out_scale, const float* __restrict__ distance, int sigmoid_weights, const float* __restrict__ head_offset,
-                               const T* __restrict__ gate, long long gate_stride, int gate_per_head, int splits, float* __restrict__ partial) {
+                               const T* __restrict__ gate, long long gate_stride, int gate_per_head, int splits, float* __restrict__ partial, int keep_first) {
     grid_dependents_launch();
     grid_dependency_wait();
     constexpr int kPer = Word<T>::kElements;
@@ -276,23 +331,21 @@ masked_attention_staged_kernel(const T* __restrict__ queries, const T* __restric
         key_row = value_row = kv_heads * (dim + vdim), key_page = value_page = key_row * page_tokens;
         keys = rows + group * dim, values = rows + kv_heads * dim + group * vdim;
     }
-    int first_key = 0;
-    if (window > 0 && position - window + 1 > 0) first_key = position - window + 1;
-    if (chunk > 0) first_key = position / chunk * chunk;
-    const int all_tiles = (position - first_key) / kTileKeys + 1;
+    const Visible seen = visible_keys(position, window, chunk, keep_first);
+    const int all_tiles = (seen.count - 1) / kTileKeys + 1;
     // This block's range of the token's tiles (all of them without splits); tiles are numbered from the range's first.
     const int per_split = (all_tiles + splits - 1) / splits, tile_begin = static_cast<int>(blockIdx.z) * per_split;
     const int n_tiles = all_tiles - tile_begin < per_split ? (all_tiles - tile_begin > 0 ? all_tiles - tile_begin : 0) : per_split;
-    first_key += tile_begin * kTileKeys;
+    const int first_number = tile_begin * kTileKeys;      // of the range's first tile, among the keys that the token sees
 
     auto stage = [&](int tile) {
         uint32_t* buffer = staged_words + (tile & 1) * tile_words;
         if (tile < n_tiles) {
-            const int base = first_key + tile * kTileKeys;
-            const int count = position - base + 1 < kTileKeys ? position - base + 1 : kTileKeys;
+            const int base = first_number + tile * kTileKeys;
+            const int count = seen.count - base < kTileKeys ? seen.count - base : kTileKeys;
             uint32_t* value_buffer = buffer + kTileKeys * key_stride;
             for (int row = warp; row < count; row += kStagedWarps) {      // a warp per row: one page lookup, then whole lines
-                const int key = base + row;
+                const int key = seen.key(base + row);
                 const long long page = pages[key / page_tokens], within_page = key % page_tokens;
                 const uint32_t* key_source = reinterpret_cast<const uint32_t*>(keys + page * key_page + within_page * key_row);
                 const uint32_t* value_source = reinterpret_cast<const uint32_t*>(values + page * value_page + within_page * value_row);
@@ -319,8 +372,8 @@ masked_attention_staged_kernel(const T* __restrict__ queries, const T* __restric
         copy_wait<1>();      // this thread's copies of `tile` are done (those of the next tile may be on their way)
         __syncthreads();     // everybody's are; the queries too
         const uint32_t* buffer = staged_words + (tile & 1) * tile_words;
-        const int base = first_key + tile * kTileKeys;
-        const int count = position - base + 1 < kTileKeys ? position - base + 1 : kTileKeys;
+        const int base = first_number + tile * kTileKeys;
+        const int count = seen.count - base < kTileKeys ? seen.count - base : kTileKeys;
         if (has_head) {
             float score = -INFINITY;
             if (lane < count) {
@@ -332,7 +385,7 @@ masked_attention_staged_kernel(const T* __restrict__ queries, const T* __restric
                     if (kPer == 2) b = fmaf(query[word * kPer + 1], Word<T>::second(both), b);
                 }
                 score = a + b;
-                if (distance) score -= far * log1pf(reach * static_cast<float>(position - (base + lane)));
+                if (distance) score -= far * log1pf(reach * static_cast<float>(position - seen.key(base + lane)));
             }
             float p;
             if (sigmoid_weights) {
@@ -426,6 +479,240 @@ masked_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__
     }
 }
 
+// ---- single tokens with mixed scores ---------------------------------------------------------------------------------------------
+//
+// grid: (tokens, splits); block: kTalkWarps warps that serve all heads of a token together, since every head's weights need every head's
+// scores.  Tiles of 32 positions, keys and values of all key/value heads, come into shared memory by cp.async, 16 bytes at a time (one or
+// two tiles deep, as they fit); key rows are an odd number of 16-byte units apart.  Then, for each tile:
+//   scores    lane = key; a warp takes two heads of one key head at a time, so that a key's elements are read once for both;
+//   mixing    lane = key; a warp takes a head: sum over all heads of talk[h, g] * score_g, running maximum, weights and sum;
+//   values    a thread owns 16 bytes' worth of a head's columns (kOwned such places) and adds the tile's weighted values to them.
+// Scores, mixing, weights and sums in 32-bit.  `splits` > 1: ranges joined by `masked_attention_merge_kernel`, as above.
+constexpr int kTalkWarps = 8;
+constexpr int kScoreStride = kTileKeys + 1;
+
+__device__ __forceinline__ void copy_16(void* target, const void* source) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(target))), "l"(source) : "memory");
+}
+
+// The elements of 16 bytes as floats.
+__device__ __forceinline__ void unpack_16(uint4 raw, float (&v)[8], bf16) {
+    const uint32_t words[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) v[2 * i] = __uint_as_float(words[i] << 16), v[2 * i + 1] = __uint_as_float(words[i] & 0xffff0000u);
+}
+__device__ __forceinline__ void unpack_16(uint4 raw, float (&v)[4], float) {
+    v[0] = __uint_as_float(raw.x), v[1] = __uint_as_float(raw.y), v[2] = __uint_as_float(raw.z), v[3] = __uint_as_float(raw.w);
+}
+
+// Shared memory by section, in bytes.
+struct TalkPlan {
+    int key_stride, value_stride, tile, stages, total;      // of a staged row of keys and of values, of one tile, tiles in flight, all together
+};
+template <typename T>
+__host__ __device__ inline TalkPlan talk_plan(int heads, int kv_heads, int dim, int vdim) {
+    TalkPlan plan = {0, 0, 0, 0, 0};
+    constexpr int kPer = 16 / static_cast<int>(sizeof(T));
+    if (dim % kPer != 0 || vdim % kPer != 0) return plan;
+    plan.key_stride = ((kv_heads * dim / kPer) | 1) * 16;
+    plan.value_stride = kv_heads * vdim / kPer * 16;
+    const long long tile = static_cast<long long>(kTileKeys) * (plan.key_stride + plan.value_stride);
+    const long long fixed = 4LL * (static_cast<long long>(heads) * dim + heads * heads + 2LL * heads * kScoreStride + 3LL * heads);
+    if (tile + fixed > kMaxShared) return plan;
+    plan.tile = static_cast<int>(tile);
+    plan.stages = 2 * tile + fixed <= kMaxShared ? 2 : 1;
+    plan.total = static_cast<int>(plan.stages * tile + fixed);
+    return plan;
+}
+
+template <typename T, int kOwned>
+__global__ void __launch_bounds__(kTalkWarps * 32)
+talking_decode_kernel(const T* __restrict__ queries, const T* __restrict__ rows, const T* __restrict__ value_pages, const float* __restrict__ talk,
+                      T* __restrict__ out, long long out_stride, const int* __restrict__ positions, const int* __restrict__ token_seq,
+                      const int* __restrict__ page_rows, int page_stride, int page_tokens, int heads, int kv_heads, int dim, int vdim, float scale, int window,
+                      int keep_first, float out_scale, int splits, float* __restrict__ partial) {
+    grid_dependents_launch();
+    constexpr int kPer = 16 / static_cast<int>(sizeof(T)), kThreads = kTalkWarps * 32;
+    extern __shared__ __align__(16) uint8_t talk_shared[];
+    const TalkPlan plan = talk_plan<T>(heads, kv_heads, dim, vdim);
+    float* query = reinterpret_cast<float*>(talk_shared + plan.stages * plan.tile);      // [heads][dim], scaled
+    float* mixing = query + heads * dim;                                                  // [heads][heads]
+    float* scores = mixing + heads * heads;                                               // [heads][kScoreStride]
+    float* weights = scores + heads * kScoreStride;                                       // the same
+    float* tops = weights + heads * kScoreStride;                                         // [heads] running maxima, sums, and the last rescaling
+    float* sums = tops + heads;
+    float* rescale = sums + heads;
+    const int token = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int index = threadIdx.x; index < heads * heads; index += kThreads) mixing[index] = talk[index];      // a weight: no earlier kernel writes it
+    for (int head = threadIdx.x; head < heads; head += kThreads) tops[head] = -INFINITY, sums[head] = 0.0f;
+    grid_dependency_wait();
+    const int position = positions[token];
+    const int* pages = page_rows + static_cast<size_t>(token_seq[token]) * page_stride;
+    const Visible seen = visible_keys(position, window, 0, keep_first);
+    const int all_tiles = (seen.count - 1) / kTileKeys + 1;
+    const int per_split = (all_tiles + splits - 1) / splits, tile_begin = static_cast<int>(blockIdx.y) * per_split;
+    const int n_tiles = all_tiles - tile_begin < per_split ? (all_tiles - tile_begin > 0 ? all_tiles - tile_begin : 0) : per_split;
+    const int first_number = tile_begin * kTileKeys;
+    const int key_pieces = dim / kPer, value_pieces = vdim / kPer;      // 16-byte pieces of one head's key and value
+    const int row_pieces = kv_heads * (key_pieces + value_pieces);
+    auto stage = [&](int tile) {
+        if (tile < n_tiles) {
+            uint8_t* buffer = talk_shared + (plan.stages == 2 ? (tile & 1) * plan.tile : 0);
+            const int base = first_number + tile * kTileKeys;
+            const int count = seen.count - base < kTileKeys ? seen.count - base : kTileKeys;
+            for (int row = warp; row < count; row += kTalkWarps) {      // a warp per row: one page lookup, then whole lines
+                const int key = seen.key(base + row);
+                const long long page = pages[key / page_tokens], within = key % page_tokens;
+                uint8_t* key_target = buffer + row * plan.key_stride;
+                uint8_t* value_target = buffer + kTileKeys * plan.key_stride + row * plan.value_stride;
+                for (int piece = lane; piece < row_pieces; piece += 32) {
+                    const bool is_key = piece < kv_heads * key_pieces;
+                    const int index = is_key ? piece : piece - kv_heads * key_pieces;
+                    const T* source;
+                    if (value_pages) {
+                        const int per = is_key ? key_pieces : value_pieces, head = index / per;
+                        source = (is_key ? rows : value_pages) + ((page * kv_heads + head) * page_tokens + within) * (is_key ? dim : vdim) + (index - head * per) * kPer;
+                    } else {
+                        source = rows + (page * page_tokens + within) * (static_cast<long long>(kv_heads) * (dim + vdim)) + piece * kPer;
+                    }
+                    copy_16((is_key ? key_target : value_target) + index * 16, source);
+                }
+            }
+        }
+        copy_commit();
+    };
+    stage(0);
+    if (plan.stages == 2) stage(1);
+    for (int index = threadIdx.x; index < heads * dim; index += kThreads) query[index] = to_float(queries[static_cast<size_t>(token) * heads * dim + index]) * scale;
+    float acc[kOwned][kPer];
+#pragma unroll
+    for (int i = 0; i < kOwned; ++i)
+#pragma unroll
+        for (int e = 0; e < kPer; ++e) acc[i][e] = 0.0f;
+    const int group_size = heads / kv_heads, pairs = (group_size + 1) / 2;
+    for (int tile = 0; tile < n_tiles; ++tile) {
+        if (plan.stages == 2) copy_wait<1>();
+        else copy_wait<0>();
+        __syncthreads();     // the tile has arrived for everybody; the queries and the mixing weights are there
+        const uint8_t* buffer = talk_shared + (plan.stages == 2 ? (tile & 1) * plan.tile : 0);
+        const int base = first_number + tile * kTileKeys;
+        const int count = seen.count - base < kTileKeys ? seen.count - base : kTileKeys;
+        for (int item = warp; item < kv_heads * pairs; item += kTalkWarps) {
+            const int group = item / pairs, in_group = item % pairs * 2, head = group * group_size + in_group;
+            const bool second = in_group + 1 < group_size;
+            if (lane < count) {
+                const uint4* k = reinterpret_cast<const uint4*>(buffer + lane * plan.key_stride) + group * key_pieces;
+                const float* q0 = query + head * dim;
+                const float* q1 = second ? q0 + dim : q0;
+                float a[2] = {0.0f, 0.0f}, b[2] = {0.0f, 0.0f};
+                for (int piece = 0; piece < key_pieces; ++piece) {
+                    float v[kPer];
+                    unpack_16(k[piece], v, T());
+#pragma unroll
+                    for (int e = 0; e < kPer; e += 4) {
+                        const float4 x = *reinterpret_cast<const float4*>(q0 + piece * kPer + e), y = *reinterpret_cast<const float4*>(q1 + piece * kPer + e);
+                        a[0] = fmaf(x.x, v[e], a[0]), a[1] = fmaf(x.y, v[e + 1], a[1]), a[0] = fmaf(x.z, v[e + 2], a[0]), a[1] = fmaf(x.w, v[e + 3], a[1]);
+                        b[0] = fmaf(y.x, v[e], b[0]), b[1] = fmaf(y.y, v[e + 1], b[1]), b[0] = fmaf(y.z, v[e + 2], b[0]), b[1] = fmaf(y.w, v[e + 3], b[1]);
+                    }
+                }
+                scores[head * kScoreStride + lane] = a[0] + a[1];
+                if (second) scores[(head + 1) * kScoreStride + lane] = b[0] + b[1];
+            }
+        }
+        __syncthreads();
+        for (int head = warp; head < heads; head += kTalkWarps) {
+            float mixed = -INFINITY;
+            if (lane < count) {
+                float sum[2] = {0.0f, 0.0f};
+                for (int g = 0; g < heads; ++g) sum[g & 1] = fmaf(mixing[head * heads + g], scores[g * kScoreStride + lane], sum[g & 1]);
+                mixed = sum[0] + sum[1];
+            }
+            const float top = tops[head], new_top = fmaxf(top, warp_max(mixed));
+            const float p = lane < count ? expf(mixed - new_top) : 0.0f, total = warp_sum(p);
+            weights[head * kScoreStride + lane] = p;
+            __syncwarp();      // every lane has read the maximum
+            if (lane == 0) {
+                const float keep = expf(top - new_top);      // exp(-inf) = 0 the first time
+                tops[head] = new_top, sums[head] = sums[head] * keep + total, rescale[head] = keep;
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < kOwned; ++i) {
+            const int place = threadIdx.x + i * kThreads;
+            if (place < heads * value_pieces) {
+                const int head = place / value_pieces, piece = place % value_pieces;
+                const float keep = rescale[head];
+#pragma unroll
+                for (int e = 0; e < kPer; ++e) acc[i][e] *= keep;
+                const uint8_t* v = buffer + kTileKeys * plan.key_stride + (head / group_size * value_pieces + piece) * 16;
+                const float* weight = weights + head * kScoreStride;
+                for (int j = 0; j < count; ++j) {
+                    float value[kPer];
+                    unpack_16(*reinterpret_cast<const uint4*>(v + j * plan.value_stride), value, T());
+                    const float w = weight[j];
+#pragma unroll
+                    for (int e = 0; e < kPer; ++e) acc[i][e] = fmaf(w, value[e], acc[i][e]);
+                }
+            }
+        }
+        __syncthreads();     // the tile's place may be written over
+        stage(tile + plan.stages);
+    }
+    copy_wait<0>();
+#pragma unroll
+    for (int i = 0; i < kOwned; ++i) {
+        const int place = threadIdx.x + i * kThreads;
+        if (place >= heads * value_pieces) continue;
+        const int head = place / value_pieces, piece = place % value_pieces;
+        if (partial) {
+            float* record = partial + ((static_cast<size_t>(token) * heads + head) * splits + blockIdx.y) * (vdim + 2);
+#pragma unroll
+            for (int e = 0; e < kPer; ++e) record[piece * kPer + e] = acc[i][e];
+            if (piece == 0) record[vdim] = tops[head], record[vdim + 1] = sums[head];
+        } else {
+            const float factor = out_scale / sums[head];
+            T* target = out + static_cast<size_t>(token) * out_stride + head * vdim + piece * kPer;
+#pragma unroll
+            for (int e = 0; e < kPer; ++e) target[e] = from_float<T>(acc[i][e] * factor);
+        }
+    }
+}
+
+template <typename T>
+bool talk_fits(int heads, int kv_heads, int dim, int vdim) {
+    return heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0 && static_cast<long long>(heads) * vdim * sizeof(T) <= 4LL * 16 * kTalkWarps * 32 &&
+           talk_plan<T>(heads, kv_heads, dim, vdim).total > 0;
+}
+
+template <typename T>
+int launch_talking_decode(const void* queries, const void* rows, const void* value_pages, const float* talk, void* out, long long out_stride, const int* positions,
+                          const int* token_seq, const int* page_rows, int page_stride, int page_tokens, int tokens, int heads, int kv_heads, int dim, int vdim,
+                          float scale, int window, int keep_first, float out_scale, int splits, float* partial, cudaStream_t s) {
+    if (!talk_fits<T>(heads, kv_heads, dim, vdim)) return cudaErrorInvalidValue;
+    const TalkPlan plan = talk_plan<T>(heads, kv_heads, dim, vdim);
+    const int places = heads * vdim * static_cast<int>(sizeof(T)) / 16, owned = (places + kTalkWarps * 32 - 1) / (kTalkWarps * 32);
+    if (splits > 1 && !partial) return cudaErrorInvalidValue;
+    if (splits <= 1) splits = 1, partial = nullptr;
+#define TAU_TALK(OWNED)                                                                                                                                          \
+    {                                                                                                                                                            \
+        const cudaError_t status = cudaFuncSetAttribute(talking_decode_kernel<T, OWNED>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxShared);                \
+        if (status != cudaSuccess) return static_cast<int>(status);                                                                                              \
+        tau_launch(talking_decode_kernel<T, OWNED>, dim3(tokens, splits), dim3(kTalkWarps * 32), plan.total, s, static_cast<const T*>(queries),                   \
+                   static_cast<const T*>(rows), static_cast<const T*>(value_pages), talk, static_cast<T*>(out), out_stride, positions, token_seq, page_rows,       \
+                   page_stride, page_tokens, heads, kv_heads, dim, vdim, scale, window, keep_first, out_scale, splits, partial);                                  \
+    }
+    if (owned <= 1) TAU_TALK(1)
+    else if (owned <= 2) TAU_TALK(2)
+    else TAU_TALK(4)
+#undef TAU_TALK
+    const int status = tau_launch_status();
+    if (status != 0 || !partial) return status;
+    tau_launch(masked_attention_merge_kernel<T>, dim3(tokens, heads), dim3(128), 0, s, partial, static_cast<T*>(out), out_stride, heads, vdim, splits, out_scale, 0,
+               static_cast<const T*>(nullptr), 0LL, 0);
+    return tau_launch_status();
+}
+
 // Shared memory of the staged kernel, or 0 where it does not serve these sizes.
 template <typename T>
 int staged_bytes(int dim, int vdim) {
@@ -439,7 +726,7 @@ template <typename T>
 int launch_staged(int bytes, const void* queries, const void* rows, const void* value_pages, void* out, long long out_stride, const int* positions,
                   const int* token_seq, const int* page_rows, int page_stride, int page_tokens, int tokens, int heads, int kv_heads, int dim, int vdim,
                   float scale, int window, int chunk, int sink, float out_scale, const float* distance, int sigmoid_weights, const float* head_offset,
-                  const void* gate, long long gate_stride, int gate_per_head, int splits, float* partial, cudaStream_t s) {
+                  const void* gate, long long gate_stride, int gate_per_head, int splits, float* partial, int keep_first, cudaStream_t s) {
     static int allowed = 48 * 1024;
     if (bytes > allowed) {
         cudaError_t status = cudaFuncSetAttribute(masked_attention_staged_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
@@ -452,7 +739,7 @@ int launch_staged(int bytes, const void* queries, const void* rows, const void* 
     tau_launch(masked_attention_staged_kernel<T>, dim3(tokens, kv_heads * passes, splits), dim3(kStagedWarps * 32), bytes, s, static_cast<const T*>(queries),
                static_cast<const T*>(rows), static_cast<const T*>(value_pages), static_cast<T*>(out), out_stride, positions, token_seq, page_rows, page_stride,
                page_tokens, heads, kv_heads, dim, vdim, scale, window, chunk, sink, out_scale, distance, sigmoid_weights, head_offset,
-               static_cast<const T*>(gate), gate_stride, gate_per_head, splits, partial);
+               static_cast<const T*>(gate), gate_stride, gate_per_head, splits, partial, keep_first);
     int status = tau_launch_status();
     if (status != 0 || !partial) return status;
     tau_launch(masked_attention_merge_kernel<T>, dim3(tokens, heads), dim3(128), 0, s, partial, static_cast<T*>(out), out_stride, heads, vdim, splits, out_scale,
@@ -474,6 +761,27 @@ sigmoid_gate_kernel(const T* __restrict__ values, long long values_stride, const
 
 }  // namespace
 
+// 1 where `tau_talking_decode` serves these sizes.
+TAU_EXPORT int tau_talking_decode_fits(int dtype, int heads, int kv_heads, int dim, int vdim) {
+    return dtype == TAU_F32 ? talk_fits<float>(heads, kv_heads, dim, vdim) : dtype == TAU_BF16 ? talk_fits<bf16>(heads, kv_heads, dim, vdim) : 0;
+}
+
+// Single tokens: queries [tokens, heads, dim] as prepare leaves them without `talk`; the cache in either layout (see tau_masked_attention).
+TAU_EXPORT int tau_talking_decode(int dtype, const void* queries, const void* rows, const void* value_pages, const float* talk, void* out, long long out_stride,
+                                  const int* positions, const int* token_seq, const int* page_rows, int page_stride, int page_tokens, int tokens, int heads,
+                                  int kv_heads, int dim, int vdim, float scale, int window, int keep_first, float out_scale, int splits, float* partial, void* stream) {
+    if (tokens <= 0) return 0;
+    if (!queries || !rows || !talk || !out || !positions || !token_seq || !page_rows || window < 0 || keep_first < 0 || page_tokens <= 0) return cudaErrorInvalidValue;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (dtype == TAU_F32)
+        return launch_talking_decode<float>(queries, rows, value_pages, talk, out, out_stride, positions, token_seq, page_rows, page_stride, page_tokens, tokens, heads,
+                                            kv_heads, dim, vdim, scale, window, keep_first, out_scale, splits, partial, s);
+    if (dtype == TAU_BF16)
+        return launch_talking_decode<bf16>(queries, rows, value_pages, talk, out, out_stride, positions, token_seq, page_rows, page_stride, page_tokens, tokens, heads,
+                                           kv_heads, dim, vdim, scale, window, keep_first, out_scale, splits, partial, s);
+    return cudaErrorInvalidValue;
+}
+
 TAU_EXPORT int tau_sigmoid_gate(int dtype, const void* values, long long values_stride, const void* gate, long long gate_stride, void* out, long long out_stride,
                                 int rows, int width, void* stream) {
     if (rows <= 0) return 0;
@@ -492,20 +800,25 @@ TAU_EXPORT int tau_sigmoid_gate(int dtype, const void* values, long long values_
 TAU_EXPORT int tau_masked_prepare(int dtype, const void* projected, long long projected_stride, const float* q_weight, const float* k_weight, float eps,
                                   const float* frequency, int rotary, float magnitude, void* queries, void* rows, void* value_pages, const int* positions,
                                   const int* token_seq, const int* page_rows, int page_stride, int page_tokens, int tokens, int heads, int kv_heads, int dim, int vdim,
-                                  int write_rows, float temperature_coef, int temperature_every, void* stream) {
+                                  int write_rows, float temperature_coef, int temperature_every, const float* talk, const void* first_values,
+                                  long long first_stride, const float* value_share, void* stream) {
     if (tokens <= 0) return 0;
     if (!projected || !queries || !positions || heads <= 0 || kv_heads <= 0 || dim <= 0 || vdim <= 0 || rotary < 0 || rotary > dim || rotary % 2 != 0 ||
-        (rotary && !frequency) || (write_rows && (!rows || !token_seq || !page_rows)))
+        (rotary && !frequency) || (write_rows && (!rows || !token_seq || !page_rows)) || (talk && heads % kv_heads != 0) || (first_values && !value_share))
         return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    const size_t bytes = static_cast<size_t>(rotary / 2) * sizeof(float2);
-    if (bytes > 40 * 1024) return cudaErrorInvalidValue;
+    const size_t bytes = static_cast<size_t>(rotary / 2) * sizeof(float2) + (talk ? static_cast<size_t>(heads) * dim * sizeof(float) : 0);
+    if (bytes > kMaxShared) return cudaErrorInvalidValue;
 #define TAU_PREPARE(T)                                                                                                                            \
+    if (bytes > 40 * 1024) {                                                                                                                      \
+        const cudaError_t status = cudaFuncSetAttribute(masked_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxShared);        \
+        if (status != cudaSuccess) return static_cast<int>(status);                                                                               \
+    }                                                                                                                                             \
     tau_launch(masked_prepare_kernel<T>, dim3(tokens), dim3(kWarps * 32), bytes, s, static_cast<const T*>(projected), projected_stride, q_weight, k_weight, eps, \
                frequency, rotary, magnitude, static_cast<T*>(queries), static_cast<T*>(rows), static_cast<T*>(value_pages), positions, token_seq, page_rows, page_stride, page_tokens, heads,   \
-               kv_heads, dim, vdim, write_rows, temperature_coef, temperature_every)
-    if (dtype == TAU_F32) TAU_PREPARE(float);
-    else if (dtype == TAU_BF16) TAU_PREPARE(bf16);
+               kv_heads, dim, vdim, write_rows, temperature_coef, temperature_every, talk, static_cast<const T*>(first_values), first_stride, value_share)
+    if (dtype == TAU_F32) { TAU_PREPARE(float); }
+    else if (dtype == TAU_BF16) { TAU_PREPARE(bf16); }
     else return cudaErrorInvalidValue;
 #undef TAU_PREPARE
     return tau_launch_status();
@@ -517,34 +830,38 @@ TAU_EXPORT int tau_masked_attention(int dtype, const void* queries, const void* 
                                     const int* token_seq, const int* page_rows, int page_stride, int page_tokens, int tokens, int heads, int kv_heads,
                                     int dim, int vdim, float scale, int window, int chunk, int sink, float out_scale, int staged, const float* distance,
                                     int sigmoid_weights, const float* head_offset, const void* gate, long long gate_stride, int gate_per_head, int splits,
-                                    float* partial, void* stream) {
+                                    float* partial, int keep_first, int shared_keys, void* stream) {
     if (tokens <= 0) return 0;
     if (!queries || !rows || !out || !positions || !token_seq || !page_rows || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || dim <= 0 ||
-        vdim <= 0 || vdim > 32 * kMaxOwned || window < 0 || chunk < 0 || (window > 0 && chunk > 0) || (sigmoid_weights && sink))
+        vdim <= 0 || vdim > 32 * kMaxOwned || window < 0 || chunk < 0 || (window > 0 && chunk > 0) || (sigmoid_weights && sink) || keep_first < 0)
         return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     // `staged` (steps of single tokens): the kernel that shares tiles of the cache among a group's heads, where the sizes allow it.
-    if (staged && (dtype == TAU_F32 || dtype == TAU_BF16)) {
+    if (staged && !shared_keys && (dtype == TAU_F32 || dtype == TAU_BF16)) {
         const int staged_size = dtype == TAU_F32 ? staged_bytes<float>(dim, vdim) : staged_bytes<bf16>(dim, vdim);
         if (staged_size > 0) {
             if (dtype == TAU_F32)
                 return launch_staged<float>(staged_size, queries, rows, value_pages, out, out_stride, positions, token_seq, page_rows, page_stride, page_tokens,
                                             tokens, heads, kv_heads, dim, vdim, scale, window, chunk, sink, out_scale, distance, sigmoid_weights, head_offset, gate, gate_stride,
-                                            gate_per_head, splits, partial, s);
+                                            gate_per_head, splits, partial, keep_first, s);
             return launch_staged<bf16>(staged_size, queries, rows, value_pages, out, out_stride, positions, token_seq, page_rows, page_stride, page_tokens,
                                        tokens, heads, kv_heads, dim, vdim, scale, window, chunk, sink, out_scale, distance, sigmoid_weights, head_offset, gate, gate_stride,
-                                       gate_per_head, splits, partial, s);
+                                       gate_per_head, splits, partial, keep_first, s);
         }
     }
-    const size_t bytes = static_cast<size_t>(kWarps) * dim * sizeof(float);
-    if (bytes > 40 * 1024) return cudaErrorInvalidValue;
+    const size_t bytes = static_cast<size_t>(kWarps) * dim * (shared_keys ? kv_heads : 1) * sizeof(float);
+    if (bytes > kMaxShared) return cudaErrorInvalidValue;
     dim3 grid(tokens, (heads + kWarps - 1) / kWarps);
 #define TAU_ATTEND(T)                                                                                                                         \
+    if (bytes > 40 * 1024) {                                                                                                                  \
+        const cudaError_t status = cudaFuncSetAttribute(masked_attention_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxShared);  \
+        if (status != cudaSuccess) return static_cast<int>(status);                                                                           \
+    }                                                                                                                                         \
     tau_launch(masked_attention_kernel<T>, grid, dim3(kWarps * 32), bytes, s, static_cast<const T*>(queries), static_cast<const T*>(rows), static_cast<const T*>(value_pages), static_cast<T*>(out), \
                out_stride, positions, token_seq, page_rows, page_stride, page_tokens, heads, kv_heads, dim, vdim, scale, window, chunk, sink, out_scale, distance,         \
-               sigmoid_weights, head_offset, static_cast<const T*>(gate), gate_stride, gate_per_head)
-    if (dtype == TAU_F32) TAU_ATTEND(float);
-    else if (dtype == TAU_BF16) TAU_ATTEND(bf16);
+               sigmoid_weights, head_offset, static_cast<const T*>(gate), gate_stride, gate_per_head, keep_first, shared_keys)
+    if (dtype == TAU_F32) { TAU_ATTEND(float); }
+    else if (dtype == TAU_BF16) { TAU_ATTEND(bf16); }
     else return cudaErrorInvalidValue;
 #undef TAU_ATTEND
     return tau_launch_status();

@@ -1,6 +1,7 @@
 // A residual stream kept in 32-bit beside activations of another dtype: embedding rows widened to float, and the
 // fused sum of up to two branches into the stream followed by RMSNorm, with the output in the activations' dtype.
-// Also the gated output stage of mixers whose result is 32-bit: optional RMS norm per group, weight, sigmoid gate.
+// Also the gated output stage of mixers whose result is 32-bit: optional RMS norm per group, weight, sigmoid gate; the same sum
+// followed by an element-wise tanh in a norm's place; and a soft cap on logits.
 #include "common.cuh"
 
 namespace {
@@ -83,6 +84,97 @@ stream_add_norm_kernel(float* __restrict__ stream, const void* __restrict__ a, i
     }
 }
 
+// r = rows ? rows[i] : i.  sum = stream[r] + branch_scale * (a[r] + b[r]) in 32-bit; if `update` the sum replaces stream[r];
+// out[i] = tanh(alpha * sum) * weight + bias, rounded once to T.  No element needs another, so a thread takes `kPer` neighbouring columns
+// of one row (16-byte accesses of the stream where kPer is 4).
+template <int kPer>
+__device__ __forceinline__ void load_columns(const void* base, int code, size_t index, float (&v)[kPer]) {
+    if (kPer == 4 && code == TAU_BF16) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(static_cast<const bf16*>(base) + index);
+        v[0] = __uint_as_float(raw.x << 16), v[1 % kPer] = __uint_as_float(raw.x & 0xffff0000u);
+        v[2 % kPer] = __uint_as_float(raw.y << 16), v[3 % kPer] = __uint_as_float(raw.y & 0xffff0000u);
+    } else if (kPer == 4) {
+        const float4 raw = *reinterpret_cast<const float4*>(static_cast<const float*>(base) + index);
+        v[0] = raw.x, v[1 % kPer] = raw.y, v[2 % kPer] = raw.z, v[3 % kPer] = raw.w;
+    } else {
+        v[0] = load_as_float(base, code, index);
+    }
+}
+
+template <int kPer>
+__device__ __forceinline__ void store_columns(float* target, const float (&v)[kPer]) {
+    if (kPer == 4) *reinterpret_cast<float4*>(target) = make_float4(v[0], v[1 % kPer], v[2 % kPer], v[3 % kPer]);
+    else target[0] = v[0];
+}
+template <int kPer>
+__device__ __forceinline__ void store_columns(bf16* target, const float (&v)[kPer]) {
+    if (kPer == 4) {
+        const __nv_bfloat162 low = __floats2bfloat162_rn(v[0], v[1 % kPer]), high = __floats2bfloat162_rn(v[2 % kPer], v[3 % kPer]);
+        *reinterpret_cast<uint2*>(target) = make_uint2(*reinterpret_cast<const unsigned*>(&low), *reinterpret_cast<const unsigned*>(&high));
+    } else {
+        target[0] = __float2bfloat16_rn(v[0]);
+    }
+}
+
+template <typename T, int kPer>
+__global__ void __launch_bounds__(kThreads)
+stream_add_tanh_kernel(float* __restrict__ stream, const void* __restrict__ a, int a_code, const void* __restrict__ b, int b_code, const int* __restrict__ rows,
+                       const float* __restrict__ alpha, const float* __restrict__ weight, const float* __restrict__ bias, T* __restrict__ out, int width,
+                       int update, float branch_scale) {
+    grid_dependents_launch();
+    grid_dependency_wait();
+    const int column = (blockIdx.y * kThreads + threadIdx.x) * kPer;
+    if (column >= width) return;
+    const size_t base = static_cast<size_t>(rows ? rows[blockIdx.x] : static_cast<int>(blockIdx.x)) * width + column;
+    float value[kPer], result[kPer];
+    load_columns<kPer>(stream, TAU_F32, base, value);
+    if (a) {
+        float branch[kPer];
+        load_columns<kPer>(a, a_code, base, branch);
+        if (b) {
+            float second[kPer];
+            load_columns<kPer>(b, b_code, base, second);
+#pragma unroll
+            for (int i = 0; i < kPer; ++i) branch[i] += second[i];
+        }
+#pragma unroll
+        for (int i = 0; i < kPer; ++i) value[i] = fmaf(branch_scale, branch[i], value[i]);
+        if (update) store_columns<kPer>(stream + base, value);
+    }
+    float w[kPer], offset[kPer];
+    load_columns<kPer>(weight, TAU_F32, column, w);
+    load_columns<kPer>(bias, TAU_F32, column, offset);
+    const float steep = *alpha;
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) result[i] = fmaf(tanhf(steep * value[i]), w[i], offset[i]);
+    store_columns<kPer>(out + static_cast<size_t>(blockIdx.x) * width + column, result);
+}
+
+template <typename T>
+void launch_add_tanh(float* stream_values, const void* a, int a_code, const void* b, int b_code, const int* rows, const float* alpha, const float* weight,
+                     const float* bias, void* out, int out_rows, int width, int update, float branch_scale, cudaStream_t s) {
+    if (width % 4 == 0)
+        tau_launch(stream_add_tanh_kernel<T, 4>, dim3(out_rows, (width / 4 + kThreads - 1) / kThreads), dim3(width / 4 < kThreads ? (width / 4 + 31) / 32 * 32 : kThreads), 0, s,
+                   stream_values, a, a_code, b, b_code, rows, alpha, weight, bias, static_cast<T*>(out), width, update, branch_scale);
+    else
+        tau_launch(stream_add_tanh_kernel<T, 1>, dim3(out_rows, (width + kThreads - 1) / kThreads), dim3(kThreads), 0, s, stream_values, a, a_code, b, b_code,
+                   rows, alpha, weight, bias, static_cast<T*>(out), width, update, branch_scale);
+}
+
+// logits = cap * tanh(logits / cap), in place.
+template <int kPer>
+__global__ void __launch_bounds__(kThreads) soft_cap_kernel(float* __restrict__ values, long long count, float cap) {
+    grid_dependents_launch();
+    grid_dependency_wait();
+    for (long long index = (blockIdx.x * static_cast<long long>(kThreads) + threadIdx.x) * kPer; index < count; index += static_cast<long long>(gridDim.x) * kThreads * kPer) {
+        float v[kPer];
+        load_columns<kPer>(values, TAU_F32, index, v);
+#pragma unroll
+        for (int i = 0; i < kPer; ++i) v[i] = cap * tanhf(v[i] / cap);
+        store_columns<kPer>(values + index, v);
+    }
+}
+
 // out[row] = left_scale * left[row] / rms(left[row]) * left_weight + right_scale * right[row] / rms(right[row]) * right_weight: two results
 // that are normalised over their whole width, each with its own weight, before they are added (eps inside the roots); all 32-bit.
 __global__ void __launch_bounds__(kThreads)
@@ -109,7 +201,7 @@ normed_pair_sum_kernel(const float* __restrict__ left, const float* __restrict__
 // apart), rounded once to T; output rows lie `out_stride` apart.
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
-gated_group_norm_kernel(const float* __restrict__ values, const float* __restrict__ weight, const T* __restrict__ gate, long long gate_stride,
+gated_group_norm_kernel(const float* __restrict__ values, const float* __restrict__ weight, const void* __restrict__ gate, int gate_code, long long gate_stride,
                         T* __restrict__ out, long long out_stride, int groups, int group_width, float eps, int normalize, int silu_gate) {
     grid_dependents_launch();
     grid_dependency_wait();
@@ -133,7 +225,7 @@ gated_group_norm_kernel(const float* __restrict__ values, const float* __restric
                 float value = source[index] * inverse;
                 if (weight) value *= weight[index];
                 if (gate) {
-                    const float z = to_float(gate[static_cast<size_t>(row) * gate_stride + index]);
+                    const float z = load_as_float(gate, gate_code, static_cast<size_t>(row) * gate_stride + index);
                     value *= (silu_gate ? z : 1.0f) / (1.0f + expf(-z));
                 }
                 out[static_cast<size_t>(row) * out_stride + index] = from_float<T>(value);
@@ -156,7 +248,7 @@ gated_group_norm_kernel(const float* __restrict__ values, const float* __restric
             float value = source[index] * inverse;
             if (weight) value *= weight[index];
             if (gate) {
-                const float z = to_float(gate[static_cast<size_t>(row) * gate_stride + index]);
+                const float z = load_as_float(gate, gate_code, static_cast<size_t>(row) * gate_stride + index);
                 value *= (silu_gate ? z : 1.0f) / (1.0f + expf(-z));
             }
             out[static_cast<size_t>(row) * out_stride + index] = from_float<T>(value);
@@ -189,6 +281,30 @@ TAU_EXPORT int tau_stream_add_norm(int out_dtype, float* stream_values, const vo
     return tau_launch_status();
 }
 
+TAU_EXPORT int tau_stream_add_tanh(int out_dtype, float* stream_values, const void* a, int a_dtype, const void* b, int b_dtype, const int* rows,
+                                   const float* alpha, const float* weight, const float* bias, void* out, int out_rows, int width, int update,
+                                   float branch_scale, void* stream) {
+    if (out_rows <= 0) return 0;
+    if (!stream_values || !alpha || !weight || !bias || !out || width <= 0 || (b && !a) || (update && rows)) return cudaErrorInvalidValue;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (out_dtype == TAU_F32) launch_add_tanh<float>(stream_values, a, a_dtype, b, b_dtype, rows, alpha, weight, bias, out, out_rows, width, update, branch_scale, s);
+    else if (out_dtype == TAU_BF16) launch_add_tanh<bf16>(stream_values, a, a_dtype, b, b_dtype, rows, alpha, weight, bias, out, out_rows, width, update, branch_scale, s);
+    else return cudaErrorInvalidValue;
+    return tau_launch_status();
+}
+
+TAU_EXPORT int tau_soft_cap(float* values, long long count, float cap, void* stream) {
+    if (count <= 0) return 0;
+    if (!values || !(cap > 0.0f)) return cudaErrorInvalidValue;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const bool vectors = count % 4 == 0 && (reinterpret_cast<uintptr_t>(values) & 15u) == 0;
+    const long long blocks = (count / (vectors ? 4 : 1) + kThreads - 1) / kThreads;
+    const dim3 grid(static_cast<unsigned>(blocks < 148 * 8 ? blocks : 148 * 8));
+    if (vectors) tau_launch(soft_cap_kernel<4>, grid, dim3(kThreads), 0, s, values, count, cap);
+    else tau_launch(soft_cap_kernel<1>, grid, dim3(kThreads), 0, s, values, count, cap);
+    return tau_launch_status();
+}
+
 TAU_EXPORT int tau_normed_pair_sum(const float* left, const float* right, const float* left_weight, const float* right_weight, float* out, int rows, int width,
                                    float eps, float left_scale, float right_scale, void* stream) {
     if (rows <= 0) return 0;
@@ -198,14 +314,14 @@ TAU_EXPORT int tau_normed_pair_sum(const float* left, const float* right, const 
     return tau_launch_status();
 }
 
-TAU_EXPORT int tau_gated_group_norm(int dtype, const float* values, const float* weight, const void* gate, long long gate_stride, void* out, long long out_stride,
+TAU_EXPORT int tau_gated_group_norm(int dtype, const float* values, const float* weight, const void* gate, int gate_dtype, long long gate_stride, void* out, long long out_stride,
                                     int rows, int groups, int group_width, float eps, int normalize, int silu_gate, void* stream) {
     if (rows <= 0) return 0;
     if (!values || !out || groups <= 0 || group_width <= 0) return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const int threads = 256;
-    if (dtype == TAU_F32) tau_launch(gated_group_norm_kernel<float>, dim3(rows), dim3(threads), 0, s, values, weight, static_cast<const float*>(gate), gate_stride, static_cast<float*>(out), out_stride, groups, group_width, eps, normalize, silu_gate);
-    else if (dtype == TAU_BF16) tau_launch(gated_group_norm_kernel<bf16>, dim3(rows), dim3(threads), 0, s, values, weight, static_cast<const bf16*>(gate), gate_stride, static_cast<bf16*>(out), out_stride, groups, group_width, eps, normalize, silu_gate);
+    if (dtype == TAU_F32) tau_launch(gated_group_norm_kernel<float>, dim3(rows), dim3(threads), 0, s, values, weight, gate, gate_dtype, gate_stride, static_cast<float*>(out), out_stride, groups, group_width, eps, normalize, silu_gate);
+    else if (dtype == TAU_BF16) tau_launch(gated_group_norm_kernel<bf16>, dim3(rows), dim3(threads), 0, s, values, weight, gate, gate_dtype, gate_stride, static_cast<bf16*>(out), out_stride, groups, group_width, eps, normalize, silu_gate);
     else return cudaErrorInvalidValue;
     return tau_launch_status();
 }

@@ -3,7 +3,11 @@
 //     o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t            S_t = diag(w_t) S_(t-1) + k_t v_t^T            (S is key_dim x value_dim)
 //
 // so the read-out sees the states of the tokens before and the token's own k v^T weighed by the head's bonus u; the state then decays
-// by w_t per key channel and takes k v^T unweighed.
+// by w_t per key channel and takes k v^T unweighed.  Two more forms share the walk; both read the state after the token has been written,
+// o_t = S_t^T r_t, and have no bonus:
+//
+//     forget writes:   S_t = diag(w_t) S_(t-1) + (1 - w_t) v_t^T           (what a channel forgets is what it writes; there is no k)
+//     constant decay:  S_t = d S_(t-1) + k_t v_t^T                         (one number d per head)
 //
 //   shift:   every projection reads its own mix of the token's input h and the input of the token before (h' = the sequence's kept
 //            last input for a run's first token, zeros when the sequence starts): mix_s = h + (h' - h) * mu_s, for `mixes` vectors mu.
@@ -89,11 +93,15 @@ constexpr int kGroup = kDim <= 256 ? 4 : 2;      // (two for very wide keys: the
 
 constexpr int kDepth = kDim <= 64 ? 4 : kDim <= 128 ? 3 : 2;
 
-template <int kColumns>
+enum Form : int { kBonus = 0, kForgetWrites = 1, kConstantDecay = 2 };
+
+// `per_head`: the bonus [heads, kDim], or the constant decays [heads].  Rows of r, k, w lie `key_stride` floats apart, rows of v `value_stride`.
+template <int kColumns, int kForm>
 __global__ void __launch_bounds__(kColumns * kSplit)
-wkv_kernel(const float* __restrict__ r, const float* __restrict__ k, const float* __restrict__ v, const float* __restrict__ w, const float* __restrict__ bonus,
-           float* __restrict__ state, long long slot_stride, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot, float* __restrict__ out,
-           int heads, int value_dim) {
+wkv_kernel(const float* __restrict__ r, const float* __restrict__ k, const float* __restrict__ v, const float* __restrict__ w, long long key_stride,
+           long long value_stride, const float* __restrict__ per_head, float* __restrict__ state, long long slot_stride, const int* __restrict__ cu_seqlens,
+           const int* __restrict__ seq_slot, float* __restrict__ out, int heads, int value_dim) {
+    constexpr bool kHasKeys = kForm != kForgetWrites, kHasDecays = kForm != kConstantDecay;
     grid_dependents_launch();
     grid_dependency_wait();
     __shared__ __align__(16) float rs[kDepth][kGroup][kDim], ks[kDepth][kGroup][kDim], ws[kDepth][kGroup][kDim];
@@ -107,8 +115,9 @@ wkv_kernel(const float* __restrict__ r, const float* __restrict__ k, const float
 #pragma unroll
     for (int i = 0; i < kRows; ++i) {
         S[i] = (live && row0 + i < kDim) ? record[row0 + i] : 0.0f;
-        own[i] = row0 + i < kDim ? bonus[static_cast<size_t>(head) * kDim + row0 + i] : 0.0f;
+        own[i] = (kForm == kBonus && row0 + i < kDim) ? per_head[static_cast<size_t>(head) * kDim + row0 + i] : 0.0f;
     }
+    const float constant = kForm == kConstantDecay ? per_head[head] : 0.0f;
     const int begin = cu_seqlens[sequence], end = cu_seqlens[sequence + 1];
     const int groups = (end - begin + kGroup - 1) / kGroup;
     constexpr int kStage = (kDim + kColumns * kSplit - 1) / (kColumns * kSplit);
@@ -119,17 +128,17 @@ wkv_kernel(const float* __restrict__ r, const float* __restrict__ k, const float
         for (int t = 0; t < kGroup; ++t) {
             const int token = begin + group * kGroup + t;
             if (group < groups && token < end) {
-                const size_t keys = (static_cast<size_t>(token) * heads + head) * kDim;
+                const size_t keys = static_cast<size_t>(token) * key_stride + head * kDim;
 #pragma unroll
                 for (int i = 0; i < kStage; ++i) {
                     const int d = threadIdx.x + i * kColumns * kSplit;
                     if (d < kDim) {
                         copy_float(&rs[half][t][d], r + keys + d);
-                        copy_float(&ks[half][t][d], k + keys + d);
-                        copy_float(&ws[half][t][d], w + keys + d);
+                        if (kHasKeys) copy_float(&ks[half][t][d], k + keys + d);
+                        if (kHasDecays) copy_float(&ws[half][t][d], w + keys + d);
                     }
                 }
-                if (part == 0 && live) copy_float(&vs[half][t][local], v + (static_cast<size_t>(token) * heads + head) * value_dim + column);
+                if (part == 0 && live) copy_float(&vs[half][t][local], v + static_cast<size_t>(token) * value_stride + head * value_dim + column);
             }
         }
         copy_commit();
@@ -148,9 +157,15 @@ wkv_kernel(const float* __restrict__ r, const float* __restrict__ k, const float
 #pragma unroll
             for (int i = 0; i < kRows; ++i) {
                 if (kExact || row0 + i < kDim) {
-                    const float write = ks[half][t][row0 + i] * value;                 // the token's own k v^T, this thread's rows of this column
-                    sums[i & 1] = fmaf(fmaf(own[i], write, S[i]), rs[half][t][row0 + i], sums[i & 1]);
-                    S[i] = fmaf(ws[half][t][row0 + i], S[i], write);
+                    const float keep = kHasDecays ? ws[half][t][row0 + i] : constant;
+                    const float write = (kHasKeys ? ks[half][t][row0 + i] : 1.0f - keep) * value;      // the token's own k v^T, this thread's rows of this column
+                    if (kForm == kBonus) {
+                        sums[i & 1] = fmaf(fmaf(own[i], write, S[i]), rs[half][t][row0 + i], sums[i & 1]);
+                        S[i] = fmaf(keep, S[i], write);
+                    } else {
+                        S[i] = fmaf(keep, S[i], write);
+                        sums[i & 1] = fmaf(S[i], rs[half][t][row0 + i], sums[i & 1]);
+                    }
                 }
             }
             parts[t][part][local] = sums[0] + sums[1];
@@ -228,11 +243,13 @@ TAU_EXPORT int tau_channel_decay(float* values, const float* offset, long long r
     return tau_launch_status();
 }
 
-// state: [heads, value_dim, key_dim] floats per slot, slots `slot_stride` apart.
-TAU_EXPORT int tau_wkv(const float* r, const float* k, const float* v, const float* w, const float* bonus, float* state, long long slot_stride,
-                       const int* cu_seqlens, const int* seq_slot, float* out, int n_seqs, int heads, int value_dim, void* stream) {
+// state: [heads, value_dim, key_dim] floats per slot, slots `slot_stride` apart.  `form`: 0 with a bonus, 1 forget writes (no k, no
+// `per_head`), 2 constant decay (no w).
+TAU_EXPORT int tau_wkv(int form, const float* r, const float* k, const float* v, const float* w, long long key_stride, long long value_stride,
+                       const float* per_head, float* state, long long slot_stride, const int* cu_seqlens, const int* seq_slot, float* out, int n_seqs,
+                       int heads, int value_dim, void* stream) {
     if (n_seqs <= 0) return 0;
-    if (!r || !k || !v || !w || !bonus || !state || !cu_seqlens || !seq_slot || !out || heads <= 0 || value_dim <= 0) return cudaErrorInvalidValue;
+    if (form < kBonus || form > kConstantDecay || !r || (form != kForgetWrites && !k) || !v || (form != kConstantDecay && !w) || (form != kForgetWrites && !per_head) || !state || !cu_seqlens || !seq_slot || !out || heads <= 0 || value_dim <= 0) return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     // Value columns to a block: 32 where that many blocks fill the machine, else 16 (blocks of 8 and 4 columns were slower: every block
     // brings the head's r, k and w for itself, and that, not the walk, is then a block's work).
@@ -240,9 +257,18 @@ TAU_EXPORT int tau_wkv(const float* r, const float* k, const float* v, const flo
     if (cudaGetDevice(&device) == cudaSuccess) cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
     const int tile = static_cast<long long>(heads) * n_seqs * ((value_dim + 31) / 32) < sms ? 16 : 32;
     dim3 grid(heads, n_seqs, (value_dim + tile - 1) / tile), block(tile * kSplit);
-#define TAU_WKV(COLUMNS) tau_launch(wkv_kernel<COLUMNS>, grid, block, 0, s, r, k, v, w, bonus, state, slot_stride, cu_seqlens, seq_slot, out, heads, value_dim)
-    if (tile == 32) TAU_WKV(32);
-    else TAU_WKV(16);
+#define TAU_WKV(COLUMNS, FORM) \
+    tau_launch(wkv_kernel<COLUMNS, FORM>, grid, block, 0, s, r, k, v, w, key_stride, value_stride, per_head, state, slot_stride, cu_seqlens, seq_slot, out, heads, value_dim)
+    if (form == kBonus) {
+        if (tile == 32) TAU_WKV(32, kBonus);
+        else TAU_WKV(16, kBonus);
+    } else if (form == kForgetWrites) {
+        if (tile == 32) TAU_WKV(32, kForgetWrites);
+        else TAU_WKV(16, kForgetWrites);
+    } else {
+        if (tile == 32) TAU_WKV(32, kConstantDecay);
+        else TAU_WKV(16, kConstantDecay);
+    }
 #undef TAU_WKV
     return tau_launch_status();
 }

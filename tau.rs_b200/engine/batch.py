@@ -79,6 +79,7 @@ class StepContext:
     all_fresh: bool = False      # every sequence starts at position 0 in this step (nothing of it is cached yet)
     results: object = None       # [runs + 1, n_tokens, hidden] 32-bit, where the model keeps every run's result (`ModelSpec.keeps_results`)
     run: int = 0                 # index of the schedule entry that is being computed
+    handed_on: Dict[str, torch.Tensor] = field(default_factory=dict)   # what a layer leaves for later layers of the same step, row by token
 
 
 def fill_step(layout: StepLayout, out: np.ndarray, entries: Sequence[StepEntry], starts: Sequence[int], cache) -> None:

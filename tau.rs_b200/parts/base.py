@@ -26,7 +26,8 @@ class CacheNeed:
     query reads only the positions of its own chunk of `chunk` positions (chunks counted from
     position 0), so that what lies before the newest chunk need not be kept.  `kind == "state"`:
     one tensor of `state_shape` and `state_dtype` for each sequence, zero when the sequence
-    starts, whatever its length.
+    starts, whatever its length.  `keep_first` (beside a window): the first that many positions
+    are read by every query and kept as long as the sequence lives.
     """
 
     kind: str
@@ -37,6 +38,7 @@ class CacheNeed:
     state_dtype: torch.dtype = torch.float32
     row_width: int = 0
     chunk: Optional[int] = None
+    keep_first: int = 0
 
 
 class Pending(tuple):

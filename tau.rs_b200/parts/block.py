@@ -24,18 +24,22 @@ class PreNormBlock(Block):
     mixer_norm_name = "input_layernorm"
     feed_forward_norm_name = "post_attention_layernorm"
 
+    norm_suffix = ".weight"
+
     def __init__(self, spec, dtype, device):
         self.spec = spec
-        prefix = spec.prefix
-        self.mixer_norm = build("norm", spec.mixer_norm, name=f"{prefix}.{self.mixer_norm_name}.weight", dtype=dtype, device=device)
+        prefix, suffix = spec.prefix, self.norm_suffix
+        self.mixer_norm = build("norm", spec.mixer_norm, name=f"{prefix}.{self.mixer_norm_name}{suffix}", dtype=dtype, device=device)
         self.mixer = build("mixer", spec.mixer, prefix=f"{prefix}.{self.mixer_name}", dtype=dtype, device=device)
-        self.feed_forward_norm = build(
-            "norm", spec.feed_forward_norm, name=f"{prefix}.{self.feed_forward_norm_name}.weight", dtype=dtype, device=device
-        )
-        self.feed_forward = build(
-            "feed_forward", spec.feed_forward, prefix=f"{prefix}.{self.feed_forward_name}", dtype=dtype, device=device
-        )
-        self._children = (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward)
+        self.feed_forward_norm = self.feed_forward = None
+        if spec.feed_forward is not None:
+            self.feed_forward_norm = build(
+                "norm", spec.feed_forward_norm, name=f"{prefix}.{self.feed_forward_norm_name}{suffix}", dtype=dtype, device=device
+            )
+            self.feed_forward = build(
+                "feed_forward", spec.feed_forward, prefix=f"{prefix}.{self.feed_forward_name}", dtype=dtype, device=device
+            )
+        self._children = tuple(part for part in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward) if part is not None)
         self.capturable = all(getattr(part, "capturable", True) for part in self._children)
 
     def cache_need(self):
@@ -69,8 +73,31 @@ class PreNormBlock(Block):
         else:
             normalized = self.mixer_norm.add_forward(branch, residual)
         mixed = self.mixer.forward(normalized, step, cache, writes_cache)
+        if self.feed_forward is None:
+            return residual, mixed
         normalized = self.feed_forward_norm.add_forward(mixed, residual)
         return residual, self.feed_forward.forward(normalized, step)
+
+
+@register_block("pre_norm_stream")
+class StreamPreNormBlock(PreNormBlock):
+    """The same arrangement on a residual stream kept in 32-bit: a sublayer's result joins it and the new stream passes the next norm in one
+    kernel (the norm's `add_forward`); the feed-forward may be absent.  What the mixer keeps beside its cache is the block's as well.
+    Weight names: `<prefix>.norm1`, `<prefix>.mix.*`, `<prefix>.norm2`, `<prefix>.mlp.*`."""
+
+    mixer_name = "mix"
+    feed_forward_name = "mlp"
+    mixer_norm_name = "norm1"
+    feed_forward_norm_name = "norm2"
+    norm_suffix = ""
+
+    def extra_cache_needs(self):
+        return self.mixer.extra_cache_needs()
+
+    def forward(self, residual, branch, step, cache, writes_cache: bool):
+        if residual.dtype != torch.float32:
+            raise ValueError("this block keeps its residual stream in 32-bit (ModelSpec.residual_dtype)")
+        return super().forward(residual, branch, step, cache, writes_cache)
 
 
 @register_block("parallel")

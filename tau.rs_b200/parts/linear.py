@@ -68,10 +68,10 @@ class StackedLinear(Part):
                       for prefix, width in self.pieces]
             self.bias = biases[0] if len(biases) == 1 else torch.cat(biases, dim=0).contiguous()
 
-    def forward_gated(self, values):
-        """`silu(first piece) * second piece`, for a stack built with `interleave`."""
+    def forward_gated(self, values, limit: float = 0.0):
+        """`silu(first piece) * second piece`, for a stack built with `interleave`; with `limit` > 0 the clamped form of `kernels.silu_mul`."""
         out = torch.empty((values.shape[0], self.out_features // 2), dtype=values.dtype, device=values.device)
-        kernels.linear_gated(values, self.weight, out)
+        kernels.linear_gated(values, self.weight, out, **({"limit": limit} if limit else {}))
         return out
 
     def forward(self, values, out_dtype=None, rows: Optional[int] = None):

@@ -1,4 +1,5 @@
-"""Gated feed-forward: `down(act(gate(x)) * up(x))`, no biases; `act` is SiLU (SwiGLU) or, by the spec's `activation`, ReLU.
+"""Gated feed-forward: `down(act(gate(x)) * up(x))`, no biases; `act` is SiLU (SwiGLU) or, by the spec's `activation`, ReLU; or the
+clamped gate `down(g sigmoid(1.702 g) (u + 1))` with `g = min(gate(x), limit)` and `u = up(x)` held between -limit and limit.
 
 crates/models/src/components/mlp.rs:99-122,177-191; gate and up are one stacked product
 followed by one fused activation kernel (crates/models/src/components/mlp/
@@ -20,11 +21,15 @@ class SwiGLU(FeedForward):
     def __init__(self, spec, prefix: str, dtype, device):
         self.spec = spec
         self.activation = getattr(spec, "activation", "silu")
-        if self.activation not in ("silu", "relu"):
+        if self.activation not in ("silu", "relu", "clamped"):
             raise ValueError(f"unknown activation {self.activation!r}")
-        # Where the gated product exists (bfloat16, aligned sizes; its epilogue is SiLU) gate and up rows are interleaved for it and
+        self.limit = float(getattr(spec, "limit", 0.0)) if self.activation == "clamped" else 0.0
+        if self.activation == "clamped" and self.limit <= 0.0:
+            raise ValueError("a clamped gate needs a positive limit")
+        self.result_dtype = torch.float32 if getattr(spec, "wide_result", False) else None
+        # Where the gated product exists (bfloat16, aligned sizes; its epilogue is SiLU or the clamped gate) gate and up rows are interleaved for it and
         # the activation is its epilogue; otherwise the two are stacked and the activation is a kernel of its own.
-        self.fused = self.activation == "silu" and kernels.gated_fits(spec.hidden, spec.intermediate, dtype)
+        self.fused = self.activation != "relu" and kernels.gated_fits(spec.hidden, spec.intermediate, dtype)
         gate, up, down = (getattr(spec, key, default) for key, default in (("gate_name", "gate_proj"), ("up_name", "up_proj"), ("down_name", "down_proj")))
         suffix = getattr(spec, "weight_suffix", ".weight")
         self.gate_up = StackedLinear(
@@ -46,11 +51,11 @@ class SwiGLU(FeedForward):
 
     def forward(self, hidden, step):
         if self.fused:
-            return self.down.forward(self.gate_up.forward_gated(hidden))
+            return self.down.forward(self.gate_up.forward_gated(hidden, self.limit), out_dtype=self.result_dtype)
         stacked = self.gate_up.forward(hidden)
         activated = torch.empty((hidden.shape[0], self.spec.intermediate), dtype=hidden.dtype, device=hidden.device)
-        kernels.silu_mul(stacked, activated, relu=self.activation == "relu")
-        return self.down.forward(activated)
+        kernels.silu_mul(stacked, activated, relu=self.activation == "relu", **({"limit": self.limit} if self.limit else {}))
+        return self.down.forward(activated, out_dtype=self.result_dtype)
 
 
 @register_feed_forward("dense_mlp")

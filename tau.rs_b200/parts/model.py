@@ -163,9 +163,12 @@ class DecoderModel:
             step.run = run
             residual, branch = self.blocks[entry.layer].forward(residual, branch, step, view, entry.writes_cache)
         step.results = None
+        step.handed_on.clear()
         if step.n_wanted == 0:
             return None
         normalized = self.final_norm.forward(residual, rows=step.want_rows, branch=branch)
         logits = torch.empty((step.n_wanted, spec.vocab_size), dtype=torch.float32, device=self.device)
         kernels.linear(normalized, self.head, None, logits)
+        if getattr(spec, "logit_cap", 0.0):
+            kernels.soft_cap(logits, spec.logit_cap)
         return logits

@@ -83,3 +83,37 @@ class LayerNorm(Norm):
         out = torch.empty((count, self.spec.width), dtype=self.dtype or values.dtype, device=values.device)
         kernels.norm_rows(values, rows, self.weight, self.bias, self.spec.eps, True, out)
         return out
+
+
+@register_norm("dynamic_tanh")
+class DynamicTanh(Norm):
+    """`tanh(alpha * x) * w + b`: no statistic of the row, each element stands alone; computed in 32-bit, one rounding.  `x` is a residual
+    stream kept in 32-bit, and a pending branch joins it in the same kernel.  Tensors: `<name>` and `<name><spec.bias_suffix>` of the
+    width, `<name>.alpha` one number."""
+
+    def __init__(self, spec, name: str, dtype, device):
+        self.spec, self.name, self.bias_name, self.alpha_name = spec, name, name + spec.bias_suffix, name + ".alpha"
+        self.dtype = dtype
+        self.weight = self.bias = self.alpha = None
+
+    def tensor_specs(self):
+        width = self.spec.width
+        return {self.name: TensorSpec((width,), role="vector", init="ones"), self.bias_name: TensorSpec((width,), role="vector"),
+                self.alpha_name: TensorSpec((), role="vector", init="ones")}
+
+    def assign(self, name, tensor):
+        attribute = {self.name: "weight", self.bias_name: "bias", self.alpha_name: "alpha"}.get(name)
+        if attribute is None:
+            raise KeyError(name)
+        setattr(self, attribute, tensor)
+
+    def forward(self, values, rows=None, branch=None):
+        count = values.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((count, self.spec.width), dtype=self.dtype or values.dtype, device=values.device)
+        kernels.stream_add_tanh(values, branch, self.alpha, self.weight, self.bias, out, rows, update=False, branch_scale=getattr(branch, "scale", 1.0))
+        return out
+
+    def add_forward(self, branch, residual):
+        out = torch.empty(residual.shape, dtype=self.dtype or residual.dtype, device=residual.device)
+        kernels.stream_add_tanh(residual, branch, self.alpha, self.weight, self.bias, out, update=True, branch_scale=getattr(branch, "scale", 1.0))
+        return out
