@@ -365,9 +365,31 @@ def nugolorn_sizes():
     }
 
 
+def bikovik_sizes():
+    """Layer sizes that resemble a real model of Bikovik's kind: two attention layers with mixed scores (128-element heads, 4 key/value heads,
+    half of each head rotated, a window of 1,024 positions beside the first 64), a matrix memory whose forget gate writes (128 by 128
+    states) and a retention (128 by 256 states), every layer with a clamped feed-forward of 8/3 of the width.  Beside it the closest design
+    that was here before, Nugolorn (attention, matrix memories), and a dense Qwen3, each of the same width, depth and vocabulary."""
+    def bikovik(width, heads, ff):
+        attention = {"heads": heads, "kv_heads": 4, "dim": 128, "vdim": 128, "mask": {"size": 1024, "keep_first": 64}, "rot": {"base": 10000.0, "dims": 64},
+                     "scale": 128 ** -0.5, "v_mix": True}
+        memory = {"heads": heads, "dim": 128, "vdim": 128}
+        retention = {"heads": heads, "dim": 128, "vdim": 256, "decay": [1.0 - 2.0 ** (-5 - 5 * head / heads) for head in range(heads)], "rot": {"base": 10000.0, "dims": 128}}
+        layers = [{"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}}
+                  for kind, mixer in (("attention", attention), ("hgrn2", memory), ("attention", attention), ("retention", retention))]
+        return {"architecture": "Bikovik", "embedding": {"scale": 1.0}, "layers": layers, "logit_softcap": 30.0, "norm": {"eps": 1e-5}, "vocab": 32768, "width": width}
+
+    nugolorn = nugolorn_sizes()
+    return {
+        "1024": (bikovik(1024, 8, 2752), nugolorn["1024"][1], nugolorn["1024"][0]),
+        "2048": (bikovik(2048, 16, 5440), nugolorn["2048"][1], nugolorn["2048"][0]),
+        "4096": (bikovik(4096, 32, 10944), nugolorn["4096"][1], nugolorn["4096"][0]),
+    }
+
+
 def design_comparison(args) -> int:
-    """`--design fasesun|bisudra|pegurax|nugolorn`: prefill and decode throughput of the design's layers at three real sizes beside a dense Qwen3
-    of equal width, depth and active feed-forward width (Pegurax also beside Fasesun, Nugolorn also beside Pegurax), with the device time of each kernel class in one
+    """`--design fasesun|bisudra|pegurax|nugolorn|bikovik`: prefill and decode throughput of the design's layers at three real sizes beside a dense Qwen3
+    of equal width, depth and active feed-forward width (Pegurax also beside Fasesun, Nugolorn also beside Pegurax, Bikovik also beside Nugolorn), with the device time of each kernel class in one
     prompt step and one decode step."""
     import numpy as np
     import torch
@@ -383,7 +405,7 @@ def design_comparison(args) -> int:
     records = []
     clocks = ClockSampler()
     clocks.start()
-    sizes = {"bisudra": bisudra_sizes, "fasesun": fasesun_sizes, "pegurax": pegurax_sizes, "nugolorn": nugolorn_sizes}[args.design]()
+    sizes = {"bisudra": bisudra_sizes, "fasesun": fasesun_sizes, "pegurax": pegurax_sizes, "nugolorn": nugolorn_sizes, "bikovik": bikovik_sizes}[args.design]()
     for size, (design_config, dense_config, *others) in sizes.items():
         if args.widths and size not in args.widths.split(","):
             continue
@@ -482,7 +504,7 @@ def main() -> int:
                         help="which measurements to run: prefill, decode, points, e2e, kernels (the counterparts of the reference arm's kernels), "
                              "classes (time per kernel class of a decode step, outside a graph)")
     parser.add_argument("--widths", default="", help="with --design: only these of the widths 1024, 2048, 4096 (comma-separated)")
-    parser.add_argument("--design", default="", choices=["", "fasesun", "bisudra", "pegurax", "nugolorn"],
+    parser.add_argument("--design", default="", choices=["", "fasesun", "bisudra", "pegurax", "nugolorn", "bikovik"],
                         help="instead of the default workload: layers of this design at real sizes beside a dense Qwen3 of equal size")
     args = parser.parse_args()
 

@@ -22,7 +22,8 @@
 // A third form (`kSegments`) is for scores mixed over the heads, score_h = sum_g talk[h, g] q_g . k: the caller's queries are mixed
 // beforehand, one piece of D elements for each key head, and S = sum over the key heads j of Q_j K_j^T accumulates in tensor memory
 // piece by piece.  The Q tile is then `n_kv_heads` pieces wide, a stage of the key ring holds one key head's tile, and one block has an
-// SM to itself.
+// SM to itself.  Where so wide a Q tile does not fit, its pieces travel with the key tiles instead, one in every stage of the ring (read
+// again for every tile of keys: slower, but of any width).
 //
 // The accumulator O is rescaled only when a row's maximum has grown by more than 2^8 since the last rescale, so most
 // tiles do not touch it; the final division by the row sum makes the result exact either way.  The score products run
@@ -310,15 +311,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                             int page_stride, int n_seqs, int n_tokens, int n_heads, int n_kv_heads, float scale, int window, int chunk, int sink,
                             float out_scale, long long out_stride, int n_items, int* __restrict__ schedule, const float* __restrict__ distance,
                             int sigmoid_weights, const float* __restrict__ head_offset, const bf16* __restrict__ head_gate, long long gate_stride,
-                            int keep_first_keys, int stages_of_keys) {
+                            int keep_first_keys, int stages_of_keys, int queries_in_ring) {
     const int keep_first = kExtended ? keep_first_keys : 0;
     const int segments = kSegments ? n_kv_heads : 1;                                        // pieces of a query, each against one key head
     const uint32_t key_stages = kSegments ? static_cast<uint32_t>(stages_of_keys) : kKeyStages;
+    const bool ring_queries = kSegments && queries_in_ring != 0;                            // a stage holds a key tile, then the piece of Q that meets it
+    const uint32_t stage_bytes = kKeyBytes + (ring_queries ? kQBytes : 0);
     extern __shared__ uint8_t shared_raw[];
     uint8_t* tiles = shared_raw;                                   // the swizzled tiles need 1,024-byte alignment
     uint8_t* q_tile = tiles;                                       // kHalves slices of [128 rows x 128 bytes]
-    uint8_t* key_tiles = tiles + segments * kQBytes;               // key_stages key tiles
-    uint8_t* value_tiles = key_tiles + key_stages * kKeyBytes;     // kValueStages value tiles
+    uint8_t* key_tiles = tiles + (ring_queries ? 0 : segments * kQBytes);   // key_stages stages
+    uint8_t* value_tiles = key_tiles + key_stages * stage_bytes;   // kValueStages value tiles
     Shared* shared = reinterpret_cast<Shared*>(value_tiles + kValueStages * kKeyBytes);
     if ((smem_address(shared_raw) & 1023u) != 0u) {   // never seen; the same for every thread, before anything is set up
         if (threadIdx.x == 0) atomicExch(&attention_tc_error, 2);
@@ -436,10 +439,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 if (span.n_tiles > 0) {
                     const int kv_head = item.head / (n_heads / n_kv_heads);
                     const int* pages = page_rows + static_cast<size_t>(item.seq) * page_stride;
-                    if (n > 0 && !barrier_wait(&shared->q_free, (n - 1) & 1u, abort_flag)) break;
-                    barrier_expect_bytes(&shared->q_full, segments * kQBytes);
-                    for (int slice = 0; slice < segments * kHalves; ++slice)
-                        tma_load_2d(q_tile + slice * (BM * 128), &q_map, item.head * segments * D + slice * 64, item.row, &shared->q_full);
+                    if (!ring_queries) {
+                        if (n > 0 && !barrier_wait(&shared->q_free, (n - 1) & 1u, abort_flag)) break;
+                        barrier_expect_bytes(&shared->q_full, segments * kQBytes);
+                        for (int slice = 0; slice < segments * kHalves; ++slice)
+                            tma_load_2d(q_tile + slice * (BM * 128), &q_map, item.head * segments * D + slice * 64, item.row, &shared->q_full);
+                    }
                     // The place of key tile i is free when the scores of the tile kKeyStages before it are done, which is
                     // earlier than the place of value tile i (free when the second product of the tile kValueStages
                     // before it is done): keys are asked for ahead of values, in the order in which their places come free.
@@ -450,9 +455,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                             const uint32_t use = kt / key_stages;
                             if (use > 0 && !barrier_wait(&shared->k_free[s], (use - 1) & 1u, abort_flag)) return false;
                             const int row = (page * n_kv_heads + (kSegments ? segment : kv_head)) * BN;
-                            barrier_expect_bytes(&shared->k_full[s], kKeyBytes);
-                            for (int half = 0; half < kHalves; ++half)
-                                tma_load_2d(key_tiles + s * kKeyBytes + half * (BN * 128), &k_map, half * 64, row, &shared->k_full[s]);
+                            uint8_t* stage = key_tiles + s * stage_bytes;
+                            barrier_expect_bytes(&shared->k_full[s], stage_bytes);
+                            for (int half = 0; half < kHalves; ++half) tma_load_2d(stage + half * (BN * 128), &k_map, half * 64, row, &shared->k_full[s]);
+                            if (ring_queries)
+                                for (int half = 0; half < kHalves; ++half)
+                                    tma_load_2d(stage + kKeyBytes + half * (BM * 128), &q_map, (item.head * segments + segment) * D + half * 64, item.row, &shared->k_full[s]);
                             ++kt;
                         }
                         return true;
@@ -506,7 +514,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 if (kSegments && tile >= 2 && !barrier_wait(&shared->s_free[tile & 1], ((tile >> 1) - 1) & 1u, abort_flag)) return false;
                 for (int segment = 0; segment < segments; ++segment) {
                     const int s = kt % key_stages;
-                    const uint32_t key_address = smem_address(key_tiles + s * kKeyBytes), piece_address = q_address + segment * kQBytes;
+                    const uint32_t key_address = smem_address(key_tiles + s * stage_bytes);
+                    const uint32_t piece_address = ring_queries ? key_address + kKeyBytes : q_address + segment * kQBytes;
                     if (!barrier_wait(&shared->k_full[s], (kt / key_stages) & 1u, abort_flag)) return false;
                     if (!kSegments && tile >= 2 && !barrier_wait(&shared->s_free[tile & 1], ((tile >> 1) - 1) & 1u, abort_flag)) return false;
                     tensor_fence_after_sync();
@@ -532,7 +541,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 if (item.seq < 0) break;
                 const int n_tiles = span_of(item, window, chunk, keep_first).n_tiles;
                 if (n_tiles == 0) continue;
-                alive = barrier_wait(&shared->q_full, n & 1u, abort_flag) && issue_scores(t, n_tiles == 1);
+                alive = (ring_queries || barrier_wait(&shared->q_full, n & 1u, abort_flag)) && issue_scores(t, n_tiles == 1);
                 for (int i = 0; i < n_tiles && alive; ++i) {
                     if (i + 1 < n_tiles && !issue_scores(t + i + 1, i + 2 == n_tiles)) { alive = false; break; }
                     const uint32_t tile = t + i;
@@ -866,7 +875,7 @@ TAU_EXPORT int tau_attention_prefill_tc_status() {
     return flag;
 }
 
-// Key tiles in flight of the segmented form for that many key heads, 0 where its tiles do not fit an SM's shared memory.
+// Key tiles in flight of the segmented form for that many key heads, 0 where a Q tile of so many pieces does not fit an SM's shared memory.
 namespace {
 constexpr int kMostShared = 227 * 1024;
 int segmented_bytes(int n_kv_heads, int key_stages) { return n_kv_heads * kQBytes + (key_stages + kValueStages) * kKeyBytes + static_cast<int>(sizeof(Shared)); }
@@ -876,9 +885,11 @@ int segmented_key_stages(int n_kv_heads) {
         if (segmented_bytes(n_kv_heads, stages) <= kMostShared) return stages;
     return 0;
 }
+// With the pieces of Q in the ring's stages.
+constexpr int kRingStages = 3;
+constexpr int kRingBytes = kRingStages * (kKeyBytes + kQBytes) + kValueStages * kKeyBytes + static_cast<int>(sizeof(Shared));
+static_assert(kRingBytes <= kMostShared, "the ring fits an SM");
 }  // namespace
-
-TAU_EXPORT int tau_attention_prefill_tc_segments_fit(int n_kv_heads) { return segmented_key_stages(n_kv_heads) > 0; }
 
 // `segmented`: queries are [n_tokens, n_heads * n_kv_heads * D], a piece for each key head, and a score is the sum over the key heads.
 // `keep_first`: the sequence's first that many positions stay visible beside a window.
@@ -904,9 +915,8 @@ TAU_EXPORT int tau_attention_prefill_tc(const void* queries, const void* keys, c
         !make_map(&v_map, values, cache_rows, D, BN) || !make_map(&out_map, out, n_tokens, static_cast<long long>(n_heads) * D, BM, out_stride))
         return cudaErrorInvalidValue;
     if (segmented) {
-        const int key_stages = segmented_key_stages(n_kv_heads);
-        if (key_stages == 0) return cudaErrorInvalidValue;
-        const int bytes = segmented_bytes(n_kv_heads, key_stages);
+        const int resident = segmented_key_stages(n_kv_heads), key_stages = resident > 0 ? resident : kRingStages;
+        const int bytes = resident > 0 ? segmented_bytes(n_kv_heads, key_stages) : kRingBytes;
         const cudaError_t status = cudaFuncSetAttribute(attention_prefill_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMostShared);
         if (status != cudaSuccess) return static_cast<int>(status);
         int device = 0, sms = 0;
@@ -917,7 +927,7 @@ TAU_EXPORT int tau_attention_prefill_tc(const void* queries, const void* keys, c
         tau_launch(attention_prefill_tc_kernel<true, true>, dim3(static_cast<unsigned>(items < fit ? items : fit)), dim3(kThreads), bytes, static_cast<cudaStream_t>(stream),
                    q_map, k_map, v_map, out_map, static_cast<bf16*>(out), cu_seqlens, seq_start, page_rows, page_stride, n_seqs, n_tokens, n_heads, n_kv_heads, scale,
                    window, chunk, sink, out_scale, out_stride, static_cast<int>(items), schedule, distance, sigmoid_weights, head_offset,
-                   static_cast<const bf16*>(head_gate), gate_stride, keep_first, key_stages);
+                   static_cast<const bf16*>(head_gate), gate_stride, keep_first, key_stages, resident > 0 ? 0 : 1);
         return tau_launch_status();
     }
     const int shared_bytes = kQBytes + (kKeyStages + kValueStages) * kKeyBytes + static_cast<int>(sizeof(Shared));
@@ -943,6 +953,6 @@ TAU_EXPORT int tau_attention_prefill_tc(const void* queries, const void* keys, c
     tau_launch(extended ? attention_prefill_tc_kernel<true, false> : attention_prefill_tc_kernel<false, false>, dim3(blocks), dim3(kThreads), shared_bytes,
                static_cast<cudaStream_t>(stream), q_map, k_map, v_map, out_map, static_cast<bf16*>(out), cu_seqlens, seq_start, page_rows, page_stride, n_seqs,
                n_tokens, n_heads, n_kv_heads, scale, window, chunk, sink, out_scale, out_stride, static_cast<int>(items), schedule, distance, sigmoid_weights,
-               head_offset, static_cast<const bf16*>(head_gate), gate_stride, keep_first, kKeyStages);
+               head_offset, static_cast<const bf16*>(head_gate), gate_stride, keep_first, kKeyStages, 0);
     return tau_launch_status();
 }

@@ -754,8 +754,7 @@ def attention_prefill_tc(queries, keys, values, out, cu_seqlens, seq_start, page
     `sigmoid(score + head_offset[head])` (float32 [n_heads] or None) instead of its share of a softmax.  `head_gate` (bfloat16
     [tokens, n_heads], rows any distance apart): a head's result is multiplied by the sigmoid of its number.  `keep_first`: the
     sequence's first that many positions stay visible beside a window.  `segmented`: a query has a piece of `head_dim` elements for each
-    key head (`queries` [tokens, n_heads * n_kv_heads * head_dim]) and a score is the sum over the key heads; where
-    `attention_prefill_tc_segments_fit`."""
+    key head (`queries` [tokens, n_heads * n_kv_heads * head_dim]) and a score is the sum over the key heads."""
     _on_device(queries, keys, values, out, cu_seqlens, seq_start, page_rows, distance, head_offset, head_gate)
     if distance is not None:
         _require(distance.dtype == torch.float32 and distance.shape == (n_heads, 2) and distance.is_contiguous(), "the distance numbers must be float32 [heads, 2]")
@@ -790,12 +789,6 @@ def attention_prefill_tc(queries, keys, values, out, cu_seqlens, seq_start, page
         ctypes.c_int(1 if sink else 0), ctypes.c_float(out_scale), ctypes.c_longlong(out.stride(0)), _pointer(schedule), _pointer(distance),
         ctypes.c_int(1 if sigmoid_weights else 0), _pointer(head_offset), _pointer(head_gate), ctypes.c_longlong(0 if head_gate is None else head_gate.stride(0)),
         ctypes.c_int(keep_first), ctypes.c_int(1 if segmented else 0), _stream()), "attention_prefill_tc")
-
-
-def attention_prefill_tc_segments_fit(head_dim: int, n_kv_heads: int) -> bool:
-    """Whether the segmented form of `attention_prefill_tc` serves that many key heads."""
-    library = build.load_library("attention_prefill_tc.cu", (f"TAU_HEAD_DIM={head_dim}",))
-    return bool(library.tau_attention_prefill_tc_segments_fit(ctypes.c_int(n_kv_heads)))
 
 
 def attention_prefill_tc_status(head_dim: int) -> int:

@@ -204,8 +204,7 @@ class MaskedAttention(JoinableMixer):
         if mixed_queries:
             options["shared_keys"] = True
         if (self.heads_layout and not step.all_single and projected.dtype == torch.bfloat16 and kernels.optimized_preferred()
-                and keys.shape[0] * spec.n_kv_heads * kernels.PAGE_TOKENS <= 0x7FFFFFFF and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
-                and (not mixed_queries or kernels.attention_prefill_tc_segments_fit(spec.dim, spec.n_kv_heads))):
+                and keys.shape[0] * spec.n_kv_heads * kernels.PAGE_TOKENS <= 0x7FFFFFFF and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0):
             # Runs of new tokens on the tensor cores; a gate per head leaves with the rows, a gate per element is a pass of its own.
             if "shared_keys" in options:
                 options["segmented"] = options.pop("shared_keys")

@@ -55,8 +55,8 @@ ODD = config([attention(heads=1, kv_heads=1, dim=12, vdim=150, size=1, keep_firs
               hgrn2(heads=1, dim=20, vdim=70, mlp=dense(14, 0.3)),
               retention(heads=1, dim=10, vdim=34, decay=[1.0], rot_dims=2, mlp=dense(22, 2.0)),
               attention(heads=9, kv_heads=3, dim=10, vdim=50, size=37, keep_first=3, rot_dims=2, mlp=None),
-              retention(heads=5, dim=6, vdim=3, decay=[0.05, 0.5, 0.9, 0.99, 1.0], rot_dims=6, mlp=None),
-              hgrn2(heads=5, dim=6, vdim=1, mlp=None),
+              retention(heads=5, dim=6, vdim=13, decay=[0.05, 0.5, 0.9, 0.99, 1.0], rot_dims=6, mlp=None),
+              hgrn2(heads=5, dim=6, vdim=5, mlp=None),
               attention(heads=3, kv_heads=3, dim=7, vdim=50, size=100, keep_first=1, rot_dims=6, mlp=dense(6, 1.0)),
               hgrn2(heads=2, dim=100, vdim=10, mlp=None)],
              width=100, vocab=77, eps=1e-6, scale=1.0, cap=30.0)
@@ -69,7 +69,7 @@ PEAKY = config([attention(heads=3, kv_heads=1, dim=16, vdim=24, size=64, keep_fi
 HEADY = config([attention(heads=4, kv_heads=2, dim=64, vdim=64, size=90, keep_first=20, rot_dims=64, scale=0.4, mlp=None),
                 attention(heads=4, kv_heads=1, dim=128, vdim=128, size=64, keep_first=1, rot_dims=64, scale=0.2, mlp=None),
                 attention(heads=3, kv_heads=3, dim=128, vdim=128, size=200, keep_first=130, rot_dims=32, scale=0.2, v_mix=False, mlp=None)], width=64, vocab=97, scale=1.3)
-# More key heads than the tensor-core kernel's tiles fit beside one another, and more value columns than the single-token kernel owns.
+# More key heads than the tensor-core kernel's query tile holds pieces for, and more value columns than the single-token kernel owns.
 WIDE = config([attention(heads=8, kv_heads=8, dim=128, vdim=128, size=70, keep_first=10, rot_dims=128, mlp=None),
                attention(heads=48, kv_heads=2, dim=16, vdim=200, size=33, keep_first=2, rot_dims=8, v_mix=False, mlp=None)], width=64, vocab=97)
 # States that forget slowly, so that one lost or restarted shows hundreds of tokens later.
@@ -113,9 +113,9 @@ def weights(cfg: dict, seed: int, slow_forgetting: bool = False) -> Dict[str, to
         if layer["type"] == "attention":
             kv_heads = mixer["kv_heads"]
             for name, rows in (("q", heads * dim), ("k", kv_heads * dim), ("v", kv_heads * vdim)):
-                matrix(f"{p}.mix.{name}", rows, width, 2.0)
+                matrix(f"{p}.mix.{name}", rows, width, 1.3)
                 vector(f"{p}.mix.{name}.b", rows, 0.0, 0.3)
-            out[f"{p}.mix.talk"] = torch.eye(heads) + 0.4 * torch.randn(heads, heads, generator=generator)
+            out[f"{p}.mix.talk"] = torch.eye(heads) + 0.4 * torch.randn(heads, heads, generator=generator) / heads ** 0.5
             if mixer["v_mix"]:
                 out[f"{p}.mix.vmix"] = 0.3 + 0.3 * torch.rand((), generator=generator)
         elif layer["type"] == "hgrn2":
@@ -128,7 +128,7 @@ def weights(cfg: dict, seed: int, slow_forgetting: bool = False) -> Dict[str, to
         else:
             for name, rows in (("q", heads * dim), ("k", heads * dim), ("v", heads * vdim), ("g", heads * vdim)):
                 matrix(f"{p}.mix.{name}", rows, width, 2.0)
-        matrix(f"{p}.mix.o", width, heads * vdim)
+        matrix(f"{p}.mix.o", width, heads * vdim, 0.7)
         if mlp is not None:
             norm(f"{p}.norm2")
             matrix(f"{p}.mlp.gate", mlp["ff"], width, 2.0)

@@ -27,11 +27,11 @@ F = torch.float64
 
 def close(found, wanted, dtype) -> bool:
     """float32: every logit within 5e-5 of the largest.  bfloat16 (the plain statement rounds nothing): half of the positions within
-    3e-2 of the largest logit and all but one in twenty (or two) within 1e-1."""
+    3e-2 of the largest logit and all but one in twenty (or two) within 8e-2."""
     if dtype == "float32":
         return relative_error(found, wanted) < TOLERANCE[dtype]
     rows = (found.double() - wanted.double()).abs().amax(dim=-1) / wanted.double().abs().max()
-    return float(rows.median()) < 3e-2 and int((rows >= 1e-1).sum()) <= max(2, rows.numel() // 20)
+    return float(rows.median()) < 3e-2 and int((rows >= 8e-2).sum()) <= max(2, rows.numel() // 20)
 
 
 def tokens_for(cfg, count, seed):
@@ -266,9 +266,8 @@ def test_mixed_scores_with_a_window_and_kept_positions_over_scattered_pages(dtyp
     tolerance = 2e-5 if dtype == "float32" else 2e-2
     per = 4 if dtype == "float32" else 8
     modes = ["kernel"] + (["single"] if dim % per == 0 and vdim % per == 0 and kernels.talking_decode_fits(kind, heads, kv_heads, dim, vdim) else [])
-    if heads_layout and dtype == "bfloat16" and kernels.attention_prefill_tc_segments_fit(dim, kv_heads):
+    if heads_layout and dtype == "bfloat16":      # (8 key heads of 128: the pieces of the queries travel with the keys)
         modes.append("tensor")
-    assert dtype == "float32" or not heads_layout or kv_heads * dim > 512 or "tensor" in modes
     for mode in modes:
         found = run_attention(q, k, v, dim ** -0.5, talk, window, keep_first, dtype, [5, 2, 7, 0], heads_layout, 210, mode)
         assert relative_error(found, wanted) < tolerance, mode
