@@ -21,9 +21,11 @@
 // hold them first, and goes on at its window's first page.
 // A third form (`kSegments`) is for scores mixed over the heads, score_h = sum_g talk[h, g] q_g . k: the caller's queries are mixed
 // beforehand, one piece of D elements for each key head, and S = sum over the key heads j of Q_j K_j^T accumulates in tensor memory
-// piece by piece.  The Q tile is then `n_kv_heads` pieces wide, a stage of the key ring holds one key head's tile, and one block has an
-// SM to itself.  Where so wide a Q tile does not fit, its pieces travel with the key tiles instead, one in every stage of the ring (read
-// again for every tile of keys: slower, but of any width).
+// piece by piece.  The Q tile is then `n_kv_heads` pieces wide and a block has an SM, and all of its tensor memory, to itself.  With one
+// block nobody fills the gaps of a chain of products that all wait for one accumulator, so two pages' scores are computed by one product
+// of 128 keys (twice the work per link of the chain, and half the reads of Q); the ring's stages are 64 elements of one key head for both
+// pages.  Where so wide a Q tile does not fit, its pieces travel with the keys instead, one in every stage of the ring (read again for
+// every pair of pages: slower, but of any width).
 //
 // The accumulator O is rescaled only when a row's maximum has grown by more than 2^8 since the last rescale, so most
 // tiles do not touch it; the final division by the row sum makes the result exact either way.  The score products run
@@ -61,7 +63,9 @@ constexpr int kKeyBytes = BN * D * 2;   // a key tile, or a value tile
 #define TAU_ATTN_KEY_STAGES 2
 #endif
 constexpr int kKeyStages = TAU_ATTN_KEY_STAGES;   // key tiles in flight: a key tile is free as soon as its scores are done
-constexpr int kMostKeyStages = kKeyStages > 4 ? kKeyStages : 4;   // the segmented form has as many as fit, up to this
+constexpr int kMostKeyStages = 8;                 // the segmented form has as many stages as fit, up to this
+constexpr int kPairUnit = 2 * BN * 128;           // its stages: 64 elements of two pages' keys,
+constexpr int kQueryUnit = BM * 128;              // and, where Q travels with the keys, 64 elements of the Q piece that meets them
 constexpr int kValueStages = 2;                   // value tiles in flight: free when the second product of their tile is done
 // Shared memory: Q, the key ring, the value ring, then the barriers; nothing is spent on aligning the tiles (dynamic
 // shared memory starts at a multiple of 1,024 bytes, which the kernel checks before it does anything else), so that
@@ -70,7 +74,7 @@ constexpr int kValueStages = 2;                   // value tiles in flight: free
 // tensor core waits for.
 constexpr uint32_t kColumns = 256;      // two score buffers in columns [0, 64) and [64, 128), O in columns [128, 128 + D);
                                         // the probabilities of a tile (bfloat16 pairs, 32 columns) take the place of its scores
-constexpr uint32_t kOColumn = 128;
+                                        // (segmented: two buffers of two tiles' scores in columns [0, 128) and [128, 256), O behind them)
 constexpr float kRescaleThreshold = 8.0f;
 constexpr unsigned long long kWaitLimitNs = 2000000000ull;
 
@@ -270,8 +274,8 @@ struct Shared {
     uint64_t v_free[kValueStages];  // the second product that read a value tile has finished
     uint64_t s_full[2];             // scores of a tile are in their buffer of tensor memory
     uint64_t s_free[2];             // the softmax has read that buffer
-    uint64_t p_ready[2];            // probabilities of a tile are in tensor memory (and O has been rescaled if need be)
-    uint64_t pv_done;               // the second product of a tile has finished
+    uint64_t p_ready[4];            // (two of them, four in the segmented form, whose softmax may be three tiles ahead) probabilities of a tile are in tensor memory (and O has been rescaled if need be)
+    uint64_t pv_done[4];            // the second product of a tile has finished (the segmented form's tiles take turns, the others use the first)
     uint64_t staged;                // the four softmax warps are done with the place of the value tiles: an item's output rows lie
                                     // there for the producer to send off (a whole tile), or have been written by the warps (a ragged one)
     uint64_t item_full[2];          // an item has been written to its place
@@ -279,6 +283,14 @@ struct Shared {
     Item item[2];
     uint32_t tensor_memory_base;
     int abort_flag;
+};
+
+// A place in a ring of stages, and how often (modulo two) the ring has been gone round.
+struct RingPlace {
+    uint32_t stage = 0, phase = 0;
+    __device__ __forceinline__ void advance(uint32_t stages) {
+        if (++stage == stages) stage = 0, phase ^= 1u;
+    }
 };
 
 // The tiles of an item: which keys its rows see.  Tiles are numbered from 0; the first `kept_tiles` are the sequence's first pages.
@@ -315,8 +327,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     const int keep_first = kExtended ? keep_first_keys : 0;
     const int segments = kSegments ? n_kv_heads : 1;                                        // pieces of a query, each against one key head
     const uint32_t key_stages = kSegments ? static_cast<uint32_t>(stages_of_keys) : kKeyStages;
-    const bool ring_queries = kSegments && queries_in_ring != 0;                            // a stage holds a key tile, then the piece of Q that meets it
-    const uint32_t stage_bytes = kKeyBytes + (ring_queries ? kQBytes : 0);
+    const bool ring_queries = kSegments && queries_in_ring != 0;                            // a stage holds keys, then what of Q meets them
+    const uint32_t stage_bytes = kSegments ? kPairUnit + (ring_queries ? kQueryUnit : 0) : kKeyBytes;
+    constexpr uint32_t kScoreColumns = kSegments ? 2 * BN : BN, kOColumn = 2 * kScoreColumns, kBlockColumns = kSegments ? 512 : kColumns;
+    constexpr uint32_t kReady = kSegments ? 4 : 2;                                          // barriers that tiles' probabilities take turns on,
+    constexpr uint32_t kDone = kSegments ? 4 : 1;                                           // and those of the second products' ends
     extern __shared__ uint8_t shared_raw[];
     uint8_t* tiles = shared_raw;                                   // the swizzled tiles need 1,024-byte alignment
     uint8_t* q_tile = tiles;                                       // kHalves slices of [128 rows x 128 bytes]
@@ -350,18 +365,20 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         for (int b = 0; b < 2; ++b) {
             barrier_init(&shared->s_full[b], 1);
             barrier_init(&shared->s_free[b], 4);     // one arrival per softmax warp
-            barrier_init(&shared->p_ready[b], 4);
             barrier_init(&shared->item_full[b], 1);
             barrier_init(&shared->item_free[b], 5);  // the issuer and the four softmax warps
         }
-        barrier_init(&shared->pv_done, 1);
+        for (int b = 0; b < 4; ++b) {
+            barrier_init(&shared->p_ready[b], 4);
+            barrier_init(&shared->pv_done[b], 1);
+        }
         barrier_init(&shared->staged, 4);
         shared->abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     if (warp == 5) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_address(&shared->tensor_memory_base)),
-                     "r"(kColumns)
+                     "r"(kBlockColumns)
                      : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
@@ -412,7 +429,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 barrier_arrive(&shared->item_full[k & 1]);   // a release: the item is written before the arrival shows
                 return true;
             };
-            uint32_t kt = 0, vt = 0, n = 0;   // key tiles, value tiles and items with work so far
+            uint32_t kt = 0, vt = 0, n = 0;   // key tiles (segmented: stages), value tiles and items with work so far
+            RingPlace ring;
             // The output rows of an item leave through the place of the value tiles when all its products are done.  A whole
             // tile (or one that ends with the step's last token, where the copy engine cuts it off) is sent by this thread
             // as soon as the four warps have put it there; the warps write a ragged tile themselves.  Either way the place
@@ -449,19 +467,32 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     // earlier than the place of value tile i (free when the second product of the tile kValueStages
                     // before it is done): keys are asked for ahead of values, in the order in which their places come free.
                     auto load_keys = [&](int i) {
-                        const int page = pages[span.page(i)];
-                        for (int segment = 0; segment < segments; ++segment) {      // (segmented: the tile of every key head, one after the other)
-                            const int s = kt % key_stages;
-                            const uint32_t use = kt / key_stages;
-                            if (use > 0 && !barrier_wait(&shared->k_free[s], (use - 1) & 1u, abort_flag)) return false;
-                            const int row = (page * n_kv_heads + (kSegments ? segment : kv_head)) * BN;
-                            uint8_t* stage = key_tiles + s * stage_bytes;
-                            barrier_expect_bytes(&shared->k_full[s], stage_bytes);
-                            for (int half = 0; half < kHalves; ++half) tma_load_2d(stage + half * (BN * 128), &k_map, half * 64, row, &shared->k_full[s]);
-                            if (ring_queries)
-                                for (int half = 0; half < kHalves; ++half)
-                                    tma_load_2d(stage + kKeyBytes + half * (BM * 128), &q_map, (item.head * segments + segment) * D + half * 64, item.row, &shared->k_full[s]);
+                        const int s = kt % kKeyStages;
+                        const uint32_t use = kt / kKeyStages;
+                        if (use > 0 && !barrier_wait(&shared->k_free[s], (use - 1) & 1u, abort_flag)) return false;
+                        const int row = (pages[span.page(i)] * n_kv_heads + kv_head) * BN;
+                        barrier_expect_bytes(&shared->k_full[s], kKeyBytes);
+                        for (int half = 0; half < kHalves; ++half)
+                            tma_load_2d(key_tiles + s * kKeyBytes + half * (BN * 128), &k_map, half * 64, row, &shared->k_full[s]);
+                        ++kt;
+                        return true;
+                    };
+                    // Segmented: 64 elements at a time of every key head, for the pair's two pages (or its one) side by side.
+                    auto load_pair = [&](int pair) {
+                        const int tile = 2 * pair;
+                        const bool both = tile + 1 < span.n_tiles;
+                        const int first_page = pages[span.page(tile)], second_page = both ? pages[span.page(tile + 1)] : 0;
+                        for (int unit = 0; unit < segments * kHalves; ++unit) {
+                            const int segment = unit / kHalves, half = unit % kHalves;
+                            if (kt >= key_stages && !barrier_wait(&shared->k_free[ring.stage], ring.phase ^ 1u, abort_flag)) return false;
+                            uint8_t* stage = key_tiles + ring.stage * stage_bytes;
+                            uint64_t* full = &shared->k_full[ring.stage];
+                            barrier_expect_bytes(full, (both ? kPairUnit : kPairUnit / 2) + (ring_queries ? kQueryUnit : 0));
+                            tma_load_2d(stage, &k_map, half * 64, (first_page * n_kv_heads + segment) * BN, full);
+                            if (both) tma_load_2d(stage + kPairUnit / 2, &k_map, half * 64, (second_page * n_kv_heads + segment) * BN, full);
+                            if (ring_queries) tma_load_2d(stage + kPairUnit, &q_map, (item.head * segments + segment) * D + half * 64, item.row, full);
                             ++kt;
+                            ring.advance(key_stages);
                         }
                         return true;
                     };
@@ -480,14 +511,20 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     // Completion order of the products: scores 0, scores 1, second product 0, scores 2, second product 1, ...; a
                     // load is issued when the product that frees its place is the next to finish, so no wait blocks a later load
                     // whose place is free already: keys run kAhead tiles ahead of values.
-                    // (Segmented: a tile's key heads take turns in the ring, and one tile ahead is as far as the scores run.)
-                    constexpr int kAhead = kSegments ? 1 : kKeyStages - kValueStages + 1;
-                    for (int i = 0; i < span.n_tiles + kAhead && alive; ++i) {
+                    constexpr int kAhead = kKeyStages - kValueStages + 1;
+                    for (int i = 0; !kSegments && i < span.n_tiles + kAhead && alive; ++i) {
                         // The next item is taken when this one has a few tiles left: late, so that blocks which are done
                         // early find the items that remain, but early enough for the answer to be here at this item's end.
                         if (i == max(0, span.n_tiles - 4)) next = take();
                         if (i < span.n_tiles) alive = load_keys(i);
                         if (alive && i >= kAhead) alive = load_values(i - kAhead);
+                    }
+                    // Segmented: scores run a pair ahead of the softmax, so a pair's keys are asked for ahead of the values of the pair before.
+                    const int n_pairs = (span.n_tiles + 1) / 2;
+                    for (int pair = 0; kSegments && pair <= n_pairs && alive; ++pair) {
+                        if (pair == max(0, n_pairs - 2)) next = take();
+                        if (pair < n_pairs) alive = load_pair(pair);
+                        for (int i = max(0, 2 * pair - 2); i < min(2 * pair, span.n_tiles) && alive; ++i) alive = load_values(i);
                     }
                     ++n;
                     sent_row = item.row, sent_head = item.head;
@@ -505,32 +542,50 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         if (lane == 0) {
             const uint32_t score_descriptor = instruction_descriptor(BN, false), value_descriptor = instruction_descriptor(D, true);
             const uint32_t q_address = smem_address(q_tile);
-            uint32_t t = 0, n = 0, kt = 0;   // tiles, items with work and key tiles so far
+            uint32_t t = 0, n = 0, pairs = 0;   // tiles, items with work and (segmented) pairs of tiles so far
+            RingPlace ring;
             // Scores run one tile ahead of the softmax: while the four warps work on tile i, the products of tile i + 1
             // fill the other score buffer, and the second product of tile i follows as soon as its probabilities are there.
             auto issue_scores = [&](uint32_t tile, bool last_of_item) {
+                const int s = tile % kKeyStages;
+                const uint32_t key_address = smem_address(key_tiles + s * kKeyBytes);
+                if (!barrier_wait(&shared->k_full[s], (tile / kKeyStages) & 1u, abort_flag)) return false;
                 // The buffer also held the probabilities of the tile two before; their product was issued before this one and
                 // the tensor core takes products in the order of issue, so only the softmax's read needs waiting for.
-                if (kSegments && tile >= 2 && !barrier_wait(&shared->s_free[tile & 1], ((tile >> 1) - 1) & 1u, abort_flag)) return false;
-                for (int segment = 0; segment < segments; ++segment) {
-                    const int s = kt % key_stages;
-                    const uint32_t key_address = smem_address(key_tiles + s * stage_bytes);
-                    const uint32_t piece_address = ring_queries ? key_address + kKeyBytes : q_address + segment * kQBytes;
-                    if (!barrier_wait(&shared->k_full[s], (kt / key_stages) & 1u, abort_flag)) return false;
-                    if (!kSegments && tile >= 2 && !barrier_wait(&shared->s_free[tile & 1], ((tile >> 1) - 1) & 1u, abort_flag)) return false;
-                    tensor_fence_after_sync();
+                if (tile >= 2 && !barrier_wait(&shared->s_free[tile & 1], ((tile >> 1) - 1) & 1u, abort_flag)) return false;
+                tensor_fence_after_sync();
 #pragma unroll
-                    for (int k = 0; k < D / 16; ++k) {
-                        const uint32_t offset = (k / 4) * 128 * BM + (k % 4) * 32;          // slice of 64 d, then 16 d inside it
-                        const uint32_t key_offset = (k / 4) * 128 * BN + (k % 4) * 32;
-                        mma_issue(tensor_base + (tile & 1) * BN, k_major_descriptor(piece_address + offset),
-                                  k_major_descriptor(key_address + key_offset), score_descriptor, (segment > 0 || k > 0) ? 1u : 0u);
-                    }
-                    mma_commit(&shared->k_free[s]);
-                    ++kt;
+                for (int k = 0; k < D / 16; ++k) {
+                    const uint32_t offset = (k / 4) * 128 * BM + (k % 4) * 32;          // slice of 64 d, then 16 d inside it
+                    const uint32_t key_offset = (k / 4) * 128 * BN + (k % 4) * 32;
+                    mma_issue(tensor_base + (tile & 1) * BN, k_major_descriptor(q_address + offset),
+                              k_major_descriptor(key_address + key_offset), score_descriptor, k > 0 ? 1u : 0u);
                 }
+                mma_commit(&shared->k_free[s]);
                 mma_commit(&shared->s_full[tile & 1]);
                 if (last_of_item) mma_commit(&shared->q_free);
+                return true;
+            };
+            // Segmented: the scores of two tiles (or of an item's last one) by products of 128 (or 64) keys; the buffers take turns pair by pair.
+            auto issue_pair = [&](bool both, bool last_of_item) {
+                const uint32_t slot = pairs & 1;
+                if (pairs >= 2 && !barrier_wait(&shared->s_free[slot], ((pairs >> 1) - 1) & 1u, abort_flag)) return false;
+                const uint32_t descriptor = instruction_descriptor(both ? 2 * BN : BN, false);
+                for (int unit = 0; unit < segments * kHalves; ++unit) {
+                    if (!barrier_wait(&shared->k_full[ring.stage], ring.phase, abort_flag)) return false;
+                    tensor_fence_after_sync();
+                    const uint32_t key_address = smem_address(key_tiles + ring.stage * stage_bytes);
+                    const uint32_t piece_address = ring_queries ? key_address + kPairUnit : q_address + unit * kQueryUnit;
+#pragma unroll
+                    for (int k = 0; k < 4; ++k)
+                        mma_issue(tensor_base + slot * kScoreColumns, k_major_descriptor(piece_address + k * 32), k_major_descriptor(key_address + k * 32), descriptor,
+                                  (unit > 0 || k > 0) ? 1u : 0u);
+                    mma_commit(&shared->k_free[ring.stage]);
+                    ring.advance(key_stages);
+                }
+                mma_commit(&shared->s_full[slot]);
+                if (last_of_item) mma_commit(&shared->q_free);
+                ++pairs;
                 return true;
             };
             bool alive = true;
@@ -541,24 +596,28 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 if (item.seq < 0) break;
                 const int n_tiles = span_of(item, window, chunk, keep_first).n_tiles;
                 if (n_tiles == 0) continue;
-                alive = (ring_queries || barrier_wait(&shared->q_full, n & 1u, abort_flag)) && issue_scores(t, n_tiles == 1);
+                const uint32_t first_pair = pairs;
+                alive = (ring_queries || barrier_wait(&shared->q_full, n & 1u, abort_flag)) && (kSegments ? issue_pair(n_tiles > 1, n_tiles <= 2) : issue_scores(t, n_tiles == 1));
                 for (int i = 0; i < n_tiles && alive; ++i) {
-                    if (i + 1 < n_tiles && !issue_scores(t + i + 1, i + 2 == n_tiles)) { alive = false; break; }
+                    if (kSegments) {
+                        if ((i & 1) == 0 && i + 2 < n_tiles && !issue_pair(i + 3 < n_tiles, i + 4 >= n_tiles)) { alive = false; break; }
+                    } else if (i + 1 < n_tiles && !issue_scores(t + i + 1, i + 2 == n_tiles)) { alive = false; break; }
                     const uint32_t tile = t + i;
+                    const uint32_t column = kSegments ? ((first_pair + (i >> 1)) & 1) * kScoreColumns + (i & 1) * BN : (tile & 1) * BN;
                     const int s = tile % kValueStages;
                     const uint32_t value_address = smem_address(value_tiles + s * kKeyBytes);
                     if (!barrier_wait(&shared->v_full[s], (tile / kValueStages) & 1u, abort_flag)) { alive = false; break; }
                     // Probabilities lie where the scores of the tile were: 16 keys are 8 columns.  The first tile of an item
                     // overwrites O: its probabilities come from the warps that have read the item before's O by then.
-                    if (!barrier_wait(&shared->p_ready[tile & 1], (tile >> 1) & 1u, abort_flag)) { alive = false; break; }
+                    if (!barrier_wait(&shared->p_ready[tile % kReady], (tile / kReady) & 1u, abort_flag)) { alive = false; break; }
                     tensor_fence_after_sync();
 #pragma unroll
                     for (int kk = 0; kk < BN / 16; ++kk) {
-                        mma_issue_from_tensor(tensor_base + kOColumn, tensor_base + (tile & 1) * BN + kk * 8,
+                        mma_issue_from_tensor(tensor_base + kOColumn, tensor_base + column + kk * 8,
                                               mn_major_descriptor(value_address + kk * 2048), value_descriptor, (i > 0 || kk > 0) ? 1u : 0u);
                     }
                     mma_commit(&shared->v_free[s]);
-                    mma_commit(&shared->pv_done);
+                    mma_commit(&shared->pv_done[tile % kDone]);
                 }
                 t += n_tiles;
                 ++n;
@@ -569,7 +628,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         const int row = warp * 32 + lane;                         // warp w may touch lanes 32 w .. 32 w + 31 of tensor memory
         const uint32_t lane_base = tensor_base + (static_cast<uint32_t>(warp * 32) << 16);
         const float scale_log2 = scale * 1.4426950408889634f;
-        uint32_t t = 0;                                           // tiles so far
+        uint32_t t = 0, pairs = 0;                                // tiles and (segmented) pairs of tiles so far
         bool alive = true;
         for (uint32_t k = 0; alive; ++k) {
             if (!barrier_wait(&shared->item_full[k & 1], (k >> 1) & 1u, abort_flag)) break;
@@ -602,13 +661,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
             for (int i = 0; i < n_tiles && alive; ++i) {
                 const uint32_t tile = t + i;
                 const int s = tile % kValueStages;
-                if (!barrier_wait(&shared->s_full[tile & 1], (tile >> 1) & 1u, abort_flag)) { alive = false; break; }
+                const uint32_t score_use = kSegments ? pairs + (i >> 1) : tile;      // of the two score buffers, which take turns
+                const uint32_t column = (score_use & 1) * kScoreColumns + (kSegments ? (i & 1) * BN : 0);
+                if ((!kSegments || (i & 1) == 0) && !barrier_wait(&shared->s_full[score_use & 1], (score_use >> 1) & 1u, abort_flag)) { alive = false; break; }
                 tensor_fence_after_sync();
                 float score[BN];
                 {
                     float low[32], high[32];
-                    tensor_load_32(lane_base + (tile & 1) * BN, low);
-                    tensor_load_32(lane_base + (tile & 1) * BN + 32, high);
+                    tensor_load_32(lane_base + column, low);
+                    tensor_load_32(lane_base + column + 32, high);
                     tensor_load_wait();
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
@@ -618,13 +679,16 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 }
                 tensor_fence_before_sync();
                 __syncwarp();
-                if (lane == 0) barrier_arrive(&shared->s_free[tile & 1]);
+                if (lane == 0 && (!kSegments || (i & 1) == 1 || i == n_tiles - 1)) barrier_arrive(&shared->s_free[score_use & 1]);
                 const int key0 = (kExtended && i < kept_tiles ? i : first_tile + i - (kExtended ? kept_tiles : 0)) * BN;
                 if (key0 + BN - 1 > last_position) {
                     // Rows of the page beyond the last position hold whatever an earlier sequence left there.  Their
                     // probabilities are zero, but zero times a stale NaN is not: clear those value rows before the product.
                     uint8_t* value_tile = value_tiles + s * kKeyBytes;
                     const int first_stale = last_position - key0 + 1;
+                    // (Segmented: the softmax may be so far ahead that the values two tiles before have not landed either; behind their product
+                    // the wait for this tile's names the right phase.)
+                    if (kSegments && i >= 2 && !barrier_wait(&shared->pv_done[(tile - 2) % kDone], ((tile - 2) / kDone) & 1u, abort_flag)) { alive = false; break; }
                     if (!barrier_wait(&shared->v_full[s], (tile / kValueStages) & 1u, abort_flag)) { alive = false; break; }   // the tile must have landed first
                     for (int entry = threadIdx.x; entry < (BN - first_stale) * kHalves * 8; entry += 128) {
                         const int chunk = entry % 8, half = (entry / 8) % kHalves, stale_row = first_stale + entry / (8 * kHalves);
@@ -685,12 +749,14 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 // an item's last probabilities are handed over it may be in phase t - 1, t or t + 1, which a wait for phase t
                 // cannot tell apart (in phase t - 1 it would pass at once, before the last two products): so the last tile
                 // always waits for phase t - 1 first, which leaves t or t + 1 for the wait behind the loop.
+                // (Segmented: the scores of tile t were issued behind the second products of the tiles up to t - 4 only, so these ends take
+                // turns on four barriers, each of which is then in the phase waited for or the next.)
                 const bool last_tile = i == n_tiles - 1 && i > 0;
                 if (__any_sync(0xffffffffu, rescale) || last_tile) {
                     // O must not be touched while the second product of the tile before is still writing it.  Only here (and
                     // at the last tile): a warp whose maxima have settled never waits for that product, and its exponentials
                     // run beside it.
-                    if (!barrier_wait(&shared->pv_done, (tile - 1) & 1u, abort_flag)) { alive = false; break; }
+                    if (!barrier_wait(&shared->pv_done[(tile - 1) % kDone], ((tile - 1) / kDone) & 1u, abort_flag)) { alive = false; break; }
                     tensor_fence_after_sync();
                 }
                 if (__any_sync(0xffffffffu, rescale)) {
@@ -720,8 +786,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     uint32_t zeros[16];
 #pragma unroll
                     for (int j = 0; j < 16; ++j) zeros[j] = 0u;
-                    tensor_store_words_16(lane_base + (tile & 1) * BN, zeros);
-                    tensor_store_words_16(lane_base + (tile & 1) * BN + 16, zeros);
+                    tensor_store_words_16(lane_base + column, zeros);
+                    tensor_store_words_16(lane_base + column + 16, zeros);
                 } else {
                     Float2 partial_sum[4] = {pair_of(0.0f, 0.0f), pair_of(0.0f, 0.0f), pair_of(0.0f, 0.0f), pair_of(0.0f, 0.0f)};
                     // Sigmoid weights: sigmoid(x) = 0.5 tanh(x / 2) + 0.5 with x = score * scale + offset, one special-function instruction a
@@ -742,7 +808,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                             partial_sum[(j >> 1) & 3] = add_pair(partial_sum[(j >> 1) & 3], pair_of(p0, p1));
                             packed[j / 2] = pack_bf16(p0, p1);
                         }
-                        tensor_store_words_16(lane_base + (tile & 1) * BN + half * 16, packed);
+                        tensor_store_words_16(lane_base + column + half * 16, packed);
                     }
                     float low, high;
                     unpair(add_pair(add_pair(partial_sum[0], partial_sum[1]), add_pair(partial_sum[2], partial_sum[3])), low, high);
@@ -752,10 +818,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 if (key0 + BN - 1 > last_position) asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // the cleared value rows, for the tensor core's reads
                 tensor_fence_before_sync();
                 __syncwarp();
-                if (lane == 0) barrier_arrive(&shared->p_ready[tile & 1]);
+                if (lane == 0) barrier_arrive(&shared->p_ready[tile % kReady]);
             }
             t += n_tiles;
-            if (!alive || !barrier_wait(&shared->pv_done, (t - 1) & 1u, abort_flag)) { alive = false; break; }
+            pairs += (n_tiles + 1) / 2;
+            if (!alive || !barrier_wait(&shared->pv_done[(t - 1) % kDone], ((t - 1) / kDone) & 1u, abort_flag)) { alive = false; break; }
             tensor_fence_after_sync();
             // With a sink the denominator has the weight of a key with score 0 and no value added: exp2(0 - used_max) in the sums' scale.
             // Where that overflows every key's weight is nothing beside it, and the row is zero.
@@ -824,7 +891,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     __syncthreads();
     if (warp == 5) {
         tensor_fence_after_sync();
-        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tensor_base), "r"(kColumns) : "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tensor_base), "r"(kBlockColumns) : "memory");
     }
     // The block that leaves last puts the counters back to zero for the next launch.
     if (threadIdx.x == 0 && atomicAdd(schedule + 1, 1) == static_cast<int>(gridDim.x) - 1) {
@@ -875,20 +942,17 @@ TAU_EXPORT int tau_attention_prefill_tc_status() {
     return flag;
 }
 
-// Key tiles in flight of the segmented form for that many key heads, 0 where a Q tile of so many pieces does not fit an SM's shared memory.
+// Stages of the segmented form for that many key heads with Q in a place of its own, 0 where a Q tile of so many pieces leaves no room for two.
 namespace {
-constexpr int kMostShared = 227 * 1024;
-int segmented_bytes(int n_kv_heads, int key_stages) { return n_kv_heads * kQBytes + (key_stages + kValueStages) * kKeyBytes + static_cast<int>(sizeof(Shared)); }
-int segmented_key_stages(int n_kv_heads) {
+constexpr int kMostShared = 227 * 1024, kSegmentedFixed = kValueStages * kKeyBytes + static_cast<int>(sizeof(Shared));
+int segmented_stages(int n_kv_heads) {
     if (n_kv_heads <= 0 || n_kv_heads > 1024) return 0;
-    for (int stages = kMostKeyStages; stages >= 2; --stages)
-        if (segmented_bytes(n_kv_heads, stages) <= kMostShared) return stages;
-    return 0;
+    const int stages = (kMostShared - kSegmentedFixed - n_kv_heads * kQBytes) / kPairUnit;
+    return stages < 2 ? 0 : stages < kMostKeyStages ? stages : kMostKeyStages;
 }
-// With the pieces of Q in the ring's stages.
-constexpr int kRingStages = 3;
-constexpr int kRingBytes = kRingStages * (kKeyBytes + kQBytes) + kValueStages * kKeyBytes + static_cast<int>(sizeof(Shared));
-static_assert(kRingBytes <= kMostShared, "the ring fits an SM");
+// ... and with Q in the ring's stages.
+constexpr int kRingStages = (kMostShared - kSegmentedFixed) / (kPairUnit + kQueryUnit) < kMostKeyStages ? (kMostShared - kSegmentedFixed) / (kPairUnit + kQueryUnit) : kMostKeyStages;
+static_assert(kRingStages >= 2, "the ring fits an SM");
 }  // namespace
 
 // `segmented`: queries are [n_tokens, n_heads * n_kv_heads * D], a piece for each key head, and a score is the sum over the key heads.
@@ -915,19 +979,21 @@ TAU_EXPORT int tau_attention_prefill_tc(const void* queries, const void* keys, c
         !make_map(&v_map, values, cache_rows, D, BN) || !make_map(&out_map, out, n_tokens, static_cast<long long>(n_heads) * D, BM, out_stride))
         return cudaErrorInvalidValue;
     if (segmented) {
-        const int resident = segmented_key_stages(n_kv_heads), key_stages = resident > 0 ? resident : kRingStages;
-        const int bytes = resident > 0 ? segmented_bytes(n_kv_heads, key_stages) : kRingBytes;
+        const int resident = segmented_stages(n_kv_heads), stages = resident > 0 ? resident : kRingStages;
+        // More than half of an SM's shared memory in any case: a block takes all columns of tensor memory, so a second one beside it would wait.
+        int bytes = kSegmentedFixed + (resident > 0 ? n_kv_heads * kQBytes + stages * kPairUnit : stages * (kPairUnit + kQueryUnit));
+        if (bytes < 120 * 1024) bytes = 120 * 1024;
         const cudaError_t status = cudaFuncSetAttribute(attention_prefill_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMostShared);
         if (status != cudaSuccess) return static_cast<int>(status);
         int device = 0, sms = 0;
         if (cudaGetDevice(&device) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device) != cudaSuccess || sms <= 0)
             return cudaErrorInvalidValue;
-        const long long items = (static_cast<long long>((n_tokens + BM - 1) / BM) + n_seqs) * n_heads, fit = bytes + 1024 <= kMostShared / 2 ? 2LL * sms : sms;
+        const long long items = (static_cast<long long>((n_tokens + BM - 1) / BM) + n_seqs) * n_heads;
         if (items > 0x7fffffffLL) return cudaErrorInvalidValue;
-        tau_launch(attention_prefill_tc_kernel<true, true>, dim3(static_cast<unsigned>(items < fit ? items : fit)), dim3(kThreads), bytes, static_cast<cudaStream_t>(stream),
+        tau_launch(attention_prefill_tc_kernel<true, true>, dim3(static_cast<unsigned>(items < sms ? items : sms)), dim3(kThreads), bytes, static_cast<cudaStream_t>(stream),
                    q_map, k_map, v_map, out_map, static_cast<bf16*>(out), cu_seqlens, seq_start, page_rows, page_stride, n_seqs, n_tokens, n_heads, n_kv_heads, scale,
                    window, chunk, sink, out_scale, out_stride, static_cast<int>(items), schedule, distance, sigmoid_weights, head_offset,
-                   static_cast<const bf16*>(head_gate), gate_stride, keep_first, key_stages, resident > 0 ? 0 : 1);
+                   static_cast<const bf16*>(head_gate), gate_stride, keep_first, stages, resident > 0 ? 0 : 1);
         return tau_launch_status();
     }
     const int shared_bytes = kQBytes + (kKeyStages + kValueStages) * kKeyBytes + static_cast<int>(sizeof(Shared));

@@ -47,6 +47,31 @@ __device__ __forceinline__ Visible visible_keys(int position, int window, int ch
     return seen;
 }
 
+constexpr int kMixColumns = 8, kMixHeads = 4;      // of a thread where rows allow 16-byte accesses
+__device__ __forceinline__ void load_columns(const float* source, float (&v)[kMixColumns]) {
+    const float4 low = reinterpret_cast<const float4*>(source)[0], high = reinterpret_cast<const float4*>(source)[1];
+    v[0] = low.x, v[1] = low.y, v[2] = low.z, v[3] = low.w, v[4] = high.x, v[5] = high.y, v[6] = high.z, v[7] = high.w;
+}
+__device__ __forceinline__ void load_columns(const bf16* source, float (&v)[kMixColumns]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(source);
+    const uint32_t words[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) v[2 * i] = __uint_as_float(words[i] << 16), v[2 * i + 1] = __uint_as_float(words[i] & 0xffff0000u);
+}
+__device__ __forceinline__ void store_columns(float* target, const float (&v)[kMixColumns]) {
+    reinterpret_cast<float4*>(target)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(target)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void store_columns(bf16* target, const float (&v)[kMixColumns]) {
+    uint32_t words[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const __nv_bfloat162 pair = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        words[i] = *reinterpret_cast<const uint32_t*>(&pair);
+    }
+    *reinterpret_cast<uint4*>(target) = make_uint4(words[0], words[1], words[2], words[3]);
+}
+
 // grid: tokens; block kWarps * 32.  projected row: [heads * dim | kv_heads * dim | kv_heads * vdim] from its first column on.
 // Dynamic shared memory: rotary / 2 float2 (cosine, sine).
 template <typename T>
@@ -58,7 +83,7 @@ masked_prepare_kernel(const T* __restrict__ projected, long long projected_strid
                       const float* __restrict__ talk, const T* __restrict__ first_values, long long first_stride, const float* __restrict__ value_share) {
     grid_dependents_launch();
     grid_dependency_wait();
-    extern __shared__ float2 turns[];       // then, with `talk`, heads * dim floats: the turned queries
+    extern __shared__ __align__(16) float2 turns[];       // then, on the next 16-byte border, with `talk`, heads * dim floats: the turned queries
     __shared__ float scratch[33];
     const int token = blockIdx.x;
     const int position = positions[token];
@@ -105,56 +130,141 @@ masked_prepare_kernel(const T* __restrict__ projected, long long projected_strid
             value_row = row + k_width;
         }
     }
-    // Items: within each head, the `half` rotated pairs, then the dim - rotary elements that pass.
-    const int per_head = half + (dim - rotary);
-    float* turned = reinterpret_cast<float*>(turns + half);
-    const int q_items = heads * per_head, items = q_items + (write_rows ? kv_heads * per_head : 0);
-    for (int item = threadIdx.x; item < items; item += blockDim.x) {
-        const bool is_query = item < q_items;
-        const int index = is_query ? item : item - q_items;
-        const int head = index / per_head, within = index % per_head;
-        const T* from = source + (is_query ? 0 : q_width) + head * dim;
-        const float* weight = is_query ? q_weight : k_weight;
-        const float inverse = is_query ? q_inverse : k_inverse;
-        T* target = is_query ? queries + static_cast<size_t>(token) * q_width + head * dim : row + head * key_head_stride;
-        if (within < half) {
-            const int first = within, second = within + half;
-            float u = to_float(from[first]) * inverse, w = to_float(from[second]) * inverse;
-            if (weight) {
-                u *= weight[head * dim + first];
-                w *= weight[head * dim + second];
+    // Rows that start on 16 bytes, pairs and heads in multiples of 8 elements, no norm weights: a thread takes 8 pairs, or 8 elements that
+    // pass, or 8 values at a time.
+    float* turned = reinterpret_cast<float*>(turns + (half + 1) / 2 * 2);
+    const T* first_row = (write_rows && first_values) ? first_values + static_cast<size_t>(token) * first_stride : nullptr;
+    const float share = first_row ? *value_share : 0.0f;
+    constexpr uintptr_t kBytes = kMixColumns * sizeof(T) < 16 ? kMixColumns * sizeof(T) - 1 : 15;
+    const bool vectors = dim % kMixColumns == 0 && half % kMixColumns == 0 && vdim % kMixColumns == 0 && !q_weight && !k_weight &&
+                         ((reinterpret_cast<uintptr_t>(source) | reinterpret_cast<uintptr_t>(queries) | reinterpret_cast<uintptr_t>(row) | reinterpret_cast<uintptr_t>(value_row) |
+                           reinterpret_cast<uintptr_t>(first_row)) & kBytes) == 0;
+    if (vectors) {
+        const int pair_pieces = half / kMixColumns, per_head = dim / kMixColumns - pair_pieces;      // of a head: pieces of pairs, then pieces that pass
+        const int head_items = (heads + (write_rows ? kv_heads : 0)) * per_head, value_pieces = vdim / kMixColumns;
+        const int all_items = head_items + (write_rows ? kv_heads * value_pieces : 0);
+        for (int item = threadIdx.x; item < all_items; item += blockDim.x) {
+            float u[kMixColumns];
+            if (item >= head_items) {
+                const int index = item - head_items, head = index / value_pieces, column = (index - head * value_pieces) * kMixColumns;
+                load_columns(source + q_width + k_width + index * kMixColumns, u);
+                if (first_row) {
+                    float first[kMixColumns];
+                    load_columns(first_row + index * kMixColumns, first);
+#pragma unroll
+                    for (int e = 0; e < kMixColumns; ++e) u[e] = (1.0f - share) * u[e] + share * first[e];
+                }
+                store_columns(value_row + head * value_head_stride + column, u);
+                continue;
             }
-            const float2 turn = turns[within];
-            const float a = u * turn.x - w * turn.y, b = w * turn.x + u * turn.y;
-            if (talk && is_query) {
-                turned[head * dim + first] = a;
-                turned[head * dim + second] = b;
-            } else {
-                target[first] = from_float<T>(a);
-                target[second] = from_float<T>(b);
+            const int any_head = item / per_head, piece = item - any_head * per_head;
+            const bool is_query = any_head < heads, pairs = piece < pair_pieces, mix = talk && is_query;
+            const int head = is_query ? any_head : any_head - heads, column = pairs ? piece * kMixColumns : half + piece * kMixColumns;
+            const float factor = is_query ? q_inverse : 1.0f;
+            const T* from = source + (is_query ? 0 : q_width) + head * dim + column;
+            T* target = is_query ? queries + static_cast<size_t>(token) * q_width + head * dim + column : row + head * key_head_stride + column;
+            float* kept = turned + head * dim + column;
+            load_columns(from, u);
+#pragma unroll
+            for (int e = 0; e < kMixColumns; ++e) u[e] *= factor;
+            if (pairs) {
+                float w[kMixColumns];
+                load_columns(from + half, w);
+#pragma unroll
+                for (int e = 0; e < kMixColumns; ++e) {
+                    const float2 turn = turns[column + e];
+                    const float a = u[e], b = w[e] * factor;
+                    u[e] = a * turn.x - b * turn.y;
+                    w[e] = b * turn.x + a * turn.y;
+                }
+                if (mix) store_columns(kept + half, w);
+                else store_columns(target + half, w);
             }
-        } else {
-            const int column = rotary + (within - half);
-            float u = to_float(from[column]) * inverse;
-            if (weight) u *= weight[head * dim + column];
-            if (talk && is_query) turned[head * dim + column] = u;
-            else target[column] = from_float<T>(u);
+            if (mix) store_columns(kept, u);
+            else store_columns(target, u);
         }
-    }
-    if (write_rows) {
-        const T* values = source + q_width + k_width;
-        const T* first = first_values ? first_values + static_cast<size_t>(token) * first_stride : nullptr;
-        const float share = first ? *value_share : 0.0f;
-        for (int column = threadIdx.x; column < kv_heads * vdim; column += blockDim.x) {
-            T value = values[column];
-            if (first) value = from_float<T>((1.0f - share) * to_float(value) + share * to_float(first[column]));
-            value_row[(column / vdim) * value_head_stride + column % vdim] = value;
+    } else {
+        // Within each head, the `half` rotated pairs, then the dim - rotary elements that pass.
+        const int per_head = half + (dim - rotary);
+        const int all_heads = heads + (write_rows ? kv_heads : 0), lane = threadIdx.x & 31;
+        for (int row_head = threadIdx.x >> 5; row_head < all_heads; row_head += kWarps) {      // a warp per head
+            const bool is_query = row_head < heads;
+            const int head = is_query ? row_head : row_head - heads;
+            const T* from = source + (is_query ? 0 : q_width) + head * dim;
+            const float* weight = is_query ? q_weight : k_weight;
+            const float inverse = is_query ? q_inverse : k_inverse;
+            T* target = is_query ? queries + static_cast<size_t>(token) * q_width + head * dim : row + head * key_head_stride;
+            for (int within = lane; within < per_head; within += 32) {
+                if (within < half) {
+                    const int first = within, second = within + half;
+                    float u = to_float(from[first]) * inverse, w = to_float(from[second]) * inverse;
+                    if (weight) {
+                        u *= weight[head * dim + first];
+                        w *= weight[head * dim + second];
+                    }
+                    const float2 turn = turns[within];
+                    const float a = u * turn.x - w * turn.y, b = w * turn.x + u * turn.y;
+                    if (talk && is_query) {
+                        turned[head * dim + first] = a;
+                        turned[head * dim + second] = b;
+                    } else {
+                        target[first] = from_float<T>(a);
+                        target[second] = from_float<T>(b);
+                    }
+                } else {
+                    const int column = rotary + (within - half);
+                    float u = to_float(from[column]) * inverse;
+                    if (weight) u *= weight[head * dim + column];
+                    if (talk && is_query) turned[head * dim + column] = u;
+                    else target[column] = from_float<T>(u);
+                }
+            }
+        }
+        if (write_rows) {
+            const T* values = source + q_width + k_width;
+            for (int column = threadIdx.x; column < kv_heads * vdim; column += blockDim.x) {
+                T value = values[column];
+                if (first_row) value = from_float<T>((1.0f - share) * to_float(value) + share * to_float(first_row[column]));
+                value_row[(column / vdim) * value_head_stride + column % vdim] = value;
+            }
         }
     }
     if (talk) {      // head h's query for key head j: the queries of j's group, weighed by row h of `talk`; rounded once
         __syncthreads();
         const int group_size = heads / kv_heads, wide = kv_heads * dim;
         T* mixed = queries + static_cast<size_t>(token) * heads * wide;
+        if (dim % kMixColumns == 0) {
+            // A thread takes 8 columns of one key head for a share of the heads, kMixHeads of them at a time.
+            const int pieces = wide / kMixColumns, shares = max(1, static_cast<int>(blockDim.x) / pieces);
+            for (int item = threadIdx.x; item < pieces * shares; item += blockDim.x) {
+                const int piece = item % pieces, group = piece * kMixColumns / dim, column = piece * kMixColumns - group * dim;
+                const float* from = turned + group * group_size * dim + column;
+                for (int head = item / pieces * kMixHeads; head < heads; head += shares * kMixHeads) {
+                    const float* rows_of_talk[kMixHeads];
+                    float sum[kMixHeads][kMixColumns];
+#pragma unroll
+                    for (int i = 0; i < kMixHeads; ++i) {
+                        rows_of_talk[i] = talk + (head + i < heads ? head + i : head) * heads + group * group_size;
+#pragma unroll
+                        for (int e = 0; e < kMixColumns; ++e) sum[i][e] = 0.0f;
+                    }
+                    for (int g = 0; g < group_size; ++g) {
+                        float x[kMixColumns];
+                        load_columns(from + g * dim, x);
+#pragma unroll
+                        for (int i = 0; i < kMixHeads; ++i) {
+                            const float weight = rows_of_talk[i][g];
+#pragma unroll
+                            for (int e = 0; e < kMixColumns; ++e) sum[i][e] = fmaf(weight, x[e], sum[i][e]);
+                        }
+                    }
+#pragma unroll
+                    for (int i = 0; i < kMixHeads; ++i)
+                        if (head + i < heads) store_columns(mixed + static_cast<size_t>(head + i) * wide + piece * kMixColumns, sum[i]);
+                }
+            }
+            return;
+        }
         for (int index = threadIdx.x; index < heads * wide; index += blockDim.x) {
             const int head = index / wide, within = index % wide, group = within / dim, column = within % dim;
             const float* from = turned + group * group_size * dim + column;
@@ -279,6 +389,7 @@ masked_attention_kernel(const T* __restrict__ queries, const T* __restrict__ row
 // context then fill the machine.
 constexpr int kStagedWarps = 4;
 constexpr int kTileKeys = 32;
+constexpr int kMaxSplits = 64;
 
 __device__ __forceinline__ void copy_word(void* target, const void* source) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(target))), "l"(source) : "memory");
@@ -456,26 +567,37 @@ masked_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__
                               int sigmoid_weights, const T* __restrict__ gate, long long gate_stride, int gate_per_head) {
     grid_dependents_launch();
     grid_dependency_wait();
+    __shared__ float factors[kMaxSplits];
     const int token = blockIdx.x, head = blockIdx.y;
     const float* records = partial + (static_cast<size_t>(token) * heads + head) * splits * (vdim + 2);
-    float top = -INFINITY;
-    if (!sigmoid_weights)
-        for (int split = 0; split < splits; ++split) top = fmaxf(top, records[static_cast<size_t>(split) * (vdim + 2) + vdim]);
-    float total = 0.0f;
-    if (!sigmoid_weights)
-        for (int split = 0; split < splits; ++split)
-            total += records[static_cast<size_t>(split) * (vdim + 2) + vdim + 1] * expf(records[static_cast<size_t>(split) * (vdim + 2) + vdim] - top);
-    const float factor = sigmoid_weights ? out_scale : out_scale / total;
+    // The first warp turns the ranges' maxima and denominators into the factors of their sums.
+    if (threadIdx.x < 32) {
+        float tops[kMaxSplits / 32], top = -INFINITY, total = 0.0f;
+#pragma unroll
+        for (int i = 0; i < kMaxSplits / 32; ++i) {
+            const int split = threadIdx.x + 32 * i;
+            tops[i] = (!sigmoid_weights && split < splits) ? records[static_cast<size_t>(split) * (vdim + 2) + vdim] : -INFINITY;
+            top = fmaxf(top, tops[i]);
+        }
+        top = warp_max(top);
+#pragma unroll
+        for (int i = 0; i < kMaxSplits / 32; ++i) {
+            const int split = threadIdx.x + 32 * i;
+            tops[i] = expf(tops[i] - top);                       // a range without keys: exp(-inf) = 0
+            if (!sigmoid_weights && split < splits) total = fmaf(records[static_cast<size_t>(split) * (vdim + 2) + vdim + 1], tops[i], total);
+        }
+        total = warp_sum(total);
+#pragma unroll
+        for (int i = 0; i < kMaxSplits / 32; ++i) factors[threadIdx.x + 32 * i] = sigmoid_weights ? out_scale : tops[i] * (out_scale / total);
+    }
+    __syncthreads();
     const T* gates = gate ? gate + static_cast<size_t>(token) * gate_stride + (gate_per_head ? head : head * vdim) : nullptr;
     for (int column = threadIdx.x; column < vdim; column += blockDim.x) {
         float sum = 0.0f;
-        for (int split = 0; split < splits; ++split) {
-            const float* record = records + static_cast<size_t>(split) * (vdim + 2);
-            sum += sigmoid_weights ? record[column] : record[column] * expf(record[vdim] - top);      // a range without keys: exp(-inf) = 0
-        }
-        float value = sum * factor;
-        if (gates) value /= 1.0f + expf(-to_float(gates[gate_per_head ? 0 : column]));
-        out[static_cast<size_t>(token) * out_stride + head * vdim + column] = from_float<T>(value);
+#pragma unroll 8
+        for (int split = 0; split < splits; ++split) sum = fmaf(records[static_cast<size_t>(split) * (vdim + 2) + column], factors[split], sum);
+        if (gates) sum /= 1.0f + expf(-to_float(gates[gate_per_head ? 0 : column]));
+        out[static_cast<size_t>(token) * out_stride + head * vdim + column] = from_float<T>(sum);
     }
 }
 
@@ -692,7 +814,7 @@ int launch_talking_decode(const void* queries, const void* rows, const void* val
     if (!talk_fits<T>(heads, kv_heads, dim, vdim)) return cudaErrorInvalidValue;
     const TalkPlan plan = talk_plan<T>(heads, kv_heads, dim, vdim);
     const int places = heads * vdim * static_cast<int>(sizeof(T)) / 16, owned = (places + kTalkWarps * 32 - 1) / (kTalkWarps * 32);
-    if (splits > 1 && !partial) return cudaErrorInvalidValue;
+    if ((splits > 1 && !partial) || splits > kMaxSplits) return cudaErrorInvalidValue;
     if (splits <= 1) splits = 1, partial = nullptr;
 #define TAU_TALK(OWNED)                                                                                                                                          \
     {                                                                                                                                                            \
@@ -734,7 +856,7 @@ int launch_staged(int bytes, const void* queries, const void* rows, const void* 
         allowed = 160 * 1024;
     }
     const int group_size = heads / kv_heads, passes = (group_size + kStagedWarps - 1) / kStagedWarps;
-    if (splits > 1 && !partial) return cudaErrorInvalidValue;
+    if ((splits > 1 && !partial) || splits > kMaxSplits) return cudaErrorInvalidValue;
     if (splits <= 1) splits = 1, partial = nullptr;
     tau_launch(masked_attention_staged_kernel<T>, dim3(tokens, kv_heads * passes, splits), dim3(kStagedWarps * 32), bytes, s, static_cast<const T*>(queries),
                static_cast<const T*>(rows), static_cast<const T*>(value_pages), static_cast<T*>(out), out_stride, positions, token_seq, page_rows, page_stride,
@@ -807,7 +929,7 @@ TAU_EXPORT int tau_masked_prepare(int dtype, const void* projected, long long pr
         (rotary && !frequency) || (write_rows && (!rows || !token_seq || !page_rows)) || (talk && heads % kv_heads != 0) || (first_values && !value_share))
         return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    const size_t bytes = static_cast<size_t>(rotary / 2) * sizeof(float2) + (talk ? static_cast<size_t>(heads) * dim * sizeof(float) : 0);
+    const size_t bytes = static_cast<size_t>((rotary / 2 + 1) / 2 * 2) * sizeof(float2) + (talk ? static_cast<size_t>(heads) * dim * sizeof(float) : 0);
     if (bytes > kMaxShared) return cudaErrorInvalidValue;
 #define TAU_PREPARE(T)                                                                                                                            \
     if (bytes > 40 * 1024) {                                                                                                                      \

@@ -275,6 +275,20 @@ def test_mixed_scores_with_a_window_and_kept_positions_over_scattered_pages(dtyp
         assert kernels.attention_prefill_tc_status(dim) == 0
 
 
+@pytest.mark.parametrize("heads, kv_heads, dim, tokens, window, keep_first", [(16, 4, 128, 1500, 600, 70), (32, 8, 64, 1100, 1000, 1), (16, 8, 128, 1300, 64, 200), (24, 1, 128, 1250, 333, 0)])
+def test_long_runs_with_more_tiles_than_the_machine_holds_blocks(heads, kv_heads, dim, tokens, window, keep_first):
+    """Every block of the tensor-core kernel walks several items with odd and even numbers of pages."""
+    generator = torch.Generator().manual_seed(tokens)
+    rounded = lambda t: t.to(torch.bfloat16).double()
+    q, k, v = rounded(rand(generator, tokens, heads, dim)), rounded(rand(generator, tokens, kv_heads, dim)), rounded(rand(generator, tokens, kv_heads, dim))
+    talk = (torch.eye(heads, dtype=F) + 0.5 * rand(generator, heads, heads) / heads ** 0.5).float().double()
+    wanted = plain.talking_attention(q, k, v, dim ** -0.5, talk, plain.visible_keys(tokens, window, keep_first)).reshape(tokens, -1)
+    pages = torch.randperm(-(-tokens // 64), generator=generator).tolist()
+    found = run_attention(q, k, v, dim ** -0.5, talk, window, keep_first, "bfloat16", pages, True, tokens, "tensor")
+    assert kernels.attention_prefill_tc_status(dim) == 0
+    assert relative_error(found, wanted) < 2e-2
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("dim, heads_layout", [(16, False), (64, True), (128, True)])
 @pytest.mark.parametrize("window, keep_first", [(64, 3), (70, 64), (100, 65), (129, 1)])
