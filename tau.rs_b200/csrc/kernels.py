@@ -87,7 +87,7 @@ _CLASS_OF = {
     "moe_combine": "routing", "diff_prepare": "attention", "diff_attention": "attention", "diff_combine": "attention", "causal_taps": "norm", "gated_add_norm": "norm",
     "side_gate": "activation", "unit_add_mix": "norm", "norm_rows": "norm", "relu_squared": "activation",
     "short_conv": "recurrence", "delta_prepare": "recurrence", "delta_rule": "recurrence", "selective_scan": "recurrence",
-    "masked_prepare": "attention", "masked_attention": "attention", "talking_decode": "attention", "gated_rows": "attention",
+    "masked_prepare": "attention", "masked_attention": "attention", "talking_decode": "attention", "shared_key_decode": "attention", "gated_rows": "attention",
     "token_shift": "recurrence", "tanh": "activation", "channel_decay": "recurrence", "wkv": "recurrence", "forget_gates": "recurrence", "turn_heads": "recurrence",
 }
 _timing = None     # while timing: [last event, [(class, event after the launch), ...]]
@@ -1459,6 +1459,41 @@ def talking_decode(queries, rows, talk, out, step, page_rows, n_kv_heads: int, v
         ctypes.c_int(splits), _pointer(partial), _stream()), "talking_decode", 2 if splits > 1 else 1)
 
 
+def shared_key_decode_fits(dtype, n_heads: int, n_kv_heads: int, dim: int, vdim: int) -> bool:
+    """Whether `shared_key_decode` serves these sizes."""
+    if dtype != torch.bfloat16:
+        return False
+    key = ("shared", n_heads, n_kv_heads, dim, vdim)
+    if key not in _talking_fits:
+        library = build.load_library("masked_attention.cu")
+        _talking_fits[key] = bool(library.tau_shared_key_decode_fits(*(ctypes.c_int(value) for value in (n_heads, n_kv_heads, dim, vdim))))
+    return _talking_fits[key]
+
+
+def shared_key_decode(queries, rows, out, step, page_rows, n_kv_heads: int, vdim: int, scale: float, window: int = 0, keep_first: int = 0,
+                      out_scale: float = 1.0, value_pages=None, splits: int = 1) -> None:
+    """Causal softmax attention of single tokens in bfloat16 on the tensor cores (mma.sync) whose queries [tokens, n_heads, n_kv_heads * dim]
+    ask the keys of all key heads side by side (`masked_prepare` with `talk` makes them), over the last `window` positions (0: all) and the
+    sequence's first `keep_first`; cache layouts, `out` and `splits` as for `talking_decode`; where `shared_key_decode_fits`."""
+    _on_device(queries, rows, out, page_rows, value_pages)
+    tokens, n_heads, dim = queries.shape
+    _require(dim % n_kv_heads == 0, "a query against all key heads has a piece for each")
+    dim //= n_kv_heads
+    _require(queries.is_contiguous() and out.shape == (tokens, n_heads * vdim) and out.stride(1) == 1 and out.dtype == queries.dtype == rows.dtype == torch.bfloat16,
+             "queries must be bfloat16 [tokens, n_heads, n_kv_heads * dim] and the output [tokens, n_heads * vdim]")
+    _require_masked_pages(rows, value_pages, queries.dtype, n_kv_heads, dim, vdim)
+    _require(rows.data_ptr() % 16 == 0 and (value_pages is None or value_pages.data_ptr() % 16 == 0), "cache pages must start on 16-byte borders")
+    _require(page_rows.dtype == torch.int32 and page_rows.dim() == 2 and page_rows.is_contiguous(), "page rows must be int32 [sequences, stride]")
+    splits = max(1, min(int(splits), 64))
+    partial = torch.empty((tokens, n_heads, splits, vdim + 2), dtype=torch.float32, device=queries.device) if splits > 1 else None
+    library = build.load_library("masked_attention.cu")
+    _check(library.tau_shared_key_decode(
+        _pointer(queries), _pointer(rows), _pointer(value_pages), _pointer(out), ctypes.c_longlong(out.stride(0)), _pointer(step.positions), _pointer(step.token_seq),
+        _pointer(page_rows), ctypes.c_int(page_rows.shape[1]), ctypes.c_int(PAGE_TOKENS), ctypes.c_int(tokens), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(dim),
+        ctypes.c_int(vdim), ctypes.c_float(scale), ctypes.c_int(window), ctypes.c_int(keep_first), ctypes.c_float(out_scale), ctypes.c_int(splits), _pointer(partial),
+        _stream()), "shared_key_decode", 2 if splits > 1 else 1)
+
+
 def gated_rows(values, gate, out) -> None:
     """`out = values * sigmoid(gate)`, element by element; [rows, width] of one dtype, rows any distance apart; `out` may be `values`."""
     _on_device(values, gate, out)
@@ -1518,7 +1553,8 @@ def wkv(r, k, v, w, per_head, state, cu_seqlens, seq_slot, out, n_heads: int, ke
     `"forget_writes"`: `S <- diag(w) S + (1 - w) v^T`, then `o = S^T r` (no `k`, no `per_head`);
     `"constant_decay"`: `S <- d S + k v^T`, then `o = S^T r` (no `w`; `per_head` float32 [n_heads], the decays).
     `r`, `k`, `w` float32 [tokens, n_heads * key_dim] (rows one distance apart), `v` float32 [tokens, n_heads * value_dim] (rows any
-    distance apart), `out` the same and contiguous, `state` float32 [slots, n_heads * value_dim * key_dim], updated in place."""
+    distance apart), `out` the same and contiguous, `state` float32 [slots, n_heads * value_dim * key_dim], updated in place.  Every sequence
+    brings at least one token."""
     _require(form in WALK_FORMS, f"unknown form {form!r}")
     _on_device(r, k, v, w, per_head, state, cu_seqlens, seq_slot, out)
     _require((k is not None) == (form != "forget_writes") and (w is not None) == (form != "constant_decay") and (per_head is not None) == (form != "forget_writes"),
@@ -1544,7 +1580,7 @@ def wkv(r, k, v, w, per_head, state, cu_seqlens, seq_slot, out, n_heads: int, ke
     library = build.load_library("wkv.cu", (f"TAU_KEY_DIM={key_dim}",))
     _check(library.tau_wkv(ctypes.c_int(WALK_FORMS[form]), _pointer(r), _pointer(k), _pointer(v), _pointer(w), ctypes.c_longlong(r.stride(0)), ctypes.c_longlong(v.stride(0)),
                            _pointer(per_head), _pointer(state), ctypes.c_longlong(state.stride(0)), _pointer(cu_seqlens), _pointer(seq_slot), _pointer(out), ctypes.c_int(n_seqs),
-                           ctypes.c_int(n_heads), ctypes.c_int(value_dim), _stream()), "wkv")
+                           ctypes.c_int(tokens), ctypes.c_int(n_heads), ctypes.c_int(value_dim), _stream()), "wkv")
 
 
 def forget_gates(rows, query_offset: int, gate_offset: int, lower) -> None:

@@ -29,7 +29,7 @@
 namespace {
 
 constexpr int kWarps = 8;
-constexpr int kMaxShared = 200 * 1024;      // dynamic shared memory that a block of these kernels may ask for
+constexpr int kMaxShared = 224 * 1024;      // dynamic shared memory that a block of these kernels may ask for
 constexpr int kMaxOwned = 16;     // value columns per lane: vdim <= 512
 
 // The keys that a query sees, numbered 0 .. count - 1: the kept first positions that lie before its window (or chunk), then the window's.
@@ -835,6 +835,222 @@ int launch_talking_decode(const void* queries, const void* rows, const void* val
     return tau_launch_status();
 }
 
+// ---- single tokens in bfloat16 against the keys of all key heads side by side ------------------------------------------------------
+//
+// The mixed queries of a token (prepare's, one piece for each key head) are a matrix of `heads` rows and kv_heads * dim columns, and every row
+// asks the same keys: a product for the tensor cores whose rows are the heads.  grid: (tokens, splits); block: kSharedWarps warps.  A tile is
+// kKeys positions, keys and values of all key/value heads, by cp.async (the values' copies run on beside the scores):
+//   scores    a warp takes 16 heads and 8 keys: mma.sync m16n8k16 over all key heads' elements, operands by ldmatrix;
+//   weights   a warp takes a head: mask, running maximum, weights (rounded to bfloat16 as the second product's operand) and their 32-bit sum;
+//   values    an item is 16 heads of one value head's group (rows beyond the group are not kept) and 8 of its columns: mma.sync over the keys.
+// Scores, weights and sums in 32-bit; accumulators in registers, kItems items to a warp.  `splits` > 1: joined by `masked_attention_merge_kernel`.
+constexpr int kSharedWarps = 8;
+
+struct SharedPlan {
+    int keys, items;                                             // positions of a tile, items of a warp; keys = 0: not served
+    int head_rows, query_stride, key_stride, value_stride;       // rows of 16-head tiles; bytes of a staged row
+    int key_offset, value_offset, score_offset, weight_offset, stat_offset, total;
+};
+__host__ __device__ inline int odd_units(int bytes) { return ((bytes / 16) | 1) * 16; }      // rows an odd number of 16-byte units apart: no bank conflicts
+__host__ __device__ inline SharedPlan shared_plan(int heads, int kv_heads, int dim, int vdim, int keys) {
+    SharedPlan plan = {};
+    const int wide = kv_heads * dim, group_tiles = (heads / kv_heads + 15) / 16;
+    if (dim % 8 != 0 || vdim % 8 != 0 || wide % 32 != 0 || heads > 256) return plan;
+    plan.items = (kv_heads * group_tiles * (vdim / 8) + kSharedWarps - 1) / kSharedWarps;
+    plan.head_rows = (heads + 15) / 16 * 16;
+    plan.query_stride = odd_units(wide * 2), plan.key_stride = plan.query_stride, plan.value_stride = odd_units(kv_heads * vdim * 2);
+    const long long query = static_cast<long long>(plan.head_rows) * plan.query_stride, key = static_cast<long long>(keys) * plan.key_stride;
+    const long long value = static_cast<long long>(keys) * plan.value_stride, score = static_cast<long long>(plan.head_rows) * (keys + 4) * 4;
+    const long long weight = static_cast<long long>(plan.head_rows + 16) * (keys + 8) * 2, total = query + key + value + score + weight + 3LL * plan.head_rows * 4;
+    if (total > kMaxShared || plan.items > 16) return plan;
+    plan.key_offset = static_cast<int>(query), plan.value_offset = static_cast<int>(query + key), plan.score_offset = static_cast<int>(query + key + value);
+    plan.weight_offset = plan.score_offset + static_cast<int>(score), plan.stat_offset = plan.weight_offset + static_cast<int>(weight);
+    plan.total = static_cast<int>(total);
+    plan.keys = keys;
+    return plan;
+}
+
+__device__ __forceinline__ void load_matrices(uint32_t (&r)[4], uint32_t address) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(address) : "memory");
+}
+__device__ __forceinline__ void load_matrices_transposed(uint32_t (&r)[4], uint32_t address) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(address) : "memory");
+}
+__device__ __forceinline__ void multiply_add(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+template <int kKeys, int kItems>
+__global__ void __launch_bounds__(kSharedWarps * 32)
+shared_key_decode_kernel(const bf16* __restrict__ queries, const bf16* __restrict__ rows, const bf16* __restrict__ value_pages, bf16* __restrict__ out,
+                         long long out_stride, const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ page_rows,
+                         int page_stride, int page_tokens, int heads, int kv_heads, int dim, int vdim, float scale, int window, int keep_first, float out_scale,
+                         int splits, float* __restrict__ partial) {
+    grid_dependents_launch();
+    constexpr int kThreads = kSharedWarps * 32, kScoreStride = kKeys + 4, kWeightStride = kKeys + 8;
+    extern __shared__ __align__(16) uint8_t shared_bytes[];
+    const SharedPlan plan = shared_plan(heads, kv_heads, dim, vdim, kKeys);
+    float* scores = reinterpret_cast<float*>(shared_bytes + plan.score_offset);        // [head_rows][kScoreStride]
+    bf16* weights = reinterpret_cast<bf16*>(shared_bytes + plan.weight_offset);         // [head_rows + 16][kWeightStride]
+    float* tops = reinterpret_cast<float*>(shared_bytes + plan.stat_offset);            // running maxima, sums, the last rescaling
+    float* sums = tops + plan.head_rows;
+    float* rescale = sums + plan.head_rows;
+    const uint32_t base = static_cast<uint32_t>(__cvta_generic_to_shared(shared_bytes));
+    const int token = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, matrix = lane >> 3, matrix_row = lane & 7;
+    const int wide = kv_heads * dim, key_pieces = wide / 8, value_pieces = kv_heads * vdim / 8;      // 16-byte pieces of a position
+    for (int head = threadIdx.x; head < plan.head_rows; head += kThreads) tops[head] = -INFINITY, sums[head] = 0.0f, rescale[head] = 0.0f;
+    grid_dependency_wait();
+    const int position = positions[token];
+    const int* pages = page_rows + static_cast<size_t>(token_seq[token]) * page_stride;
+    const Visible seen = visible_keys(position, window, 0, keep_first);
+    const int all_tiles = (seen.count - 1) / kKeys + 1;
+    const int per_split = (all_tiles + splits - 1) / splits, tile_begin = static_cast<int>(blockIdx.y) * per_split;
+    const int n_tiles = all_tiles - tile_begin < per_split ? (all_tiles - tile_begin > 0 ? all_tiles - tile_begin : 0) : per_split;
+    // Rows of keys or of values of a tile: a warp brings rows warp, warp + kSharedWarps, ...; lane n knows where the n-th of them lies (`place`,
+    // in positions of the cache; -1 behind the tile's last one, where zeros go: the weights there are zero, what lies there is not known).
+    auto stage = [&](long long place, bool is_key) {
+        const int pieces = is_key ? key_pieces : value_pieces, size = is_key ? dim : vdim, per_head = size / 8;
+        uint8_t* buffer = shared_bytes + (is_key ? plan.key_offset : plan.value_offset);
+        const int stride = is_key ? plan.key_stride : plan.value_stride;
+        const bf16* source = value_pages && !is_key ? value_pages : rows + (value_pages || is_key ? 0 : wide);
+        const long long row_width = value_pages ? size : static_cast<long long>(wide) + kv_heads * vdim;
+        for (int first = 0; first < pieces; first += 32) {
+            const int piece = first + lane, head = piece / per_head;
+            const bf16* from = source + (value_pages ? static_cast<long long>(head) * page_tokens * size + (piece - head * per_head) * 8 : piece * 8LL);
+            uint8_t* target = buffer + warp * stride + piece * 16;
+#pragma unroll
+            for (int n = 0; n < kKeys / kSharedWarps; ++n) {
+                const long long at = __shfl_sync(0xffffffffu, place, n);
+                if (piece < pieces) {
+                    if (at >= 0) copy_16(target + n * kSharedWarps * stride, from + at * row_width);
+                    else *reinterpret_cast<uint4*>(target + n * kSharedWarps * stride) = make_uint4(0u, 0u, 0u, 0u);
+                }
+            }
+        }
+        copy_commit();
+    };
+    // The token's queries, with the first tile's keys.
+    for (int head = warp; head < heads; head += kSharedWarps)
+        for (int piece = lane; piece < key_pieces; piece += 32)
+            copy_16(shared_bytes + head * plan.query_stride + piece * 16, queries + (static_cast<size_t>(token) * heads + head) * wide + piece * 8);
+    float acc[kItems][4];
+#pragma unroll
+    for (int i = 0; i < kItems; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[i][e] = 0.0f;
+    const int group_size = heads / kv_heads, group_tiles = (group_size + 15) / 16, columns = vdim / 8, items = kv_heads * group_tiles * columns;
+    for (int tile = 0; tile < n_tiles; ++tile) {
+        const int base_number = (tile_begin + tile) * kKeys;
+        const int count = seen.count - base_number < kKeys ? seen.count - base_number : kKeys;
+        const int row = warp + kSharedWarps * lane;
+        long long place = -1;
+        if (lane < kKeys / kSharedWarps && row < count) {
+            const int key = seen.key(base_number + row);
+            place = static_cast<long long>(pages[key / page_tokens]) * (value_pages ? kv_heads : 1) * page_tokens + key % page_tokens;
+        }
+        stage(place, true);
+        stage(place, false);
+        copy_wait<1>();
+        __syncthreads();     // the keys (and the queries) have arrived for everybody
+        for (int item = warp; item < plan.head_rows / 16 * (kKeys / 8); item += kSharedWarps) {
+            const int head0 = item / (kKeys / 8) * 16, key0 = item % (kKeys / 8) * 8;
+            const uint32_t a_address = base + (head0 + matrix_row + (matrix & 1) * 8) * plan.query_stride + (matrix >> 1) * 16;
+            const uint32_t b_address = base + plan.key_offset + (key0 + matrix_row) * plan.key_stride + matrix * 16;
+            float c[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
+#pragma unroll 4
+            for (int k = 0; k < wide; k += 32) {
+                uint32_t a0[4], a1[4], b[4];
+                load_matrices(b, b_address + k * 2);
+                load_matrices(a0, a_address + k * 2);
+                load_matrices(a1, a_address + k * 2 + 32);
+                multiply_add(c[0], a0, b[0], b[1]);
+                multiply_add(c[1], a1, b[2], b[3]);
+            }
+            float* target = scores + (head0 + (lane >> 2)) * kScoreStride + key0 + (lane & 3) * 2;
+            target[0] = c[0][0] + c[1][0], target[1] = c[0][1] + c[1][1];
+            target[8 * kScoreStride] = c[0][2] + c[1][2], target[8 * kScoreStride + 1] = c[0][3] + c[1][3];
+        }
+        __syncthreads();
+        for (int head = warp; head < heads; head += kSharedWarps) {
+            float value[kKeys / 32], tile_top = -INFINITY, total = 0.0f;
+#pragma unroll
+            for (int i = 0; i < kKeys / 32; ++i) {
+                const int key = lane + 32 * i;
+                value[i] = key < count ? scores[head * kScoreStride + key] * scale : -INFINITY;
+                tile_top = fmaxf(tile_top, value[i]);
+            }
+            const float top = tops[head], new_top = fmaxf(top, warp_max(tile_top));
+#pragma unroll
+            for (int i = 0; i < kKeys / 32; ++i) {
+                const float p = expf(value[i] - new_top);      // exp(-inf) = 0 behind the last key
+                total += p;
+                weights[head * kWeightStride + lane + 32 * i] = __float2bfloat16_rn(p);
+            }
+            total = warp_sum(total);      // every lane has read the maximum by now
+            if (lane == 0) {
+                const float keep = expf(top - new_top);
+                tops[head] = new_top, sums[head] = sums[head] * keep + total, rescale[head] = keep;
+            }
+        }
+        copy_wait<0>();
+        __syncthreads();     // weights and values are there
+#pragma unroll
+        for (int i = 0; i < kItems; ++i) {
+            const int item = warp + i * kSharedWarps;
+            if (item < items) {
+                const int column = item % columns, group_tile = item / columns, group = group_tile / group_tiles;
+                const int head0 = group * group_size + group_tile % group_tiles * 16, end = (group + 1) * group_size;
+                const int low = head0 + (lane >> 2), high = low + 8;
+                const float keep_low = low < end ? rescale[low] : 0.0f, keep_high = high < end ? rescale[high] : 0.0f;
+                acc[i][0] *= keep_low, acc[i][1] *= keep_low, acc[i][2] *= keep_high, acc[i][3] *= keep_high;
+                const uint32_t a_address = base + plan.weight_offset + ((head0 + matrix_row + (matrix & 1) * 8) * kWeightStride + (matrix >> 1) * 8) * 2;
+                const uint32_t b_address = base + plan.value_offset + lane * plan.value_stride + (group * vdim + column * 8) * 2;
+#pragma unroll
+                for (int k = 0; k < kKeys; k += 32) {
+                    uint32_t a0[4], a1[4], b[4];
+                    load_matrices(a0, a_address + k * 2);
+                    load_matrices(a1, a_address + k * 2 + 32);
+                    load_matrices_transposed(b, b_address + k * plan.value_stride);
+                    multiply_add(acc[i], a0, b[0], b[1]);
+                    multiply_add(acc[i], a1, b[2], b[3]);
+                }
+            }
+        }
+        __syncthreads();     // the tile's place may be written over
+    }
+    copy_commit();       // (a block whose range is empty has asked for the queries alone)
+    copy_wait<0>();
+#pragma unroll
+    for (int i = 0; i < kItems; ++i) {
+        const int item = warp + i * kSharedWarps;
+        if (item >= items) continue;
+        const int column = item % columns, group_tile = item / columns, group = group_tile / group_tiles;
+        const int head0 = group * group_size + group_tile % group_tiles * 16, end = (group + 1) * group_size;
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int head = head0 + (lane >> 2) + half * 8, within = column * 8 + (lane & 3) * 2;
+            if (head >= end) continue;
+            if (partial) {
+                float* record = partial + ((static_cast<size_t>(token) * heads + head) * splits + blockIdx.y) * (vdim + 2);
+                record[within] = acc[i][2 * half], record[within + 1] = acc[i][2 * half + 1];
+                if (within == 0) record[vdim] = tops[head], record[vdim + 1] = sums[head];
+            } else {
+                const float factor = out_scale / sums[head];
+                bf16* target = out + static_cast<size_t>(token) * out_stride + head * vdim + within;
+                target[0] = __float2bfloat16_rn(acc[i][2 * half] * factor), target[1] = __float2bfloat16_rn(acc[i][2 * half + 1] * factor);
+            }
+        }
+    }
+}
+
+SharedPlan choose_shared_plan(int heads, int kv_heads, int dim, int vdim) {
+    if (heads <= 0 || kv_heads <= 0 || dim <= 0 || vdim <= 0 || heads % kv_heads != 0 || static_cast<long long>(kv_heads) * (dim + vdim) > 65536) return SharedPlan{};
+    const SharedPlan wide = shared_plan(heads, kv_heads, dim, vdim, 64);
+    return wide.keys ? wide : shared_plan(heads, kv_heads, dim, vdim, 32);
+}
+
 // Shared memory of the staged kernel, or 0 where it does not serve these sizes.
 template <typename T>
 int staged_bytes(int dim, int vdim) {
@@ -882,6 +1098,43 @@ sigmoid_gate_kernel(const T* __restrict__ values, long long values_stride, const
 }
 
 }  // namespace
+
+// 1 where `tau_shared_key_decode` (bfloat16) serves these sizes.
+TAU_EXPORT int tau_shared_key_decode_fits(int heads, int kv_heads, int dim, int vdim) { return choose_shared_plan(heads, kv_heads, dim, vdim).keys > 0; }
+
+// Single tokens in bfloat16: queries [tokens, heads, kv_heads * dim] as prepare leaves them with `talk`; the cache in either layout.
+TAU_EXPORT int tau_shared_key_decode(const void* queries, const void* rows, const void* value_pages, void* out, long long out_stride, const int* positions,
+                                     const int* token_seq, const int* page_rows, int page_stride, int page_tokens, int tokens, int heads, int kv_heads, int dim,
+                                     int vdim, float scale, int window, int keep_first, float out_scale, int splits, float* partial, void* stream) {
+    if (tokens <= 0) return 0;
+    const SharedPlan plan = choose_shared_plan(heads, kv_heads, dim, vdim);
+    if (!queries || !rows || !out || !positions || !token_seq || !page_rows || window < 0 || keep_first < 0 || page_tokens <= 0 || plan.keys == 0 ||
+        (splits > 1 && !partial) || splits > kMaxSplits)
+        return cudaErrorInvalidValue;
+    if (splits <= 1) splits = 1, partial = nullptr;
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+#define TAU_SHARED(KEYS, ITEMS)                                                                                                                                     \
+    {                                                                                                                                                               \
+        const cudaError_t status = cudaFuncSetAttribute(shared_key_decode_kernel<KEYS, ITEMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMaxShared);             \
+        if (status != cudaSuccess) return static_cast<int>(status);                                                                                                 \
+        tau_launch(shared_key_decode_kernel<KEYS, ITEMS>, dim3(tokens, splits), dim3(kSharedWarps * 32), plan.total, s, static_cast<const bf16*>(queries),           \
+                   static_cast<const bf16*>(rows), static_cast<const bf16*>(value_pages), static_cast<bf16*>(out), out_stride, positions, token_seq, page_rows,     \
+                   page_stride, page_tokens, heads, kv_heads, dim, vdim, scale, window, keep_first, out_scale, splits, partial);                                     \
+    }
+    if (plan.keys == 64) {
+        if (plan.items <= 8) TAU_SHARED(64, 8)
+        else TAU_SHARED(64, 16)
+    } else {
+        if (plan.items <= 8) TAU_SHARED(32, 8)
+        else TAU_SHARED(32, 16)
+    }
+#undef TAU_SHARED
+    const int status = tau_launch_status();
+    if (status != 0 || !partial) return status;
+    tau_launch(masked_attention_merge_kernel<bf16>, dim3(tokens, heads), dim3(128), 0, s, partial, static_cast<bf16*>(out), out_stride, heads, vdim, splits, out_scale, 0,
+               static_cast<const bf16*>(nullptr), 0LL, 0);
+    return tau_launch_status();
+}
 
 // 1 where `tau_talking_decode` serves these sizes.
 TAU_EXPORT int tau_talking_decode_fits(int dtype, int heads, int kv_heads, int dim, int vdim) {

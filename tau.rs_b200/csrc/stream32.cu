@@ -209,8 +209,8 @@ gated_group_norm_kernel(const float* __restrict__ values, const float* __restric
     const int width = groups * group_width;
     const float* source = values + static_cast<size_t>(row) * width;
     __shared__ float scratch[33];
-    if (groups >= warps) {       // many groups: a warp takes a group at a time
-        for (int group = warp; group < groups; group += warps) {
+    if (groups >= warps || gridDim.y > 1) {       // many groups: a warp takes a group at a time (of the row's share of this block)
+        for (int group = blockIdx.y * warps + warp; group < groups; group += warps * gridDim.y) {
             float inverse = 1.0f;
             if (normalize) {
                 float squares = 0.0f;
@@ -319,9 +319,12 @@ TAU_EXPORT int tau_gated_group_norm(int dtype, const float* values, const float*
     if (rows <= 0) return 0;
     if (!values || !out || groups <= 0 || group_width <= 0) return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    const int threads = 256;
-    if (dtype == TAU_F32) tau_launch(gated_group_norm_kernel<float>, dim3(rows), dim3(threads), 0, s, values, weight, gate, gate_dtype, gate_stride, static_cast<float*>(out), out_stride, groups, group_width, eps, normalize, silu_gate);
-    else if (dtype == TAU_BF16) tau_launch(gated_group_norm_kernel<bf16>, dim3(rows), dim3(threads), 0, s, values, weight, gate, gate_dtype, gate_stride, static_cast<bf16*>(out), out_stride, groups, group_width, eps, normalize, silu_gate);
+    // Few rows of many groups: a warp to a group, two warps to a block, so that a row's groups meet as many SMs as they can.
+    const bool spread = groups > 1 && rows * 4 <= 148 * 2 && group_width <= 1024;
+    const int threads = spread ? 64 : 256;
+    const dim3 grid(rows, spread ? (groups + 1) / 2 : 1);
+    if (dtype == TAU_F32) tau_launch(gated_group_norm_kernel<float>, grid, dim3(threads), 0, s, values, weight, gate, gate_dtype, gate_stride, static_cast<float*>(out), out_stride, groups, group_width, eps, normalize, silu_gate);
+    else if (dtype == TAU_BF16) tau_launch(gated_group_norm_kernel<bf16>, grid, dim3(threads), 0, s, values, weight, gate, gate_dtype, gate_stride, static_cast<bf16*>(out), out_stride, groups, group_width, eps, normalize, silu_gate);
     else return cudaErrorInvalidValue;
     return tau_launch_status();
 }

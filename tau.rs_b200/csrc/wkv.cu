@@ -15,6 +15,8 @@
 //   walk:    one block owns (sequence, head, tile of value columns) and walks the run's tokens in order, the next tokens' r, k, w and
 //            values on their way into shared memory meanwhile (cp.async).  A column of S is shared by kSplit threads with kRows key
 //            rows each in registers; a token costs one pass over the rows, and the threads of a column meet once in four tokens (two for very wide keys).
+//   step:    where every sequence brings one token nothing is left to walk, and reading and writing the state is all there is: a warp holds
+//            the token's r, k, w in registers and takes columns of S, whole lines at a time, several on their way at once.
 //
 // The state is 32-bit and lives in the cache, [heads, value_dim, key_dim] per slot.  TAU_KEY_DIM fixes key_dim.
 #include "common.cuh"
@@ -195,6 +197,79 @@ wkv_kernel(const float* __restrict__ r, const float* __restrict__ k, const float
     }
 }
 
+// One token per sequence.  grid (heads, sequences, blocks of columns); a warp's lanes share a column's rows, kWide neighbouring ones each, and a
+// warp takes kTogether columns at a time.
+constexpr int kWide = kDim % 128 == 0 ? 4 : kDim % 64 == 0 ? 2 : 1;
+constexpr int kPieces = (kDim + 32 * kWide - 1) / (32 * kWide);
+constexpr int kStepWarps = 8;
+constexpr int kTogether = kWide * kPieces <= 4 ? 4 : kWide * kPieces <= 8 ? 2 : 1;
+
+template <int kForm>
+__global__ void __launch_bounds__(kStepWarps * 32)
+wkv_step_kernel(const float* __restrict__ r, const float* __restrict__ k, const float* __restrict__ v, const float* __restrict__ w, long long key_stride,
+                long long value_stride, const float* __restrict__ per_head, float* __restrict__ state, long long slot_stride, const int* __restrict__ cu_seqlens,
+                const int* __restrict__ seq_slot, float* __restrict__ out, int heads, int value_dim) {
+    grid_dependents_launch();
+    grid_dependency_wait();
+    const int head = blockIdx.x, sequence = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const size_t token = cu_seqlens[sequence];
+    float* records = state + static_cast<size_t>(seq_slot[sequence]) * slot_stride + static_cast<size_t>(head) * value_dim * kDim;
+    const int first = (blockIdx.z * kStepWarps + warp) * kTogether;
+    if (first >= value_dim) return;
+    __align__(16) float S[kTogether][kPieces][kWide];
+    float value[kTogether];
+    auto row_of = [&](int piece) { return (piece * 32 + lane) * kWide; };      // kWide divides kDim: a piece is inside or outside as a whole
+#pragma unroll
+    for (int c = 0; c < kTogether; ++c) {
+        const int column = first + c < value_dim ? first + c : first;
+        value[c] = v[token * value_stride + head * value_dim + column];
+#pragma unroll
+        for (int p = 0; p < kPieces; ++p)
+            if (row_of(p) < kDim) {
+                const float* source = records + static_cast<size_t>(column) * kDim + row_of(p);
+                if (kWide == 4) *reinterpret_cast<float4*>(S[c][p]) = *reinterpret_cast<const float4*>(source);
+                else
+#pragma unroll
+                    for (int e = 0; e < kWide; ++e) S[c][p][e] = source[e];
+            }
+    }
+    float sums[kTogether];
+#pragma unroll
+    for (int c = 0; c < kTogether; ++c) sums[c] = 0.0f;
+#pragma unroll
+    for (int p = 0; p < kPieces; ++p) {
+        if (row_of(p) >= kDim) continue;
+#pragma unroll
+        for (int e = 0; e < kWide; ++e) {
+            const size_t at = token * key_stride + head * kDim + row_of(p) + e;
+            const float read = r[at], keep = kForm == kConstantDecay ? per_head[head] : w[at], key = kForm == kForgetWrites ? 1.0f - keep : k[at];
+            const float own = kForm == kBonus ? per_head[static_cast<size_t>(head) * kDim + row_of(p) + e] : 0.0f;
+#pragma unroll
+            for (int c = 0; c < kTogether; ++c) {
+                const float write = key * value[c];
+                if (kForm == kBonus) sums[c] = fmaf(fmaf(own, write, S[c][p][e]), read, sums[c]);
+                S[c][p][e] = fmaf(keep, S[c][p][e], write);
+                if (kForm != kBonus) sums[c] = fmaf(S[c][p][e], read, sums[c]);
+            }
+        }
+    }
+#pragma unroll
+    for (int c = 0; c < kTogether; ++c) {
+        const float sum = warp_sum(sums[c]);
+        if (first + c >= value_dim) break;
+        if (lane == 0) out[(token * heads + head) * value_dim + first + c] = sum;
+#pragma unroll
+        for (int p = 0; p < kPieces; ++p)
+            if (row_of(p) < kDim) {
+                float* target = records + static_cast<size_t>(first + c) * kDim + row_of(p);
+                if (kWide == 4) *reinterpret_cast<float4*>(target) = *reinterpret_cast<const float4*>(S[c][p]);
+                else
+#pragma unroll
+                    for (int e = 0; e < kWide; ++e) target[e] = S[c][p][e];
+            }
+    }
+}
+
 }  // namespace
 
 TAU_EXPORT int tau_wkv_key_dim() { return kDim; }
@@ -243,14 +318,24 @@ TAU_EXPORT int tau_channel_decay(float* values, const float* offset, long long r
     return tau_launch_status();
 }
 
+// `tokens` new tokens of `n_seqs` sequences, at least one of each.
 // state: [heads, value_dim, key_dim] floats per slot, slots `slot_stride` apart.  `form`: 0 with a bonus, 1 forget writes (no k, no
 // `per_head`), 2 constant decay (no w).
 TAU_EXPORT int tau_wkv(int form, const float* r, const float* k, const float* v, const float* w, long long key_stride, long long value_stride,
                        const float* per_head, float* state, long long slot_stride, const int* cu_seqlens, const int* seq_slot, float* out, int n_seqs,
-                       int heads, int value_dim, void* stream) {
+                       int tokens, int heads, int value_dim, void* stream) {
     if (n_seqs <= 0) return 0;
     if (form < kBonus || form > kConstantDecay || !r || (form != kForgetWrites && !k) || !v || (form != kConstantDecay && !w) || (form != kForgetWrites && !per_head) || !state || !cu_seqlens || !seq_slot || !out || heads <= 0 || value_dim <= 0) return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (tokens == n_seqs && slot_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15u) == 0) {      // every sequence brings one token
+        dim3 grid(heads, n_seqs, (value_dim + kStepWarps * kTogether - 1) / (kStepWarps * kTogether)), block(kStepWarps * 32);
+#define TAU_WKV_STEP(FORM) tau_launch(wkv_step_kernel<FORM>, grid, block, 0, s, r, k, v, w, key_stride, value_stride, per_head, state, slot_stride, cu_seqlens, seq_slot, out, heads, value_dim)
+        if (form == kBonus) TAU_WKV_STEP(kBonus);
+        else if (form == kForgetWrites) TAU_WKV_STEP(kForgetWrites);
+        else TAU_WKV_STEP(kConstantDecay);
+#undef TAU_WKV_STEP
+        return tau_launch_status();
+    }
     // Value columns to a block: 32 where that many blocks fill the machine, else 16 (blocks of 8 and 4 columns were slower: every block
     // brings the head's r, k and w for itself, and that, not the walk, is then a block's work).
     int device = 0, sms = 148;

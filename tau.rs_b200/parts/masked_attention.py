@@ -138,13 +138,13 @@ class MaskedAttention(JoinableMixer):
 
     def _splits(self, step) -> int:
         """Ranges that a step of single tokens cuts every context into: as many as fill the machine with the staged kernel's blocks (six
-        to an SM), each at least 64 positions of what a token reads (its window or chunk bounds that), 32 at most.  Any number computes
+        to an SM), each at least 64 positions of what a token reads (its window or chunk bounds that), 32 at most (64 with mixed scores).  Any number computes
         the same sums, so a captured graph that serves other lengths than the one it was captured at stays right."""
         if not step.all_single:
             return 1
         reach = min(step.max_len, (self.spec.window or self.spec.chunk or step.max_len) + self.spec.keep_first)
         if self.spec.talk:      # a block serves all heads, and one or two of them fill an SM
-            return max(1, min(2 * kernels.sm_count() // max(1, step.n_seqs), reach // 64, 32))
+            return max(1, min(2 * kernels.sm_count() // max(1, step.n_seqs), -(-reach // 64), 64))
         return max(1, min(6 * kernels.sm_count() // max(1, step.n_seqs * self.decode_blocks()), reach // 64, 32))
 
     def extra_cache_needs(self):
@@ -183,8 +183,12 @@ class MaskedAttention(JoinableMixer):
                 step.handed_on["values"] = own_values
             else:
                 first_values = step.handed_on["values"]
-        # Single tokens mix scores in the attention kernel; runs of tokens (and sizes that it does not serve) mix queries beforehand.
-        talking = spec.talk and step.all_single and kernels.optimized_preferred() and kernels.talking_decode_fits(projected.dtype, spec.n_heads, spec.n_kv_heads, spec.dim, spec.value_dim)
+        # Mixed queries against the keys of all key heads everywhere but for single tokens of sizes (or a dtype) that only the kernel which
+        # mixes scores serves.
+        sizes = (projected.dtype, spec.n_heads, spec.n_kv_heads, spec.dim, spec.value_dim)
+        single = spec.talk and step.all_single and kernels.optimized_preferred()
+        side_by_side = single and kernels.shared_key_decode_fits(*sizes)
+        talking = single and not side_by_side and kernels.talking_decode_fits(*sizes)
         mixed_queries = spec.talk and not talking
         queries = torch.empty((tokens, spec.n_heads, spec.dim * (spec.n_kv_heads if mixed_queries else 1)), dtype=projected.dtype, device=projected.device)
         options = {}      # what only some models ask of the kernels
@@ -199,6 +203,10 @@ class MaskedAttention(JoinableMixer):
         if talking:
             kernels.talking_decode(queries, keys, self.talk, out, step, pages, spec.n_kv_heads, spec.value_dim, spec.softmax_scale, spec.window or 0, spec.keep_first,
                                    self.out_scale, values, splits=self._splits(step))
+            return
+        if side_by_side:
+            kernels.shared_key_decode(queries, keys, out, step, pages, spec.n_kv_heads, spec.value_dim, spec.softmax_scale, spec.window or 0, spec.keep_first,
+                                      self.out_scale, values, splits=self._splits(step))
             return
         options = {"keep_first": spec.keep_first} if spec.keep_first else {}
         if mixed_queries:

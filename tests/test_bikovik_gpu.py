@@ -224,7 +224,8 @@ def test_a_gate_of_another_dtype_behind_the_norm_per_head(dtype):
 # ---- attention -------------------------------------------------------------------------------------------------------------
 def run_attention(q, k, v, scale, talk, window, keep_first, dtype, page_of, heads_layout, single_from, mode):
     """One sequence: the first `single_from` tokens as one run, the others one by one.  `mode` says how: "kernel" (mixed queries against all
-    key heads, a warp per head), "single" (single tokens through the kernel that mixes scores), "tensor" (runs on the tensor cores)."""
+    key heads, a warp per head), "single" (single tokens through the kernel that mixes scores), "side" (single tokens, mixed queries on the tensor cores), "tensor" (runs on the
+    tensor cores)."""
     tokens, heads, dim = q.shape
     kv_heads, vdim = v.shape[1], v.shape[2]
     kind, n_pages = TORCH[dtype], max(page_of) + 2
@@ -241,6 +242,8 @@ def run_attention(q, k, v, scale, talk, window, keep_first, dtype, page_of, head
                                talk=None if single else talk)
         if single:
             kernels.talking_decode(queries, keys, talk, out[begin:end], step, pages, kv_heads, vdim, scale, window, keep_first, 1.0, values, splits=1 + (begin - single_from) % 5)
+        elif mode == "side" and end - begin == 1:
+            kernels.shared_key_decode(queries, keys, out[begin:end], step, pages, kv_heads, vdim, scale, window, keep_first, 1.0, values, splits=1 + (begin - single_from) % 5)
         elif mode == "tensor" and end - begin > 1:
             kernels.attention_prefill_tc(queries.view(end - begin, -1), keys, values, out[begin:end], as_ints([0, end - begin]), as_ints([begin]), pages, heads, kv_heads, dim,
                                          scale, window, keep_first=keep_first, segmented=True)
@@ -250,7 +253,7 @@ def run_attention(q, k, v, scale, talk, window, keep_first, dtype, page_of, head
 
 
 SIZES = [(4, 2, 16, 24, False), (1, 1, 12, 150, False), (9, 3, 10, 6, False), (6, 1, 96, 96, False), (2, 1, 64, 64, True), (4, 2, 128, 128, True), (5, 5, 8, 16, False),
-         (16, 4, 128, 128, True), (8, 8, 64, 64, True), (20, 4, 32, 48, False), (8, 8, 128, 128, True)]
+         (16, 4, 128, 128, True), (8, 8, 64, 64, True), (20, 4, 32, 48, False), (8, 8, 128, 128, True), (40, 2, 48, 40, False), (18, 6, 16, 8, False)]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -266,6 +269,9 @@ def test_mixed_scores_with_a_window_and_kept_positions_over_scattered_pages(dtyp
     tolerance = 2e-5 if dtype == "float32" else 2e-2
     per = 4 if dtype == "float32" else 8
     modes = ["kernel"] + (["single"] if dim % per == 0 and vdim % per == 0 and kernels.talking_decode_fits(kind, heads, kv_heads, dim, vdim) else [])
+    if kernels.shared_key_decode_fits(kind, heads, kv_heads, dim, vdim):
+        modes.append("side")
+    assert dtype == "float32" or dim % 16 or "side" in modes
     if heads_layout and dtype == "bfloat16":      # (8 key heads of 128: the pieces of the queries travel with the keys)
         modes.append("tensor")
     for mode in modes:
@@ -308,8 +314,8 @@ def test_one_key_that_stands_out_is_seen_exactly_inside_the_window_and_among_the
         v = rand(generator, tokens, kv_heads, dim)
         rounded = v.to(TORCH[dtype]).double()
         edges = [far, far + window - 1, far + window, far + 300]
-        for mode in ["single"] + (["tensor"] if heads_layout and dtype == "bfloat16" else ["kernel"]):
-            single_from = 2 if mode == "single" else tokens
+        for mode in ["single"] + (["side"] if dtype == "bfloat16" else []) + (["tensor"] if heads_layout and dtype == "bfloat16" else ["kernel"]):
+            single_from = 2 if mode in ("single", "side") else tokens
             found = run_attention(q, k, v, 1.0, talk, window, keep_first, dtype, [4, 1, 6, 3, 0, 2], heads_layout, single_from, mode).reshape(tokens, heads, dim)
             for position in edges:
                 if position >= tokens:
