@@ -9,6 +9,7 @@ from .bisudra import BisudraConfig
 from .pegurax import PeguraxConfig
 from .nugolorn import NugolornConfig
 from .bikovik import BikovikConfig
+from .tukulorn import TukulornConfig
 from .specs import (AttentionSpec, BlockSpec, ChannelDecayMemorySpec, DeltaRuleSpec, DenseFeedForwardSpec, DifferentialAttentionSpec, MaskedAttentionSpec, SandwichBlockSpec,
                     ScaledRotationSpec, SelectiveScanSpec, SideBySideSpec, LatentAttentionSpec, LinearRecurrenceSpec, ModelSpec, NormSpec, PairRotationSpec,
                     PositionSpec, RoutedExpertsSpec, ScheduleEntry, SublayerNormBlockSpec, SwiGLUSpec, TokenSideSpec)

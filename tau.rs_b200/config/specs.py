@@ -17,7 +17,8 @@ from typing import Optional, Tuple
 class NormSpec:
     """`kind == "rms_norm"`: `x / sqrt(mean(x^2) + eps) * w`.  `kind == "layer_norm"`: `(x - mean) / sqrt(variance + eps) * w + b`,
     the bias being the tensor `<weight's name><bias_suffix>`.  With `groups` > 1 an RMS norm cuts the row into that many equal
-    consecutive pieces and divides each by its own root mean square (on a residual stream kept in 32-bit).  `kind == "dynamic_tanh"`:
+    consecutive pieces and divides each by its own root mean square (on a residual stream kept in 32-bit).  An RMS norm multiplies by
+    `weight_offset + w` (1 for weights stored around zero).  `kind == "dynamic_tanh"`:
     `tanh(alpha * x) * w + b` with `alpha` the one number `<weight's name>.alpha`, no statistic at all (`eps` is not used), on a residual
     stream kept in 32-bit."""
 
@@ -27,6 +28,7 @@ class NormSpec:
     bias_suffix: str = ".bias"
     bias: bool = True          # a layer norm without a bias has no such tensor
     groups: int = 1
+    weight_offset: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -84,23 +86,27 @@ class PairRotationSpec:
 @dataclass(frozen=True)
 class LatentAttentionSpec:
     """Softmax attention whose keys and values are expanded from a cached latent of `kv_rank` elements per position, with
-    `rot_dim` rotated key elements per position that all heads share, queries through a latent of `q_rank` elements, an
-    optional learned sink per head in the softmax denominator and an optional sigmoid output gate."""
+    `rot_dim` rotated key elements per position that all heads share, queries through a latent of `q_rank` elements (None: straight
+    from the input), an optional learned sink per head in the softmax denominator and an optional sigmoid output gate, one number per
+    element or (`gate_per_head`) per head.  `window` limits how far back a query sees (itself and the `window - 1` positions before
+    it).  `wide_result`: the output projection leaves in 32-bit whatever the run's dtype."""
 
     hidden: int
     n_heads: int
     head_dim: int          # unrotated query/key elements per head
     rot_dim: int           # rotated query/key elements per head (the key's are shared by the heads)
     value_dim: int
-    q_rank: int
+    q_rank: Optional[int]
     kv_rank: int
     softmax_scale: float
-    eps: float             # of the two latent norms
+    eps: float             # of the latent norms
     position: Optional[PairRotationSpec] = None
     sink: bool = True
     gate: bool = True
     window: Optional[int] = None
     kind: str = "latent_attention"
+    gate_per_head: bool = False
+    wide_result: bool = False
 
 
 @dataclass(frozen=True)
@@ -109,9 +115,10 @@ class DifferentialAttentionSpec:
     (laid out head by head as [map 1, map 2]) over one value of `value_dim` elements; a head's result is
     `map 1 - lambda * map 2` with `lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff` (four learned vectors of `dim` elements, one
     number for the layer), divided by its root mean square over `value_dim` (eps inside the root, no weight), times `1 - diff`.
-    Queries and keys pass an RMS norm over `dim` whose weight all heads and maps share, then `position`; `window` limits how far
-    back a query sees (itself and the `window - 1` positions before it); `gate` multiplies the heads by a sigmoid of one more
-    projection of the input before the output projection."""
+    Queries and keys pass an RMS norm over `dim` whose weight all heads and maps share (if `qk_norm`), then `position`; `window` limits
+    how far back a query sees (itself and the `window - 1` positions before it); `gate` multiplies the heads by a sigmoid of one more
+    projection of the input before the output projection.  `bias`: q, k, v and the output projection have biases (`<name>.b`).
+    `temperature` = (coef, every): the query at position p is multiplied by `1 + coef * ln(floor((p + 1) / every) + 1)`."""
 
     hidden: int
     n_heads: int
@@ -125,6 +132,9 @@ class DifferentialAttentionSpec:
     window: Optional[int] = None
     gate: bool = True
     kind: str = "differential_attention"
+    qk_norm: bool = True
+    bias: bool = False
+    temperature: Optional[Tuple[float, int]] = None
 
 
 @dataclass(frozen=True)
@@ -335,7 +345,11 @@ class RoutedExpertsSpec:
     alone).  `router_bias` adds the tensor `<prefix>.router.b` to the logits.  `weigh` says what an expert's weight multiplies:
     its `"output"`, or its `"input"` (the expert then reads `weight * h`).  `shared` is a feed-forward that every token passes; with
     `shared_gate` its output is scaled by the sigmoid of one more projection of the token.  `identity` > 0: the router has that
-    many more outputs, behind the experts', which stand for experts without tensors that return what they read."""
+    many more outputs, behind the experts', which stand for experts without tensors that return what they read.
+
+    `groups` > 1: the experts form that many equal groups of neighbours, a group is ranked by the sum of its two largest choosing
+    scores, and only experts of the best `keep_groups` groups can be chosen.  `scale` multiplies the weights.  `activation`: `"silu"`,
+    or `"clamped"` with `limit` (as in `SwiGLUSpec`)."""
 
     hidden: int
     intermediate: int
@@ -350,13 +364,19 @@ class RoutedExpertsSpec:
     router_bias: bool = False
     weigh: str = "output"
     identity: int = 0
+    groups: int = 1
+    keep_groups: int = 1
+    scale: float = 1.0
+    activation: str = "silu"
+    limit: float = 0.0
 
 
 @dataclass(frozen=True)
 class BlockSpec:
     """One layer: its weight-name prefix, its two parts (the feed-forward may be None in parallel and `"pre_norm_stream"` blocks) and the
     norm before each.  `residual_scale` (parallel blocks): what the two
-    parts return is multiplied by it as it joins the residual stream."""
+    parts return is multiplied by it as it joins the residual stream.  `layer_scale` (`"pre_norm_stream"` blocks): what each part
+    returns is multiplied element by element by a vector of its own (`<prefix>.ls1`, `<prefix>.ls2`) as it joins the stream."""
 
     prefix: str
     mixer: object
@@ -365,6 +385,7 @@ class BlockSpec:
     feed_forward_norm: Optional[NormSpec]
     kind: str = "pre_norm"
     residual_scale: float = 1.0
+    layer_scale: bool = False
 
 
 @dataclass(frozen=True)
@@ -415,7 +436,8 @@ class ScheduleEntry:
     then runs several times with the same weights).  `cache_group` and `cache_layer`
     say where the mixer keeps what it remembers; two entries with the same pair share
     that storage, and an entry with `writes_cache=False` only reads what another entry
-    wrote earlier in the same step.
+    wrote earlier in the same step.  `joins_embedding`: the embedding output (what entered
+    the first run) is added to the residual stream right before this run.
     """
 
     layer: int
@@ -424,6 +446,7 @@ class ScheduleEntry:
     writes_cache: bool = True
     # What the block keeps beside its mixer's cache (`Block.extra_cache_needs()`): (role, cache group, cache layer) for each role.
     extra_cache: Tuple[Tuple[str, str, int], ...] = ()
+    joins_embedding: bool = False
 
 
 @dataclass(frozen=True)

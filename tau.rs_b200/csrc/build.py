@@ -45,7 +45,7 @@ def _build_dir() -> str:
     preferred = os.path.join(_HERE, "_build")
     try:
         os.makedirs(preferred, exist_ok=True)
-        probe = os.path.join(preferred, f".probe-{os.getpid()}")
+        probe = os.path.join(preferred, f".probe-{os.getpid()}-{threading.get_ident()}")
         with open(probe, "w"):
             pass
         os.remove(probe)

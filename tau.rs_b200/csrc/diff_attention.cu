@@ -5,7 +5,9 @@
 // One cached row per position: [kv_heads x (map 1 key | map 2 key) | kv_heads x value], keys normalised and rotated already.
 //
 //   prepare:    per (head, map): q and k divided by their root mean square over `dim` (eps inside the root), times a weight shared
-//               by all heads and maps, the first `rotary` elements turned pair by pair (2i, 2i + 1) by position * inv_freq[i];
+//               by all heads and maps (left as they are without weights), the first `rotary` elements turned pair by pair
+//               (2i, 2i + 1) by position * inv_freq[i]; the query at position p times 1 + coef * ln(floor((p + 1) / every) + 1) if
+//               `every` is not 0;
 //               queries to [tokens, heads, 2, dim], keys and values to the token's row.
 //   attention:  a warp per (token, head): 32 keys at a time, a lane scores one key for both maps, then every lane sums its own
 //               value columns; running maximum and sum per map; scores, weights and sums in 32-bit.
@@ -38,6 +40,22 @@ __device__ __forceinline__ float2 turn_of(const float2* turns, const float* __re
 __device__ __forceinline__ void store_two(float* target, float a, float b) { *reinterpret_cast<float2*>(target) = make_float2(a, b); }
 __device__ __forceinline__ void store_two(bf16* target, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(target) = __floats2bfloat162_rn(a, b); }
 
+// 1 / sqrt(mean of the squares + eps) over `dim` elements, by a warp.
+template <typename T>
+__device__ __forceinline__ float inverse_rms(const T* __restrict__ source, int dim, float eps, int lane) {
+    float squares = 0.0f;
+    for (int column = lane; column < dim; column += 32) {
+        const float value = to_float(source[column]);
+        squares += value * value;
+    }
+    return 1.0f / sqrtf(warp_sum(squares) / static_cast<float>(dim) + eps);
+}
+
+// What the query at `position` is multiplied by.
+__device__ __forceinline__ float query_temperature(float coef, int every, int position) {
+    return every > 0 ? 1.0f + coef * logf(static_cast<float>((position + 1) / every + 1)) : 1.0f;
+}
+
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // grid: tokens; a warp per map.  projected row: [heads * 2 * dim | kv_heads * 2 * dim | kv_heads * vdim | ...].
@@ -46,13 +64,14 @@ __global__ void __launch_bounds__(kWarps * 32)
 diff_prepare_kernel(const T* __restrict__ projected, long long projected_stride, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                     float eps, const float* __restrict__ inv_freq, int rotary, T* __restrict__ queries, T* __restrict__ rows,
                     const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ page_rows, int page_stride,
-                    int page_tokens, int heads, int kv_heads, int dim, int vdim, int write_rows) {
+                    int page_tokens, int heads, int kv_heads, int dim, int vdim, int write_rows, float temperature_coef, int temperature_every) {
     grid_dependents_launch();
     grid_dependency_wait();
     const int token = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int position = positions[token];
     __shared__ float2 turns[kMaxPairs];
     fill_turns(turns, inv_freq, rotary, position);
+    const float query_factor = query_temperature(temperature_coef, temperature_every, position);
     const int row_width = kv_heads * (2 * dim + vdim);
     const T* source_row = projected + static_cast<size_t>(token) * projected_stride;
     T* row = nullptr;
@@ -66,17 +85,12 @@ diff_prepare_kernel(const T* __restrict__ projected, long long projected_stride,
         const T* source = source_row + static_cast<size_t>(map) * dim;      // the key maps follow the query maps in the projected row
         T* target = is_query ? queries + (static_cast<size_t>(token) * q_maps + map) * dim : row + static_cast<size_t>(map - q_maps) * dim;
         const float* weight = is_query ? q_weight : k_weight;
-        float squares = 0.0f;
-        for (int column = lane; column < dim; column += 32) {
-            const float value = to_float(source[column]);
-            squares += value * value;
-        }
-        const float inverse = 1.0f / sqrtf(warp_sum(squares) / static_cast<float>(dim) + eps);
+        const float inverse = (weight ? inverse_rms(source, dim, eps, lane) : 1.0f) * (is_query ? query_factor : 1.0f);
         for (int pair = lane; 2 * pair < dim; pair += 32) {
             const int first = 2 * pair;
             const bool second = first + 1 < dim;
-            float u = to_float(source[first]) * inverse * weight[first];
-            float w = second ? to_float(source[first + 1]) * inverse * weight[first + 1] : 0.0f;
+            float u = to_float(source[first]) * inverse * (weight ? weight[first] : 1.0f);
+            float w = second ? to_float(source[first + 1]) * inverse * (weight ? weight[first + 1] : 1.0f) : 0.0f;
             if (first + 1 < rotary) {
                 const float2 turn = turn_of(turns, inv_freq, pair, position);
                 const float a = u * turn.x - w * turn.y, b = w * turn.x + u * turn.y;
@@ -189,7 +203,7 @@ diff_prepare_wide_kernel(const T* __restrict__ projected, long long projected_st
                          float eps, const float* __restrict__ inv_freq, int rotary, T* __restrict__ queries, T* __restrict__ key_pages,
                          T* __restrict__ value_pages, const int* __restrict__ positions, const int* __restrict__ token_seq,
                          const int* __restrict__ page_rows, int page_stride, int page_tokens, int heads, int kv_heads, int dim, int vdim, int wide,
-                         int write_cache) {
+                         int write_cache, float temperature_coef, int temperature_every) {
     // grid: (tokens, y); the warps of a token's y blocks share out its items: the query maps, then (with `write_cache`) the key
     // maps, then the value heads.  Few tokens get a warp per item, many tokens one block each.
     grid_dependents_launch();
@@ -198,6 +212,7 @@ diff_prepare_wide_kernel(const T* __restrict__ projected, long long projected_st
     const int position = positions[token];
     __shared__ float2 turns[kMaxPairs];
     fill_turns(turns, inv_freq, rotary, position);
+    const float query_factor = query_temperature(temperature_coef, temperature_every, position);
     const int q_maps = heads * 2, maps = q_maps + (write_cache ? kv_heads * 2 : 0), items = maps + (write_cache ? kv_heads * 2 : 0);
     const int per_group = heads / kv_heads;
     const T* source_row = projected + static_cast<size_t>(token) * projected_stride;
@@ -228,16 +243,11 @@ diff_prepare_wide_kernel(const T* __restrict__ projected, long long projected_st
             target = key_pages + page_base + static_cast<size_t>(map - q_maps) * head_pitch;
         }
         const float* weight = is_query ? q_weight : k_weight;
-        float squares = 0.0f;
-        for (int column = lane; column < dim; column += 32) {
-            const float value = to_float(source[column]);
-            squares += value * value;
-        }
-        const float inverse = 1.0f / sqrtf(warp_sum(squares) / static_cast<float>(dim) + eps);
+        const float inverse = (weight ? inverse_rms(source, dim, eps, lane) : 1.0f) * (is_query ? query_factor : 1.0f);
         for (int pair = lane; 2 * pair < wide; pair += 32) {
             const int first = 2 * pair;
-            float u = first < dim ? to_float(source[first]) * inverse * weight[first] : 0.0f;
-            float w = first + 1 < dim ? to_float(source[first + 1]) * inverse * weight[first + 1] : 0.0f;
+            float u = first < dim ? to_float(source[first]) * inverse * (weight ? weight[first] : 1.0f) : 0.0f;
+            float w = first + 1 < dim ? to_float(source[first + 1]) * inverse * (weight ? weight[first + 1] : 1.0f) : 0.0f;
             if (first + 1 < rotary) {
                 const float2 turn = turn_of(turns, inv_freq, pair, position);
                 const float a = u * turn.x - w * turn.y, b = w * turn.x + u * turn.y;
@@ -315,9 +325,9 @@ diff_combine_kernel(const T* __restrict__ attended, const T* __restrict__ gate, 
 TAU_EXPORT int tau_diff_prepare_wide(int dtype, const void* projected, long long projected_stride, const float* q_weight, const float* k_weight, float eps,
                                      const float* inv_freq, int rotary, void* queries, void* key_pages, void* value_pages, const int* positions,
                                      const int* token_seq, const int* page_rows, int page_stride, int page_tokens, int tokens, int heads, int kv_heads,
-                                     int dim, int vdim, int wide, int write_cache, void* stream) {
+                                     int dim, int vdim, int wide, int write_cache, float temperature_coef, int temperature_every, void* stream) {
     if (tokens <= 0) return 0;
-    if (!projected || !q_weight || !k_weight || !queries || !positions || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || dim <= 0 || vdim <= 0
+    if (!projected || !q_weight != !k_weight || temperature_every < 0 || !queries || !positions || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || dim <= 0 || vdim <= 0
         || wide < dim || wide < vdim || (wide & 1) || rotary < 0 || rotary > dim || (rotary & 1) || (rotary > 0 && !inv_freq)
         || (write_cache && (!key_pages || !value_pages || !token_seq || !page_rows)))
         return cudaErrorInvalidValue;
@@ -327,11 +337,11 @@ TAU_EXPORT int tau_diff_prepare_wide(int dtype, const void* projected, long long
     if (dtype == TAU_F32)
         tau_launch(diff_prepare_wide_kernel<float>, grid, dim3(kWarps * 32), 0, s, static_cast<const float*>(projected), projected_stride, q_weight,
                    k_weight, eps, inv_freq, rotary, static_cast<float*>(queries), static_cast<float*>(key_pages), static_cast<float*>(value_pages), positions,
-                   token_seq, page_rows, page_stride, page_tokens, heads, kv_heads, dim, vdim, wide, write_cache);
+                   token_seq, page_rows, page_stride, page_tokens, heads, kv_heads, dim, vdim, wide, write_cache, temperature_coef, temperature_every);
     else if (dtype == TAU_BF16)
         tau_launch(diff_prepare_wide_kernel<bf16>, grid, dim3(kWarps * 32), 0, s, static_cast<const bf16*>(projected), projected_stride, q_weight,
                    k_weight, eps, inv_freq, rotary, static_cast<bf16*>(queries), static_cast<bf16*>(key_pages), static_cast<bf16*>(value_pages), positions,
-                   token_seq, page_rows, page_stride, page_tokens, heads, kv_heads, dim, vdim, wide, write_cache);
+                   token_seq, page_rows, page_stride, page_tokens, heads, kv_heads, dim, vdim, wide, write_cache, temperature_coef, temperature_every);
     else
         return cudaErrorInvalidValue;
     return tau_launch_status();
@@ -360,20 +370,20 @@ TAU_EXPORT int tau_diff_combine(int dtype, const void* attended, const void* gat
 TAU_EXPORT int tau_diff_prepare(int dtype, const void* projected, long long projected_stride, const float* q_weight, const float* k_weight, float eps,
                                 const float* inv_freq, int rotary, void* queries, void* rows, const int* positions, const int* token_seq,
                                 const int* page_rows, int page_stride, int page_tokens, int tokens, int heads, int kv_heads, int dim, int vdim,
-                                int write_rows, void* stream) {
+                                int write_rows, float temperature_coef, int temperature_every, void* stream) {
     if (tokens <= 0) return 0;
-    if (!projected || !q_weight || !k_weight || !queries || !positions || heads <= 0 || kv_heads <= 0 || dim <= 0 || vdim <= 0 || rotary < 0 || rotary > dim
+    if (!projected || !q_weight != !k_weight || temperature_every < 0 || !queries || !positions || heads <= 0 || kv_heads <= 0 || dim <= 0 || vdim <= 0 || rotary < 0 || rotary > dim
         || (rotary & 1) || (rotary > 0 && !inv_freq) || (write_rows && (!rows || !token_seq || !page_rows)))
         return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     if (dtype == TAU_F32)
         tau_launch(diff_prepare_kernel<float>, dim3(tokens), dim3(kWarps * 32), 0, s, static_cast<const float*>(projected), projected_stride, q_weight, k_weight,
                    eps, inv_freq, rotary, static_cast<float*>(queries), static_cast<float*>(rows), positions, token_seq, page_rows, page_stride, page_tokens,
-                   heads, kv_heads, dim, vdim, write_rows);
+                   heads, kv_heads, dim, vdim, write_rows, temperature_coef, temperature_every);
     else if (dtype == TAU_BF16)
         tau_launch(diff_prepare_kernel<bf16>, dim3(tokens), dim3(kWarps * 32), 0, s, static_cast<const bf16*>(projected), projected_stride, q_weight, k_weight,
                    eps, inv_freq, rotary, static_cast<bf16*>(queries), static_cast<bf16*>(rows), positions, token_seq, page_rows, page_stride, page_tokens,
-                   heads, kv_heads, dim, vdim, write_rows);
+                   heads, kv_heads, dim, vdim, write_rows, temperature_coef, temperature_every);
     else
         return cudaErrorInvalidValue;
     return tau_launch_status();

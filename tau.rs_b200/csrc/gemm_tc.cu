@@ -1070,7 +1070,7 @@ int prepare_group_streams() {
 }  // namespace
 
 TAU_EXPORT int tau_gemm_tc_groups(int out_dtype, const void* x, const void* w, void* out, const int* bounds, int groups, int N, int K,
-                                  long long x_stride, long long w_stride, long long out_stride, long long w_group, int gated, void* workspace,
+                                  long long x_stride, long long w_stride, long long out_stride, long long w_group, int gated, float gate_limit, void* workspace,
                                   long long workspace_floats, void* tickets, void* stream) {
     if (!bounds || groups <= 0) return cudaErrorInvalidValue;
     cudaStream_t caller = static_cast<cudaStream_t>(stream);
@@ -1091,7 +1091,7 @@ TAU_EXPORT int tau_gemm_tc_groups(int out_dtype, const void* x, const void* w, v
         result = tau_gemm_tc(out_dtype, static_cast<const bf16*>(x) + static_cast<size_t>(begin) * x_stride,
                              static_cast<const bf16*>(w) + static_cast<size_t>(group) * w_group, nullptr,
                              static_cast<char*>(out) + static_cast<size_t>(begin) * out_stride * out_bytes, rows, N, K, x_stride, w_stride,
-                             out_stride, 0, gated, spread ? 1 : 0, workspace, workspace_floats, tickets, -1, 1, 0.0f,
+                             out_stride, 0, gated, spread ? 1 : 0, workspace, workspace_floats, tickets, -1, 1, gate_limit,
                              spread ? static_cast<void*>(group_streams[launched % kGroupStreams]) : stream);
         ++launched;
     }

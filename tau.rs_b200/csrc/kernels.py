@@ -83,7 +83,7 @@ _CLASS_OF = {
     "attention_decode": "attention", "attention_prefill": "attention", "attention_prefill_tc": "attention", "argmax": "selection",
     "sample_gumbel": "selection", "store_words_host": "selection", "random_normal": "other",
     "stream_add_norm": "norm", "stream_add_tanh": "norm", "soft_cap": "other", "normed_pair_sum": "norm", "gated_group_norm": "norm", "gemm_simt_batched": "product", "linear_recurrence": "recurrence",
-    "latent_prepare": "attention", "latent_attention": "attention", "latent_expand": "attention", "moe_route": "routing", "moe_gate_up": "experts", "moe_down": "experts", "gemm_tc_groups": "experts", "moe_sort": "routing", "moe_gather": "routing",
+    "latent_prepare": "attention", "latent_attention": "attention", "latent_expand": "attention", "head_gate": "attention", "moe_route": "routing", "moe_gate_up": "experts", "moe_down": "experts", "gemm_tc_groups": "experts", "moe_sort": "routing", "moe_gather": "routing",
     "moe_combine": "routing", "diff_prepare": "attention", "diff_attention": "attention", "diff_combine": "attention", "causal_taps": "norm", "gated_add_norm": "norm",
     "side_gate": "activation", "unit_add_mix": "norm", "norm_rows": "norm", "relu_squared": "activation",
     "short_conv": "recurrence", "delta_prepare": "recurrence", "delta_rule": "recurrence", "selective_scan": "recurrence",
@@ -167,14 +167,15 @@ def embedding(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scal
                                  ctypes.c_int(table.shape[1]), ctypes.c_int(table.shape[0]), _stream()), "embedding")
 
 
-def rms_norm(values, weight, eps: float, out, rows=None, branch=None, groups: int = 1, branch_scale: float = 1.0) -> None:
+def rms_norm(values, weight, eps: float, out, rows=None, branch=None, groups: int = 1, branch_scale: float = 1.0, channel_scale=None, table_rows=None) -> None:
     """`out[i] = norm(round(values[r] + branch[r])) * weight`, `r = rows[i]` or `i`; `values` is not changed.
 
     Where `values` is a 32-bit stream and the output is not, or there are two branches (a tuple), the sum is taken in
     32-bit (`values[r] + branch_scale * (a[r] + b[r])`) and only the output is rounded; a norm over `groups` > 1 pieces of the row,
-    or a scale on the branches, needs the 32-bit stream as well."""
-    if isinstance(branch, (tuple, list)) or values.dtype != out.dtype or groups != 1 or branch_scale != 1.0:
-        return stream_add_norm(values, branch, weight, eps, out, rows=rows, update=False, groups=groups, branch_scale=branch_scale)
+    a scale on the branches or rows of a table that join (see `stream_add_norm`) need the 32-bit stream as well."""
+    if isinstance(branch, (tuple, list)) or values.dtype != out.dtype or groups != 1 or branch_scale != 1.0 or channel_scale is not None or table_rows is not None:
+        return stream_add_norm(values, branch, weight, eps, out, rows=rows, update=False, groups=groups, branch_scale=branch_scale, channel_scale=channel_scale,
+                               table_rows=table_rows)
     _on_device(values, weight, out, rows, branch)
     width = values.shape[-1]
     _f32_vector(weight, width, "the norm weight")
@@ -191,11 +192,12 @@ def rms_norm(values, weight, eps: float, out, rows=None, branch=None, groups: in
                                 ctypes.c_int(count), ctypes.c_int(width), ctypes.c_float(eps), _stream()), "rms_norm")
 
 
-def add_rms_norm(branch, residual, weight, eps: float, out, groups: int = 1, branch_scale: float = 1.0) -> None:
+def add_rms_norm(branch, residual, weight, eps: float, out, groups: int = 1, branch_scale: float = 1.0, channel_scale=None, table_rows=None) -> None:
     """`residual = round(residual + branch)` in place; `out = norm(residual) * weight`.  A 32-bit residual beside an output
-    of another dtype, two branches (a tuple), a norm in `groups` pieces or a scale on the branches go to `stream_add_norm`."""
-    if isinstance(branch, (tuple, list)) or residual.dtype != out.dtype or groups != 1 or branch_scale != 1.0:
-        return stream_add_norm(residual, branch, weight, eps, out, update=True, groups=groups, branch_scale=branch_scale)
+    of another dtype, two branches (a tuple), a norm in `groups` pieces, a scale on the branches or rows of a table go to `stream_add_norm`."""
+    if isinstance(branch, (tuple, list)) or residual.dtype != out.dtype or groups != 1 or branch_scale != 1.0 or channel_scale is not None or table_rows is not None:
+        return stream_add_norm(residual, branch, weight, eps, out, update=True, groups=groups, branch_scale=branch_scale, channel_scale=channel_scale,
+                               table_rows=table_rows)
     _on_device(branch, residual, weight, out)
     width = residual.shape[-1]
     _f32_vector(weight, width, "the norm weight")
@@ -211,11 +213,14 @@ def add_rms_norm(branch, residual, weight, eps: float, out, groups: int = 1, bra
 NORM_MAX_GROUPS = 1024
 
 
-def stream_add_norm(stream, branches, weight, eps: float, out, rows=None, update: bool = True, groups: int = 1, branch_scale: float = 1.0) -> None:
+def stream_add_norm(stream, branches, weight, eps: float, out, rows=None, update: bool = True, groups: int = 1, branch_scale: float = 1.0,
+                    channel_scale=None, table_rows=None) -> None:
     """A residual stream kept in 32-bit: `sum = stream[r] + branch_scale * (a[r] + b[r])` in 32-bit for up to two branches of any
     dtype (`branches`: None, a tensor or a tuple of one or two), `r = rows[i]` or `i`; with `update` (no `rows` then) the sum
     replaces `stream[r]`; `out[i] = sum / sqrt(mean(sum^2) + eps) * weight`, rounded once to the output's dtype.  With `groups` > 1
-    the row is cut into that many equal consecutive pieces, each divided by its own root mean square."""
+    the row is cut into that many equal consecutive pieces, each divided by its own root mean square.  `channel_scale` (float32
+    [width]) multiplies the branches' sum as well; `table_rows` = (table [any, width], numbers int32 [rows of the stream], factor) adds
+    `factor * table[numbers[r]]`, with or without branches."""
     _require(1 <= groups <= NORM_MAX_GROUPS and stream.shape[-1] % groups == 0, f"the groups (at most {NORM_MAX_GROUPS}) must divide the width")
     if branches is None:
         branches = ()
@@ -237,11 +242,23 @@ def stream_add_norm(stream, branches, weight, eps: float, out, rows=None, update
     _require(count == (rows.shape[0] if rows is not None else stream.numel() // width), "output row count does not match")
     first = branches[0] if branches else None
     second = branches[1] if len(branches) > 1 else None
+    _f32_vector(channel_scale, width, "the factors of the channels")
+    table, numbers, factor = (None, None, 1.0) if table_rows is None else table_rows
+    if table is not None:
+        _on_device(table, numbers)
+        _int_vector(numbers, "the table's row numbers")
+        _require(table.dim() == 2 and table.shape[1] == width and table.is_contiguous() and numbers.numel() == stream.numel() // width,
+                 "the table's rows must be as wide as the stream, one number for each of the stream's rows")
+    if first is None:
+        channel_scale = None      # nothing that it multiplies
+    _on_device(channel_scale)
     library = build.load_library("stream32.cu")
     _check(library.tau_stream_add_norm(_code(out), _pointer(stream), _pointer(first), ctypes.c_int(_code(first) if first is not None else 0),
                                        _pointer(second), ctypes.c_int(_code(second) if second is not None else 0), _pointer(rows), _pointer(weight),
                                        _pointer(out), ctypes.c_int(count), ctypes.c_int(width), ctypes.c_float(eps), ctypes.c_int(1 if update else 0),
-                                       ctypes.c_int(groups), ctypes.c_float(branch_scale), _stream()), "stream_add_norm")
+                                       ctypes.c_int(groups), ctypes.c_float(branch_scale), _pointer(channel_scale), _pointer(table),
+                                       ctypes.c_int(_code(table) if table is not None else 0), ctypes.c_int(table.shape[0] if table is not None else 0),
+                                       _pointer(numbers), ctypes.c_float(factor), _stream()), "stream_add_norm")
 
 
 def stream_add_tanh(stream, branches, alpha, weight, bias, out, rows=None, update: bool = True, branch_scale: float = 1.0) -> None:
@@ -471,9 +488,10 @@ def gemm_tc(values, weight, bias, out, token_box: int = 0, gated: bool = False, 
                                ctypes.c_float(gate_limit), _stream()), "gemm_tc")
 
 
-def gemm_tc_groups(values, weights, out, bounds, gated: bool = False) -> None:
+def gemm_tc_groups(values, weights, out, bounds, gated: bool = False, gate_limit: float = 0.0) -> None:
     """One tensor-core product per group of consecutive rows: rows `bounds[g] .. bounds[g + 1]` of `values` [M, K] meet
-    `weights[g]` ([groups, N, K]) and land in the same rows of `out` ([M, N], or [M, N / 2] = silu(gate) * up with `gated`).
+    `weights[g]` ([groups, N, K]) and land in the same rows of `out` ([M, N], or [M, N / 2] = silu(gate) * up with `gated`, its clamped
+    form with `gate_limit` > 0, see `silu_mul`).
     `bounds` is a host list of `groups + 1` ascending row numbers.  bfloat16, K % 8 == 0, 16-byte aligned rows."""
     _on_device(values, weights, out)
     rows, depth = values.shape
@@ -490,7 +508,7 @@ def gemm_tc_groups(values, weights, out, bounds, gated: bool = False) -> None:
     launched = sum(1 for index in range(groups) if bounds[index + 1] > bounds[index])
     _check(library.tau_gemm_tc_groups(_code(out), _pointer(values), _pointer(weights), _pointer(out), table, ctypes.c_int(groups), ctypes.c_int(features),
                                       ctypes.c_int(depth), ctypes.c_longlong(values.stride(0)), ctypes.c_longlong(weights.stride(1)),
-                                      ctypes.c_longlong(out.stride(0)), ctypes.c_longlong(weights.stride(0)), ctypes.c_int(1 if gated else 0),
+                                      ctypes.c_longlong(out.stride(0)), ctypes.c_longlong(weights.stride(0)), ctypes.c_int(1 if gated else 0), ctypes.c_float(gate_limit),
                                       _pointer(workspace), ctypes.c_longlong(workspace.numel()), _pointer(tickets), _stream()), "gemm_tc_groups", launched)
 
 
@@ -877,18 +895,21 @@ def latent_expand(q, down, expanded, queries, key_pages, value_pages, inv_freq, 
         ctypes.c_int(rot_dim), ctypes.c_int(rank), ctypes.c_int(value_dim), _stream()), "latent_expand")
 
 
-def head_gate(values, gate, out, n_heads: int, width: int, value_dim: int) -> None:
-    """`out[token, head, :] = values[token, head, :value_dim] * sigmoid(gate[token, head, :])`: `values` [tokens, n_heads * width],
-    `gate` [tokens, n_heads * value_dim] (rows any distance apart) or None, `out` [tokens, n_heads * value_dim]."""
+def head_gate(values, gate, out, n_heads: int, width: int, value_dim: int, per_head: bool = False) -> None:
+    """`out[token, head, :] = values[token, head, :value_dim] * sigmoid(gate[token, head, :])`: `values` [tokens, n_heads * width]
+    (the output's dtype or float32), `gate` [tokens, n_heads * value_dim] (rows any distance apart; with `per_head` [tokens, n_heads], one
+    number per head) or None, `out` [tokens, n_heads * value_dim]."""
     _on_device(values, gate, out)
     tokens = values.shape[0]
     _require(values.shape == (tokens, n_heads * width) and values.is_contiguous() and out.shape == (tokens, n_heads * value_dim) and out.is_contiguous()
-             and out.dtype == values.dtype and value_dim <= width, "values must be [tokens, heads * width] and the output [tokens, heads * value_dim]")
+             and values.dtype in (out.dtype, torch.float32) and value_dim <= width, "values must be [tokens, heads * width] and the output [tokens, heads * value_dim]")
     if gate is not None:
-        _require(gate.shape == out.shape and gate.dtype == out.dtype and gate.stride(1) == 1, "the gate must match the output")
+        _require(gate.shape == (tokens, n_heads if per_head else n_heads * value_dim) and gate.dtype == out.dtype and (gate.shape[1] == 1 or gate.stride(1) == 1),
+                 "the gate must be [tokens, heads] or match the output")
     library = build.load_library("latent_attention.cu")
-    _check(library.tau_head_gate(_code(values), _pointer(values), _pointer(gate), ctypes.c_longlong(0 if gate is None else gate.stride(0)), _pointer(out),
-                                 ctypes.c_int(tokens), ctypes.c_int(n_heads), ctypes.c_int(width), ctypes.c_int(value_dim), _stream()), "latent_expand")
+    _check(library.tau_head_gate(_code(values), _code(out), _pointer(values), _pointer(gate), ctypes.c_longlong(0 if gate is None else gate.stride(0)), _pointer(out),
+                                 ctypes.c_int(tokens), ctypes.c_int(n_heads), ctypes.c_int(width), ctypes.c_int(value_dim),
+                                 ctypes.c_int(1 if per_head else 0), _stream()), "head_gate")
 
 
 LATENT_MAX_RANK = 1024   # what the latent attention kernel keeps per lane (rows of up to 768 elements take the vector form)
@@ -939,12 +960,20 @@ def latent_attention(queries, rows, out, sinks, positions, token_seq, page_rows,
 DIFF_MAX_VALUE_DIM = 512
 
 
+def _temperature(temperature):
+    """The query temperature's two constants for a kernel (no factor at all: a period of 0)."""
+    coef, every = (0.0, 0) if temperature is None else (float(temperature[0]), int(temperature[1]))
+    _require(temperature is None or every > 0, "the temperature's period must be positive")
+    return ctypes.c_float(coef), ctypes.c_int(every)
+
+
 def diff_prepare(projected, q_weight, k_weight, eps: float, inv_freq, rotary_dim: int, queries, rows, positions, token_seq, page_rows,
-                 n_heads: int, n_kv_heads: int, dim: int, vdim: int, write_rows: bool = True) -> None:
+                 n_heads: int, n_kv_heads: int, dim: int, vdim: int, write_rows: bool = True, temperature=None) -> None:
     """`projected` [tokens, >= n_heads * 2 * dim + n_kv_heads * (2 * dim + vdim)] holds, per token, the two query maps of every head,
     the two key maps of every key/value head and the values.  Every map is divided by its root mean square over `dim` (eps inside
-    the root), multiplied by `q_weight` or `k_weight` (float32 [dim]) and its first `rotary_dim` elements are turned pair by pair
-    (2i, 2i + 1) by `position * inv_freq[i]`.  Queries go to `queries` [tokens, n_heads, 2, dim]; with `write_rows` keys and values
+    the root), multiplied by `q_weight` or `k_weight` (float32 [dim]; None: neither) and its first `rotary_dim` elements are turned pair by pair
+    (2i, 2i + 1) by `position * inv_freq[i]`.  `temperature` = (coef, every): the query at position p is multiplied by
+    `1 + coef * ln(floor((p + 1) / every) + 1)`.  Queries go to `queries` [tokens, n_heads, 2, dim]; with `write_rows` keys and values
     go to the token's row of the cache pages `rows` [pages, 64, n_kv_heads * (2 * dim + vdim)] as [keys of all heads | values]."""
     _on_device(projected, q_weight, k_weight, inv_freq, queries, rows, positions, token_seq, page_rows)
     tokens = projected.shape[0]
@@ -966,7 +995,7 @@ def diff_prepare(projected, q_weight, k_weight, eps: float, inv_freq, rotary_dim
         _code(projected), _pointer(projected), ctypes.c_longlong(projected.stride(0)), _pointer(q_weight), _pointer(k_weight), ctypes.c_float(eps),
         _pointer(inv_freq), ctypes.c_int(rotary_dim), _pointer(queries), _pointer(rows if write_rows else None), _pointer(positions), _pointer(token_seq),
         _pointer(page_rows), ctypes.c_int(page_rows.shape[1] if write_rows else 0), ctypes.c_int(PAGE_TOKENS), ctypes.c_int(tokens), ctypes.c_int(n_heads),
-        ctypes.c_int(n_kv_heads), ctypes.c_int(dim), ctypes.c_int(vdim), ctypes.c_int(1 if write_rows else 0), _stream()), "diff_prepare")
+        ctypes.c_int(n_kv_heads), ctypes.c_int(dim), ctypes.c_int(vdim), ctypes.c_int(1 if write_rows else 0), *_temperature(temperature), _stream()), "diff_prepare")
 
 
 def diff_attention(queries, rows, gate, out, step, page_rows, n_kv_heads: int, vdim: int, scale: float, window: int, lam: float, eps: float,
@@ -994,7 +1023,7 @@ def diff_attention(queries, rows, gate, out, step, page_rows, n_kv_heads: int, v
 
 
 def diff_prepare_wide(projected, q_weight, k_weight, eps: float, inv_freq, rotary_dim: int, queries, key_pages, value_pages, positions, token_seq,
-                      page_rows, n_heads: int, n_kv_heads: int, dim: int, vdim: int, write_cache: bool = True) -> None:
+                      page_rows, n_heads: int, n_kv_heads: int, dim: int, vdim: int, write_cache: bool = True, temperature=None) -> None:
     """As `diff_prepare`, for the cache of ordinary heads: every map becomes a head of `wide` = `queries.shape[2]` >= max(dim, vdim)
     elements, zeros behind what it holds.  `queries` [tokens, 2 * n_heads, wide] holds query (head, map) in slot
     `(group * 2 + map) * (n_heads / n_kv_heads) + head % (n_heads / n_kv_heads)`; `key_pages` and `value_pages`
@@ -1023,7 +1052,8 @@ def diff_prepare_wide(projected, q_weight, k_weight, eps: float, inv_freq, rotar
         _pointer(inv_freq), ctypes.c_int(rotary_dim), _pointer(queries), _pointer(key_pages if write_cache else None),
         _pointer(value_pages if write_cache else None), _pointer(positions), _pointer(token_seq), _pointer(page_rows),
         ctypes.c_int(page_rows.shape[1] if write_cache else 0), ctypes.c_int(PAGE_TOKENS), ctypes.c_int(tokens), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads),
-        ctypes.c_int(dim), ctypes.c_int(vdim), ctypes.c_int(wide), ctypes.c_int(1 if write_cache else 0), _stream()), "diff_prepare")
+        ctypes.c_int(dim), ctypes.c_int(vdim), ctypes.c_int(wide), ctypes.c_int(1 if write_cache else 0), *_temperature(temperature),
+        _stream()), "diff_prepare")
 
 
 def diff_combine(attended, gate, out, n_heads: int, n_kv_heads: int, vdim: int, lam: float, eps: float, post_scale: float) -> None:
@@ -1614,15 +1644,19 @@ def turn_heads(rows, positions, frequency, rotary_dim: int, n_heads: int, dim: i
 
 # ---------------------------------------------------------------------------- routed experts
 def moe_route(hidden, router, correction, shared_gate_weight, chosen, weights, shared_gate, top: int, softmax: bool = False,
-              renormalize: bool = False, logit_bias=None) -> None:
+              renormalize: bool = False, logit_bias=None, groups: int = 1, keep: int = 1, scale: float = 1.0) -> None:
     """Scores the experts of every token in 32-bit and chooses `top` of them: `router` float32 [experts, width];
     scores = sigmoid (or softmax) of `router @ hidden + logit_bias` (float32 [experts] or None); chosen by score + `correction` (float32 [experts] or None), the
-    lowest index among equals; `weights` are the chosen scores themselves (divided by their sum with `renormalize`).
+    lowest index among equals; `weights` are the chosen scores themselves (divided by their sum with `renormalize`), times `scale`.
+    `groups` > 1: the experts form that many equal groups of neighbours, ranked by the sum of their two largest choosing scores, and
+    only experts of the `keep` best groups can be chosen.
     `shared_gate[token] = sigmoid(shared_gate_weight . hidden[token])` where that weight (float32 [width]) is given."""
     _on_device(hidden, router, correction, shared_gate_weight, chosen, weights, shared_gate, logit_bias)
     tokens, width = hidden.shape
     experts = router.shape[0]
     _f32_vector(logit_bias, experts, "the router's bias")
+    _require(groups >= 1 and experts % groups == 0 and 1 <= keep <= groups and top <= keep * (experts // groups),
+             "the groups must be equal and those that are kept must hold enough experts")
     _require(hidden.is_contiguous() and router.dtype == torch.float32 and router.shape == (experts, width) and router.is_contiguous(),
              "the router must be float32 [experts, width]")
     _f32_vector(correction, experts, "the correction")
@@ -1635,15 +1669,15 @@ def moe_route(hidden, router, correction, shared_gate_weight, chosen, weights, s
     _check(library.tau_moe_route(_code(hidden), _pointer(hidden), _pointer(router), _pointer(logit_bias), _pointer(correction), _pointer(shared_gate_weight),
                                  _pointer(chosen), _pointer(weights), _pointer(shared_gate), ctypes.c_int(tokens), ctypes.c_int(width),
                                  ctypes.c_int(experts), ctypes.c_int(top), ctypes.c_int(1 if softmax else 0), ctypes.c_int(1 if renormalize else 0),
-                                 _stream()), "moe_route")
+                                 ctypes.c_int(groups), ctypes.c_int(keep), ctypes.c_float(scale), _stream()), "moe_route")
 
 
-def moe_gate_up(hidden, gate_up, chosen, inner, interleave: int = 0, input_weights=None) -> None:
+def moe_gate_up(hidden, gate_up, chosen, inner, interleave: int = 0, input_weights=None, limit: float = 0.0) -> None:
     # A pair whose expert number is not below `gate_up.shape[0]` chose an identity expert: its place of `inner` is left unwritten.
     """`inner[token, place] = silu(gate_e @ x) * (up_e @ x)` with `e = chosen[token, place]` and `x = h`, or
     `x = input_weights[token, place] * h` (float32 [tokens, top]; the weight multiplies the two products' 32-bit sums); `gate_up`
     [experts, 2 * I, width] holds each expert's gate rows, then its up rows, or with `interleave` groups of that many gate rows
-    each followed by their up rows (what `linear_gated` reads); `inner` [tokens, top, I]."""
+    each followed by their up rows (what `linear_gated` reads); `inner` [tokens, top, I].  `limit` > 0: the clamped form of `silu_mul`."""
     _require(interleave == 0 or inner.shape[2] % interleave == 0, "the interleaved groups must divide the expert's width")
     _on_device(hidden, gate_up, chosen, inner)
     tokens, width = hidden.shape
@@ -1657,7 +1691,8 @@ def moe_gate_up(hidden, gate_up, chosen, inner, interleave: int = 0, input_weigh
         _require(input_weights.shape == (tokens, top) and input_weights.dtype == torch.float32 and input_weights.is_contiguous(), "input weights must be float32 [tokens, top]")
     library = build.load_library("moe.cu")
     _check(library.tau_moe_gate_up(_code(hidden), _pointer(hidden), _pointer(gate_up), _pointer(chosen), _pointer(input_weights), _pointer(inner), ctypes.c_int(tokens),
-                                   ctypes.c_int(width), ctypes.c_int(size), ctypes.c_int(top), ctypes.c_int(interleave), ctypes.c_int(gate_up.shape[0]), _stream()), "moe_gate_up")
+                                   ctypes.c_int(width), ctypes.c_int(size), ctypes.c_int(top), ctypes.c_int(interleave), ctypes.c_int(gate_up.shape[0]),
+                                   ctypes.c_float(limit), _stream()), "moe_gate_up")
 
 
 def moe_down(inner, down, chosen, weights, shared_out, shared_gate, out, hidden=None) -> None:

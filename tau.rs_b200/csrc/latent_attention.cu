@@ -370,19 +370,57 @@ latent_expand_kernel(const T* __restrict__ q, long long q_stride, const T* __res
 }
 
 // out[token, head, :value_dim] = values[token, head, :value_dim] * sigmoid(gate[token, head, :]) where a head's values are the
-// first `value_dim` of `width` elements.
-template <typename T>
-__global__ void head_gate_kernel(const T* __restrict__ values, const T* __restrict__ gate, long long gate_stride, T* __restrict__ out, int heads,
-                                 int width, int value_dim) {
+// first `value_dim` of `width` elements; with `per_head` the gate is one number per head.  A thread takes V neighbouring columns
+// (V = 4 where rows and pointers allow).
+template <typename T> __device__ __forceinline__ void load_four(const T* source, float (&v)[4]);
+template <> __device__ __forceinline__ void load_four<float>(const float* source, float (&v)[4]) {
+    const float4 raw = *reinterpret_cast<const float4*>(source);
+    v[0] = raw.x; v[1] = raw.y; v[2] = raw.z; v[3] = raw.w;
+}
+template <> __device__ __forceinline__ void load_four<bf16>(const bf16* source, float (&v)[4]) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(source);
+    v[0] = __uint_as_float(raw.x << 16); v[1] = __uint_as_float(raw.x & 0xffff0000u);
+    v[2] = __uint_as_float(raw.y << 16); v[3] = __uint_as_float(raw.y & 0xffff0000u);
+}
+__device__ __forceinline__ void store_four(float* target, const float (&v)[4]) { *reinterpret_cast<float4*>(target) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store_four(bf16* target, const float (&v)[4]) {
+    const __nv_bfloat162 low = __floats2bfloat162_rn(v[0], v[1]), high = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(target) = make_uint2(*reinterpret_cast<const unsigned*>(&low), *reinterpret_cast<const unsigned*>(&high));
+}
+
+template <typename TV, typename T, int V>
+__global__ void __launch_bounds__(256)
+head_gate_kernel(const TV* __restrict__ values, const T* __restrict__ gate, long long gate_stride, T* __restrict__ out, int heads, int width, int value_dim,
+                 int per_head) {
     grid_dependents_launch();
     grid_dependency_wait();
     const size_t token = blockIdx.x;
-    for (int item = threadIdx.x; item < heads * value_dim; item += blockDim.x) {
-        const int head = item / value_dim, column = item % value_dim;
-        float value = to_float(values[(token * heads + head) * width + column]);
-        if (gate) value *= 1.0f / (1.0f + expf(-to_float(gate[token * gate_stride + item])));
-        out[token * heads * value_dim + item] = from_float<T>(value);
+    const int per_row = value_dim / V;
+    for (int item = threadIdx.x; item < heads * per_row; item += blockDim.x) {
+        const int head = item / per_row, column = item % per_row * V;
+        const TV* source = values + (token * heads + head) * width + column;
+        T* target = out + token * heads * value_dim + head * value_dim + column;
+        const T* g = gate ? gate + token * gate_stride + (per_head ? head : head * value_dim + column) : nullptr;
+        const float head_factor = g && per_head ? 1.0f / (1.0f + expf(-to_float(*g))) : 1.0f;
+        if constexpr (V == 4) {
+            float v[4];
+            load_four<TV>(source, v);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) v[i] *= g && !per_head ? 1.0f / (1.0f + expf(-to_float(g[i]))) : head_factor;
+            store_four(target, v);
+        } else {
+            *target = from_float<T>(to_float(*source) * (g && !per_head ? 1.0f / (1.0f + expf(-to_float(*g))) : head_factor));
+        }
     }
+}
+
+template <typename TV, typename T>
+int launch_head_gate(const void* values, const void* gate, long long gate_stride, void* out, int tokens, int heads, int width, int value_dim, int per_head,
+                     cudaStream_t s) {
+    const bool four = value_dim % 4 == 0 && width % 4 == 0 && ((reinterpret_cast<uintptr_t>(values) | reinterpret_cast<uintptr_t>(out)) & 15u) == 0;
+    tau_launch(four ? head_gate_kernel<TV, T, 4> : head_gate_kernel<TV, T, 1>, dim3(tokens), dim3(256), 0, s, static_cast<const TV*>(values),
+               static_cast<const T*>(gate), gate_stride, static_cast<T*>(out), heads, width, value_dim, per_head);
+    return tau_launch_status();
 }
 
 template <typename T>
@@ -486,18 +524,14 @@ TAU_EXPORT int tau_latent_expand(int dtype, const void* q, long long q_stride, c
     return tau_launch_status();
 }
 
-TAU_EXPORT int tau_head_gate(int dtype, const void* values, const void* gate, long long gate_stride, void* out, int tokens, int heads, int width,
-                             int value_dim, void* stream) {
+// `gate` and `out` have `dtype`, `values` that dtype or 32-bit.
+TAU_EXPORT int tau_head_gate(int values_dtype, int dtype, const void* values, const void* gate, long long gate_stride, void* out, int tokens, int heads, int width,
+                             int value_dim, int per_head, void* stream) {
     if (tokens <= 0) return 0;
     if (!values || !out || heads <= 0 || value_dim <= 0 || value_dim > width) return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    if (dtype == TAU_BF16)
-        tau_launch(head_gate_kernel<bf16>, dim3(tokens), dim3(256), 0, s, static_cast<const bf16*>(values), static_cast<const bf16*>(gate), gate_stride,
-                   static_cast<bf16*>(out), heads, width, value_dim);
-    else if (dtype == TAU_F32)
-        tau_launch(head_gate_kernel<float>, dim3(tokens), dim3(256), 0, s, static_cast<const float*>(values), static_cast<const float*>(gate), gate_stride,
-                   static_cast<float*>(out), heads, width, value_dim);
-    else
-        return cudaErrorInvalidValue;
-    return tau_launch_status();
+    if (values_dtype == TAU_BF16 && dtype == TAU_BF16) return launch_head_gate<bf16, bf16>(values, gate, gate_stride, out, tokens, heads, width, value_dim, per_head, s);
+    if (values_dtype == TAU_F32 && dtype == TAU_BF16) return launch_head_gate<float, bf16>(values, gate, gate_stride, out, tokens, heads, width, value_dim, per_head, s);
+    if (values_dtype == TAU_F32 && dtype == TAU_F32) return launch_head_gate<float, float>(values, gate, gate_stride, out, tokens, heads, width, value_dim, per_head, s);
+    return cudaErrorInvalidValue;
 }

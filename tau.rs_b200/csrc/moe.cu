@@ -3,8 +3,12 @@
 //
 //   route:    z = W_router h + bias (32-bit weights and sums; the bias is optional); s = sigmoid(z) or softmax(z); the `top` largest of
 //             s + correction are chosen (the lowest index among equals), their weights are s itself, divided by
-//             their sum if `renormalize`; shared_gate = sigmoid(w_sg . h).
-//   gate_up:  inner[token, place] = silu(W_gate[e] h) * (W_up[e] h) for the expert e of each (token, place).
+//             their sum (+ 1e-20) if `renormalize`, times a constant; shared_gate = sigmoid(w_sg . h).  With `groups` > 1 the
+//             experts form that many equal groups of neighbours; a group is ranked by the sum of the two largest of its
+//             s + correction (by its only one in groups of one), and only experts of the `keep` best groups (the lowest index
+//             among equals) can be chosen.
+//   gate_up:  inner[token, place] = silu(W_gate[e] h) * (W_up[e] h) for the expert e of each (token, place), or with a limit
+//             L > 0 g sigmoid(1.702 g) (u + 1), g = min(W_gate[e] h, L), u = W_up[e] h held between -L and L.
 //   down:     out[token] = sum over places of weight * (W_down[e] inner[token, place]) + shared_gate * shared[token], 32-bit.
 //
 // Experts numbered `real_experts` and up have no weights: they return what they read (identity experts), so a pair that chose one adds
@@ -129,13 +133,14 @@ template <typename T>
 __global__ void __launch_bounds__(kThreads)
 moe_route_kernel(const T* __restrict__ hidden, const float* __restrict__ router, const float* __restrict__ logit_bias, const float* __restrict__ correction,
                  const float* __restrict__ shared_gate_weight, int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ shared_gate,
-                 int width, int experts, int top, int softmax, int renormalize) {
+                 int width, int experts, int top, int softmax, int renormalize, int groups, int keep, float scale) {
     grid_dependents_launch();
     grid_dependency_wait();
     extern __shared__ __align__(16) float shared[];
     float* row = shared;               // [width]
     float* scores = shared + width;    // [experts]
     float* choice = scores + experts;  // [experts]
+    float* ranks = choice + experts;   // [groups], if there are several
     const int token = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     for (int column = threadIdx.x; column < width; column += blockDim.x) row[column] = to_float(hidden[static_cast<size_t>(token) * width + column]);
     __syncthreads();
@@ -162,6 +167,27 @@ moe_route_kernel(const T* __restrict__ hidden, const float* __restrict__ router,
     }
     for (int expert = lane; expert < experts; expert += 32) choice[expert] = scores[expert] + (correction ? correction[expert] : 0.0f);
     __syncwarp();
+    if (groups > 1) {
+        const int size = experts / groups;
+        for (int group = lane; group < groups; group += 32) {
+            float first = -INFINITY, second = -INFINITY;
+            for (int expert = group * size; expert < (group + 1) * size; ++expert) {
+                const float value = choice[expert];
+                if (value > first) { second = first; first = value; }
+                else if (value > second) second = value;
+            }
+            ranks[group] = size > 1 ? first + second : first;
+        }
+        __syncwarp();
+        // A group stays if fewer than `keep` groups stand before it.
+        for (int expert = lane; expert < experts; expert += 32) {
+            const int mine = expert / size;
+            int before = 0;
+            for (int group = 0; group < groups; ++group) before += ranks[group] > ranks[mine] || (ranks[group] == ranks[mine] && group < mine);
+            if (before >= keep) choice[expert] = -INFINITY;
+        }
+        __syncwarp();
+    }
     float total = 0.0f;
     for (int place = 0; place < top; ++place) {
         float best = -INFINITY;
@@ -185,15 +211,18 @@ moe_route_kernel(const T* __restrict__ hidden, const float* __restrict__ router,
         total += scores[best_expert];
         __syncwarp();
     }
-    if (renormalize && lane == 0)
-        for (int place = 0; place < top; ++place) weights[static_cast<size_t>(token) * top + place] /= total;
+    if ((renormalize || scale != 1.0f) && lane == 0)
+        for (int place = 0; place < top; ++place) {
+            float* weight = weights + static_cast<size_t>(token) * top + place;
+            *weight = (renormalize ? *weight / (total + 1e-20f) : *weight) * scale;
+        }
 }
 
 // grid (token-place pairs, feature tiles).  gate_up: [experts, 2 * inner, width], gate rows first.
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
 moe_gate_up_kernel(const T* __restrict__ hidden, const T* __restrict__ gate_up, const int* __restrict__ chosen, const float* __restrict__ input_weights,
-                   T* __restrict__ inner_out, int width, int inner, int top, int features_per_block, int interleave, int real_experts) {
+                   T* __restrict__ inner_out, int width, int inner, int top, int features_per_block, int interleave, int real_experts, float limit) {
     grid_dependents_launch();
     grid_dependency_wait();
     extern __shared__ __align__(16) float row[];
@@ -213,7 +242,8 @@ moe_gate_up_kernel(const T* __restrict__ hidden, const T* __restrict__ gate_up, 
         warp_dot_pair(weights + static_cast<size_t>(gate_row) * width, row, weights + static_cast<size_t>(up_row) * width, row, width, lane, gate, up);
         gate *= input_weight;
         up *= input_weight;
-        if (lane == 0) inner_out[static_cast<size_t>(pair) * inner + feature] = from_float<T>(gate / (1.0f + expf(-gate)) * up);
+        if (lane == 0)
+            inner_out[static_cast<size_t>(pair) * inner + feature] = from_float<T>(limit > 0.0f ? clamped_gate_exact(gate, up, limit) : gate / (1.0f + expf(-gate)) * up);
     }
 }
 
@@ -331,20 +361,23 @@ __global__ void moe_combine_kernel(const float* __restrict__ rows, const int* __
 
 template <typename T>
 int launch_all(int what, const void* a, const void* b, const void* c, const void* d, const void* e, const void* f, void* o1, void* o2, void* o3,
-               int tokens, int width, int inner, int experts, int top, int flag_a, int flag_b, cudaStream_t s, const void* g = nullptr) {
+               int tokens, int width, int inner, int experts, int top, int flag_a, int flag_b, cudaStream_t s, const void* g = nullptr, float constant = 1.0f,
+               int groups = 1, int keep = 1) {
     if (what == 0) {
-        const size_t bytes = (static_cast<size_t>(width) + 2 * experts) * sizeof(float);
+        const size_t bytes = (static_cast<size_t>(width) + 2 * experts + groups) * sizeof(float);
         if (bytes > 48 * 1024 && cudaFuncSetAttribute(moe_route_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)) != cudaSuccess)
             return cudaErrorInvalidValue;
         tau_launch(moe_route_kernel<T>, dim3(tokens), dim3(kThreads), bytes, s, static_cast<const T*>(a), static_cast<const float*>(b), static_cast<const float*>(e),
-                   static_cast<const float*>(c), static_cast<const float*>(d), static_cast<int*>(o1), static_cast<float*>(o2), static_cast<float*>(o3), width, experts, top, flag_a, flag_b);
+                   static_cast<const float*>(c), static_cast<const float*>(d), static_cast<int*>(o1), static_cast<float*>(o2), static_cast<float*>(o3), width, experts, top, flag_a, flag_b,
+                   groups, keep, constant);
     } else if (what == 1) {
         const int per_block = 64;
         const size_t bytes = static_cast<size_t>(width) * sizeof(float);
         if (bytes > 48 * 1024 && cudaFuncSetAttribute(moe_gate_up_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)) != cudaSuccess)
             return cudaErrorInvalidValue;
         tau_launch(moe_gate_up_kernel<T>, dim3(tokens * top, (inner + per_block - 1) / per_block), dim3(kThreads), bytes, s, static_cast<const T*>(a),
-                   static_cast<const T*>(b), static_cast<const int*>(c), static_cast<const float*>(d), static_cast<T*>(o1), width, inner, top, per_block, flag_a, experts);
+                   static_cast<const T*>(b), static_cast<const int*>(c), static_cast<const float*>(d), static_cast<T*>(o1), width, inner, top, per_block, flag_a, experts,
+                   constant);
     } else {
         const int per_block = tokens * ((width + 63) / 64) >= 1024 ? 64 : tokens * ((width + 31) / 32) >= 1024 ? 32 : 16;   // few tokens: smaller tiles, more blocks
         const size_t bytes = static_cast<size_t>(top) * inner * sizeof(float);
@@ -360,24 +393,26 @@ int launch_all(int what, const void* a, const void* b, const void* c, const void
 }  // namespace
 
 TAU_EXPORT int tau_moe_route(int dtype, const void* hidden, const float* router, const float* logit_bias, const float* correction, const float* shared_gate_weight, int* chosen,
-                             float* weights, float* shared_gate, int tokens, int width, int experts, int top, int softmax, int renormalize, void* stream) {
+                             float* weights, float* shared_gate, int tokens, int width, int experts, int top, int softmax, int renormalize, int groups, int keep,
+                             float scale, void* stream) {
     if (tokens <= 0) return 0;
-    if (!hidden || !router || !chosen || !weights || width <= 0 || experts <= 0 || top <= 0 || top > experts || (shared_gate_weight && !shared_gate))
+    if (!hidden || !router || !chosen || !weights || width <= 0 || experts <= 0 || top <= 0 || top > experts || (shared_gate_weight && !shared_gate)
+        || groups < 1 || experts % groups != 0 || keep < 1 || keep > groups || top > keep * (experts / groups))
         return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    if (dtype == TAU_F32) return launch_all<float>(0, hidden, router, correction, shared_gate_weight, logit_bias, nullptr, chosen, weights, shared_gate, tokens, width, 0, experts, top, softmax, renormalize, s);
-    if (dtype == TAU_BF16) return launch_all<bf16>(0, hidden, router, correction, shared_gate_weight, logit_bias, nullptr, chosen, weights, shared_gate, tokens, width, 0, experts, top, softmax, renormalize, s);
+    if (dtype == TAU_F32) return launch_all<float>(0, hidden, router, correction, shared_gate_weight, logit_bias, nullptr, chosen, weights, shared_gate, tokens, width, 0, experts, top, softmax, renormalize, s, nullptr, scale, groups, keep);
+    if (dtype == TAU_BF16) return launch_all<bf16>(0, hidden, router, correction, shared_gate_weight, logit_bias, nullptr, chosen, weights, shared_gate, tokens, width, 0, experts, top, softmax, renormalize, s, nullptr, scale, groups, keep);
     return cudaErrorInvalidValue;
 }
 
 // `real_experts`: experts with weights (gate_up holds that many); a pair that chose a higher number is left alone.
 TAU_EXPORT int tau_moe_gate_up(int dtype, const void* hidden, const void* gate_up, const int* chosen, const float* input_weights, void* inner_out, int tokens,
-                               int width, int inner, int top, int interleave, int real_experts, void* stream) {
+                               int width, int inner, int top, int interleave, int real_experts, float limit, void* stream) {
     if (tokens <= 0) return 0;
     if (!hidden || !gate_up || !chosen || !inner_out || width <= 0 || inner <= 0 || top <= 0 || static_cast<long long>(tokens) * top > 0x7fffffff) return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    if (dtype == TAU_F32) return launch_all<float>(1, hidden, gate_up, chosen, input_weights, nullptr, nullptr, inner_out, nullptr, nullptr, tokens, width, inner, real_experts, top, interleave, 0, s);
-    if (dtype == TAU_BF16) return launch_all<bf16>(1, hidden, gate_up, chosen, input_weights, nullptr, nullptr, inner_out, nullptr, nullptr, tokens, width, inner, real_experts, top, interleave, 0, s);
+    if (dtype == TAU_F32) return launch_all<float>(1, hidden, gate_up, chosen, input_weights, nullptr, nullptr, inner_out, nullptr, nullptr, tokens, width, inner, real_experts, top, interleave, 0, s, nullptr, limit);
+    if (dtype == TAU_BF16) return launch_all<bf16>(1, hidden, gate_up, chosen, input_weights, nullptr, nullptr, inner_out, nullptr, nullptr, tokens, width, inner, real_experts, top, interleave, 0, s, nullptr, limit);
     return cudaErrorInvalidValue;
 }
 

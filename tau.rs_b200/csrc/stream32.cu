@@ -24,29 +24,53 @@ __global__ void embedding_f32_kernel(const int* __restrict__ tokens, const T* __
     for (int column = threadIdx.x; column < width; column += blockDim.x) target[column] = inside ? to_float(source[column]) * scale : 0.0f;
 }
 
-// r = rows ? rows[i] : i.  sum = stream[r] + branch_scale * (a[r] + b[r]) in 32-bit; if `update` the sum replaces stream[r];
-// out[i] = sum / sqrt(mean(sum^2) + eps) * weight, rounded once to T.  With `groups` > 1 the row is cut into that many equal
-// consecutive pieces and each is divided by its own root mean square (a warp sums a piece's squares).
+// What joins a row of the stream: up to two branches, the factors on their sum (one number, and one per channel if there is a vector), and
+// a row of a table (row table_ids[r] of `table_rows` rows, times `table_scale`), which no other factor touches.
+struct Joining {
+    const void* a;
+    const void* b;
+    const float* channel_scale;
+    const void* table;
+    const int* table_ids;
+    int a_code, b_code, table_code, table_rows;
+    float branch_scale, table_scale;
+};
+
+__device__ __forceinline__ bool anything_joins(const Joining& j) { return j.a != nullptr || j.table != nullptr; }
+
+// The table's row that joins row r of the stream (nothing is read of a table whose row number lies outside it).
+__device__ __forceinline__ long long table_row_of(const Joining& j, int r) {
+    if (!j.table) return -1;
+    const int id = j.table_ids[r];
+    return id >= 0 && id < j.table_rows ? id : -1;
+}
+
+// r = rows ? rows[i] : i.  sum = stream[r] + branch_scale * channel_scale * (a[r] + b[r]) + table_scale * table[ids[r]] in 32-bit; if
+// `update` the sum replaces stream[r]; out[i] = sum / sqrt(mean(sum^2) + eps) * weight, rounded once to T.  With `groups` > 1 the row is cut
+// into that many equal consecutive pieces and each is divided by its own root mean square (a warp sums a piece's squares).
 constexpr int kMaxNormGroups = 1024;
 
 template <typename T>
 __global__ void __launch_bounds__(kThreads)
-stream_add_norm_kernel(float* __restrict__ stream, const void* __restrict__ a, int a_code, const void* __restrict__ b, int b_code,
-                       const int* __restrict__ rows, const float* __restrict__ weight, T* __restrict__ out, int width, float eps, int update,
-                       int groups, float branch_scale) {
+stream_add_norm_kernel(float* __restrict__ stream, const Joining join, const int* __restrict__ rows, const float* __restrict__ weight,
+                       T* __restrict__ out, int width, float eps, int update, int groups) {
     grid_dependents_launch();
     grid_dependency_wait();
     __shared__ float scratch[33];
     __shared__ float inverses[kMaxNormGroups];
     const int row = rows ? rows[blockIdx.x] : blockIdx.x;
     const size_t base = static_cast<size_t>(row) * width;
+    const bool a = anything_joins(join);
+    const long long table_row = table_row_of(join, row);
     auto joined = [&](int column) {
         float value = stream[base + column];
-        if (a) {
-            float branch = load_as_float(a, a_code, base + column);
-            if (b) branch += load_as_float(b, b_code, base + column);
-            value = fmaf(branch_scale, branch, value);
+        if (join.a) {
+            float branch = load_as_float(join.a, join.a_code, base + column);
+            if (join.b) branch += load_as_float(join.b, join.b_code, base + column);
+            if (join.channel_scale) branch *= join.channel_scale[column];
+            value = fmaf(join.branch_scale, branch, value);
         }
+        if (table_row >= 0) value = fmaf(join.table_scale, load_as_float(join.table, join.table_code, static_cast<size_t>(table_row) * width + column), value);
         return value;
     };
     T* target = out + static_cast<size_t>(blockIdx.x) * width;
@@ -114,6 +138,82 @@ __device__ __forceinline__ void store_columns(bf16* target, const float (&v)[kPe
     } else {
         target[0] = __float2bfloat16_rn(v[0]);
     }
+}
+
+// The same sum and norm (one group) for rows of whole 16-byte pieces: a thread holds its columns of the sum in registers between the two
+// passes, four neighbouring ones at a time, `kPieces` times; width <= 4 * blockDim.x * kPieces.
+template <typename T, int kPieces>
+__global__ void __launch_bounds__(kThreads)
+stream_add_norm_vec_kernel(float* __restrict__ stream, const Joining join, const int* __restrict__ rows, const float* __restrict__ weight,
+                           T* __restrict__ out, int width, float eps, int update) {
+    grid_dependents_launch();
+    grid_dependency_wait();
+    __shared__ float scratch[33];
+    const int row = rows ? rows[blockIdx.x] : blockIdx.x;
+    const size_t base = static_cast<size_t>(row) * width;
+    const long long table_row = table_row_of(join, row);
+    const bool store = update && anything_joins(join);
+    float sum[kPieces][4];
+    float squares = 0.0f;
+#pragma unroll
+    for (int piece = 0; piece < kPieces; ++piece) {
+        const int column = (piece * blockDim.x + threadIdx.x) * 4;
+        if (column >= width) break;
+        load_columns<4>(stream, TAU_F32, base + column, sum[piece]);
+        if (join.a) {
+            float branch[4], other[4];
+            load_columns<4>(join.a, join.a_code, base + column, branch);
+            if (join.b) {
+                load_columns<4>(join.b, join.b_code, base + column, other);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) branch[i] += other[i];
+            }
+            if (join.channel_scale) {
+                load_columns<4>(join.channel_scale, TAU_F32, column, other);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) branch[i] *= other[i];
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) sum[piece][i] = fmaf(join.branch_scale, branch[i], sum[piece][i]);
+        }
+        if (table_row >= 0) {
+            float looked_up[4];
+            load_columns<4>(join.table, join.table_code, static_cast<size_t>(table_row) * width + column, looked_up);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) sum[piece][i] = fmaf(join.table_scale, looked_up[i], sum[piece][i]);
+        }
+        if (store) store_columns<4>(stream + base + column, sum[piece]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) squares = fmaf(sum[piece][i], sum[piece][i], squares);
+    }
+    const float inverse = 1.0f / sqrtf(block_sum(squares, scratch) / static_cast<float>(width) + eps);
+    T* target = out + static_cast<size_t>(blockIdx.x) * width;
+#pragma unroll
+    for (int piece = 0; piece < kPieces; ++piece) {
+        const int column = (piece * blockDim.x + threadIdx.x) * 4;
+        if (column >= width) break;
+        float w[4], result[4];
+        load_columns<4>(weight, TAU_F32, column, w);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) result[i] = sum[piece][i] * inverse * w[i];
+        store_columns<4>(target + column, result);
+    }
+}
+
+template <typename T>
+void launch_add_norm(float* stream_values, const Joining& join, const int* rows, const float* weight, void* out, int out_rows, int width, float eps, int update,
+                     int groups, cudaStream_t s) {
+    auto whole = [](const void* pointer) { return (reinterpret_cast<uintptr_t>(pointer) & 15u) == 0; };      // a null pointer is aligned
+    const bool vectors = groups == 1 && width % 4 == 0 && width <= 4 * kThreads * 8 && whole(stream_values) && whole(join.a) && whole(join.b) && whole(join.channel_scale)
+                         && whole(join.table) && whole(weight) && whole(out);
+    if (!vectors) {
+        tau_launch(stream_add_norm_kernel<T>, dim3(out_rows), dim3(kThreads), 0, s, stream_values, join, rows, weight, static_cast<T*>(out), width, eps, update, groups);
+        return;
+    }
+    const int pieces = (width / 4 + kThreads - 1) / kThreads;      // of four columns to a thread
+    const dim3 block(pieces == 1 ? (width / 4 + 31) / 32 * 32 : kThreads);
+    auto* kernel = pieces == 1 ? stream_add_norm_vec_kernel<T, 1> : pieces == 2 ? stream_add_norm_vec_kernel<T, 2> : pieces <= 4 ? stream_add_norm_vec_kernel<T, 4> : stream_add_norm_vec_kernel<T, 8>;
+    tau_launch(kernel, dim3(out_rows), block, 0, s, stream_values, join, rows, weight, static_cast<T*>(out), width, eps, update);
 }
 
 template <typename T, int kPer>
@@ -270,13 +370,16 @@ TAU_EXPORT int tau_embedding_f32(int table_dtype, const int* tokens, const void*
 
 TAU_EXPORT int tau_stream_add_norm(int out_dtype, float* stream_values, const void* a, int a_dtype, const void* b, int b_dtype, const int* rows,
                                    const float* weight, void* out, int out_rows, int width, float eps, int update, int groups, float branch_scale,
+                                   const float* channel_scale, const void* table, int table_dtype, int table_rows, const int* table_ids, float table_scale,
                                    void* stream) {
     if (out_rows <= 0) return 0;
-    if (!stream_values || !weight || !out || width <= 0 || (b && !a) || (update && rows) || groups < 1 || groups > kMaxNormGroups || width % groups != 0)
+    if (!stream_values || !weight || !out || width <= 0 || (b && !a) || (update && rows) || groups < 1 || groups > kMaxNormGroups || width % groups != 0
+        || (table && (!table_ids || table_rows <= 0)) || (channel_scale && !a))
         return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    if (out_dtype == TAU_F32) tau_launch(stream_add_norm_kernel<float>, dim3(out_rows), dim3(kThreads), 0, s, stream_values, a, a_dtype, b, b_dtype, rows, weight, static_cast<float*>(out), width, eps, update, groups, branch_scale);
-    else if (out_dtype == TAU_BF16) tau_launch(stream_add_norm_kernel<bf16>, dim3(out_rows), dim3(kThreads), 0, s, stream_values, a, a_dtype, b, b_dtype, rows, weight, static_cast<bf16*>(out), width, eps, update, groups, branch_scale);
+    const Joining join{a, b, channel_scale, table, table_ids, a_dtype, b_dtype, table_dtype, table_rows, branch_scale, table_scale};
+    if (out_dtype == TAU_F32) launch_add_norm<float>(stream_values, join, rows, weight, out, out_rows, width, eps, update, groups, s);
+    else if (out_dtype == TAU_BF16) launch_add_norm<bf16>(stream_values, join, rows, weight, out, out_rows, width, eps, update, groups, s);
     else return cudaErrorInvalidValue;
     return tau_launch_status();
 }

@@ -1,2 +1,2 @@
 """Architectures.  Importing this package registers each of them by name."""
-from . import bikovik, bisudra, fasesun, nugolorn, pegurax, qwen3  # noqa: F401
+from . import bikovik, bisudra, fasesun, nugolorn, pegurax, qwen3, tukulorn  # noqa: F401

@@ -42,15 +42,30 @@ class CacheNeed:
 
 
 class Pending(tuple):
-    """Results that have yet to join the residual stream (one or two tensors), and the factor that they join it with: the norm that
-    adds them computes `stream + scale * (sum of the results)`."""
+    """What has yet to join the residual stream: results (up to two tensors), the factors that they join it with (one number, and a
+    32-bit vector over the channels or None), and rows of a table (None, or `(table, row numbers, factor)`): the norm that adds them
+    computes `stream + scale * channel_scale * (sum of the results) + factor * table[row numbers]`."""
 
-    scale = 1.0
+    scale, channel_scale, rows = 1.0, None, None
 
-    def __new__(cls, results, scale: float = 1.0):
+    def __new__(cls, results, scale: float = 1.0, channel_scale=None, rows=None):
         pending = super().__new__(cls, results)
-        pending.scale = float(scale)
+        pending.scale, pending.channel_scale, pending.rows = float(scale), channel_scale, rows
         return pending
+
+    @classmethod
+    def with_rows(cls, branch, rows) -> "Pending":
+        """`branch` (None, a tensor, a tuple or a Pending) and the rows of a table beside it."""
+        results = () if branch is None else tuple(branch) if isinstance(branch, (tuple, list)) else (branch,)
+        if getattr(branch, "rows", None) is not None:
+            raise ValueError("rows of a table are pending already")
+        return cls(results, getattr(branch, "scale", 1.0), getattr(branch, "channel_scale", None), rows)
+
+
+def require_plain_pending(branch) -> None:
+    """For norms that add results alone: refuses a factor per channel and rows of a table."""
+    if getattr(branch, "channel_scale", None) is not None or getattr(branch, "rows", None) is not None:
+        raise ValueError("a norm of this kind adds results with one factor; a factor per channel or rows of a table are not served")
 
 
 class Part:

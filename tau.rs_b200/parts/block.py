@@ -13,7 +13,7 @@ import math
 import torch
 
 from ..csrc import kernels
-from .base import Block
+from .base import Block, Pending
 from .registry import build, register_block
 
 
@@ -25,9 +25,12 @@ class PreNormBlock(Block):
     feed_forward_norm_name = "post_attention_layernorm"
 
     norm_suffix = ".weight"
+    scale_names = ()
 
     def __init__(self, spec, dtype, device):
         self.spec = spec
+        if getattr(spec, "layer_scale", False) and not self.scale_names:
+            raise ValueError(f"a block of kind {spec.kind!r} has no factor per channel on its results")
         prefix, suffix = spec.prefix, self.norm_suffix
         self.mixer_norm = build("norm", spec.mixer_norm, name=f"{prefix}.{self.mixer_norm_name}{suffix}", dtype=dtype, device=device)
         self.mixer = build("mixer", spec.mixer, prefix=f"{prefix}.{self.mixer_name}", dtype=dtype, device=device)
@@ -82,22 +85,52 @@ class PreNormBlock(Block):
 @register_block("pre_norm_stream")
 class StreamPreNormBlock(PreNormBlock):
     """The same arrangement on a residual stream kept in 32-bit: a sublayer's result joins it and the new stream passes the next norm in one
-    kernel (the norm's `add_forward`); the feed-forward may be absent.  What the mixer keeps beside its cache is the block's as well.
-    Weight names: `<prefix>.norm1`, `<prefix>.mix.*`, `<prefix>.norm2`, `<prefix>.mlp.*`."""
+    kernel (the norm's `add_forward`); the feed-forward may be absent.  With `layer_scale` each result is multiplied by a vector of the
+    stream's width in that same kernel, in 32-bit.  What the mixer keeps beside its cache is the block's as well.
+    Weight names: `<prefix>.norm1`, `<prefix>.mix.*`, `<prefix>.norm2`, `<prefix>.mlp.*`, `<prefix>.ls1`, `<prefix>.ls2`."""
 
     mixer_name = "mix"
     feed_forward_name = "mlp"
     mixer_norm_name = "norm1"
     feed_forward_norm_name = "norm2"
     norm_suffix = ""
+    scale_names = ("ls1", "ls2")
+
+    def __init__(self, spec, dtype, device):
+        from ..weights.tensor_spec import TensorSpec
+
+        super().__init__(spec, dtype, device)
+        names = self.scale_names[: 2 if self.feed_forward is not None else 1] if getattr(spec, "layer_scale", False) else ()
+        self._own = {f"{spec.prefix}.{name}": TensorSpec((spec.mixer_norm.width,), role="vector", init="ones") for name in names}
+        self._scales = {}
 
     def extra_cache_needs(self):
         return self.mixer.extra_cache_needs()
 
+    def tensor_specs(self):
+        return {**self._own, **super().tensor_specs()}
+
+    def assign(self, name, tensor):
+        if name in self._own:
+            self._scales[name] = tensor
+        else:
+            super().assign(name, tensor)
+
+    def bytes_read_per_step(self, dtype) -> int:
+        return sum(4 * math.prod(spec.shape) for spec in self._own.values()) + super().bytes_read_per_step(dtype)
+
+    def _scaled(self, result, name):
+        return Pending((result,), channel_scale=self._scales[f"{self.spec.prefix}.{name}"]) if self._own else result
+
     def forward(self, residual, branch, step, cache, writes_cache: bool):
         if residual.dtype != torch.float32:
             raise ValueError("this block keeps its residual stream in 32-bit (ModelSpec.residual_dtype)")
-        return super().forward(residual, branch, step, cache, writes_cache)
+        normalized = self.mixer_norm.forward(residual) if branch is None else self.mixer_norm.add_forward(branch, residual)
+        mixed = self._scaled(self.mixer.forward(normalized, step, cache, writes_cache), self.scale_names[0])
+        if self.feed_forward is None:
+            return residual, mixed
+        normalized = self.feed_forward_norm.add_forward(mixed, residual)
+        return residual, self._scaled(self.feed_forward.forward(normalized, step), self.scale_names[1])
 
 
 @register_block("parallel")

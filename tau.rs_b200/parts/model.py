@@ -14,7 +14,7 @@ import torch
 from ..config.specs import ModelSpec
 from ..csrc import kernels
 from ..weights.tensor_spec import TensorSpec
-from .base import CacheNeed
+from .base import CacheNeed, Pending
 from .registry import build
 
 
@@ -37,6 +37,8 @@ class DecoderModel:
         for entry in spec.schedule:
             if not 0 <= entry.layer < len(self.blocks):
                 raise ValueError(f"schedule names layer {entry.layer}, the model has {len(self.blocks)}")
+            if getattr(entry, "joins_embedding", False) and (self.residual_dtype != torch.float32 or spec.input_position is not None):
+                raise ValueError("the embedding output joins again on a stream kept in 32-bit and without an encoding added to it")
         self._groups = self._collect_cache_groups()
         self._shared = {name: TensorSpec(tuple(shape), role=role) for name, shape, role in getattr(spec, "shared_tensors", ())}
         self.shared: Dict[str, torch.Tensor] = {}
@@ -161,6 +163,8 @@ class DecoderModel:
                     raise ValueError("a block that keeps something beside its mixer's cache needs that cache as well")
                 view.extra = {role: cache.layer_view(group, layer) for role, group, layer in extra}
             step.run = run
+            if getattr(entry, "joins_embedding", False):      # looked up again by the norm that adds it, so that no copy is kept
+                branch = Pending.with_rows(branch, (self.embedding, step.token_ids, getattr(spec, "embedding_scale", 1.0)))
             residual, branch = self.blocks[entry.layer].forward(residual, branch, step, view, entry.writes_cache)
         step.results = None
         step.handed_on.clear()

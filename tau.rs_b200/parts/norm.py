@@ -1,5 +1,6 @@
 """RMSNorm: `x * rsqrt(mean(x^2) + eps) * w`, statistic in 32-bit, one rounding; with `groups` > 1 each of that many equal
-consecutive pieces of the row is divided by its own root mean square.
+consecutive pieces of the row is divided by its own root mean square.  The weight's tensor may be stored around zero
+(`weight_offset`, added in 32-bit when the weights are loaded).
 
 crates/models/src/components/rms_norm.rs:205-210 and :147-150; the in-tree norm scales
 by `1 + w`, this part by `w`.  The fused form first rounds `residual + branch` to the
@@ -12,7 +13,7 @@ import torch
 
 from ..csrc import kernels
 from ..weights.tensor_spec import TensorSpec
-from .base import Norm
+from .base import Norm, require_plain_pending
 from .registry import register_norm
 
 
@@ -24,19 +25,30 @@ class RMSNorm(Norm):
         self.weight = None
 
     def tensor_specs(self):
-        return {self.name: TensorSpec((self.spec.width,), role="vector", init="ones")}
+        around_zero = getattr(self.spec, "weight_offset", 0.0) != 0.0
+        return {self.name: TensorSpec((self.spec.width,), role="vector", init="normal" if around_zero else "ones")}
 
     def assign(self, name, tensor):
         if name != self.name:
             raise KeyError(name)
         self.weight = tensor
 
+    def finalize_weights(self):
+        offset = getattr(self.spec, "weight_offset", 0.0)
+        if offset != 0.0:
+            self.weight = self.weight + offset
+
     def _options(self, branch) -> dict:
-        """What only some models ask of the kernel: pieces of the row normalised one by one, a factor on what joins the stream."""
+        """What only some models ask of the kernel: pieces of the row normalised one by one, factors on what joins the stream, rows of
+        a table that join it too."""
         groups, scale = getattr(self.spec, "groups", 1), getattr(branch, "scale", 1.0)
         options = {} if groups == 1 else {"groups": groups}
         if scale != 1.0:
             options["branch_scale"] = scale
+        if getattr(branch, "channel_scale", None) is not None:
+            options["channel_scale"] = branch.channel_scale
+        if getattr(branch, "rows", None) is not None:
+            options["table_rows"] = branch.rows
         return options
 
     def forward(self, values, rows=None, branch=None):
@@ -108,12 +120,14 @@ class DynamicTanh(Norm):
         setattr(self, attribute, tensor)
 
     def forward(self, values, rows=None, branch=None):
+        require_plain_pending(branch)
         count = values.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((count, self.spec.width), dtype=self.dtype or values.dtype, device=values.device)
         kernels.stream_add_tanh(values, branch, self.alpha, self.weight, self.bias, out, rows, update=False, branch_scale=getattr(branch, "scale", 1.0))
         return out
 
     def add_forward(self, branch, residual):
+        require_plain_pending(branch)
         out = torch.empty(residual.shape, dtype=self.dtype or residual.dtype, device=residual.device)
         kernels.stream_add_tanh(residual, branch, self.alpha, self.weight, self.bias, out, update=True, branch_scale=getattr(branch, "scale", 1.0))
         return out

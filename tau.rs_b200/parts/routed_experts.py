@@ -1,7 +1,8 @@
 """Routed experts: each token passes `top` of `experts` gated feed-forwards, and optionally a shared one.
 
     z = W_router h (+ b_router) (32-bit);   s = sigmoid(z) (or softmax(z))
-    chosen = the `top` experts with the largest s + correction;   weights = s of the chosen (renormalised only if asked)
+    chosen = the `top` experts with the largest s + correction (among the best groups of experts only, if the router has groups);
+    weights = s of the chosen (renormalised only if asked), times a constant
     out = sum over chosen e of weight_e * W_down,e (silu(W_gate,e h) * (W_up,e h))  +  sigmoid(w_sg . h) * shared(h)
     (`weigh == "input"`: the weight multiplies what the expert reads instead, out = sum over chosen e of expert_e(weight_e * h))
 
@@ -14,6 +15,8 @@ The router, the choice and the weighted sum are 32-bit, and so is the output.  T
   device, each expert's rows pass through the tensor-core products that dense feed-forwards use (gate and up as one gated
   product), and a last kernel sums each token's places in place order.  The host reads the experts' row counts for this
   (one small copy per layer), which a prompt's step can afford and a captured decode step could not.
+
+`activation == "clamped"`: an expert is `W_down (g sigmoid(1.702 g) (u + 1))`, `g` and `u` the clamped gate and up values.
 
 `identity` experts have no tensors: the router scores them like the others (its last outputs), and a token that chooses one adds
 its weight times the token itself.  The expert kernels skip such places and the summing kernels put the token's row in their stead.
@@ -52,7 +55,17 @@ class RoutedExperts(FeedForward):
             raise ValueError("the number of identity experts cannot be negative")
         if self.identity and getattr(spec, "weigh", "output") == "input":
             raise ValueError("identity experts are summed with their weights on the output; weights on the experts' input are not served beside them")
+        if getattr(spec, "activation", "silu") not in ("silu", "clamped"):
+            raise ValueError(f"unknown activation {spec.activation!r}")
+        self.limit = float(spec.limit) if getattr(spec, "activation", "silu") == "clamped" else 0.0
+        if getattr(spec, "activation", "silu") == "clamped" and self.limit <= 0.0:
+            raise ValueError("a clamped gate needs a positive limit")
         self.outputs = spec.experts + self.identity      # what the router scores
+        self.groups, self.keep_groups = getattr(spec, "groups", 1), getattr(spec, "keep_groups", 1)
+        if self.groups < 1 or self.outputs % self.groups or not 1 <= self.keep_groups <= self.groups:
+            raise ValueError("the router's groups must be equal and at most all of them kept")
+        if spec.top > self.keep_groups * (self.outputs // self.groups):
+            raise ValueError("top exceeds the experts of the groups that are kept")
         if spec.top > self.outputs:
             raise ValueError("top must lie between 1 and the number of router outputs")
         self.shared = None if spec.shared is None else build("feed_forward", spec.shared, prefix=f"{prefix}.shared", dtype=dtype, device=device)
@@ -118,8 +131,11 @@ class RoutedExperts(FeedForward):
         chosen = torch.empty((tokens, spec.top), dtype=torch.int32, device=device)
         weights = torch.empty((tokens, spec.top), dtype=torch.float32, device=device)
         shared_gate = torch.empty((tokens,), dtype=torch.float32, device=device) if spec.shared_gate else None
+        options = {} if self.groups == 1 else {"groups": self.groups, "keep": self.keep_groups}
+        if getattr(spec, "scale", 1.0) != 1.0:
+            options["scale"] = spec.scale
         kernels.moe_route(hidden, self.router, self.correction, self.shared_gate, chosen, weights, shared_gate, spec.top,
-                          spec.score == "softmax", spec.renormalize, self.router_bias)
+                          spec.score == "softmax", spec.renormalize, self.router_bias, **options)
         shared_out = None if self.shared is None else self.shared.forward(hidden, step)
         out = torch.empty((tokens, spec.hidden), dtype=torch.float32, device=device)
         if self.interleave and not step.all_single and tokens * spec.top >= GROUPED_FROM and not torch.cuda.is_current_stream_capturing():
@@ -127,9 +143,12 @@ class RoutedExperts(FeedForward):
             return out
         inner = torch.empty((tokens, spec.top, spec.intermediate), dtype=hidden.dtype, device=device)
         on_input = getattr(spec, "weigh", "output") == "input"
-        kernels.moe_gate_up(hidden, self.gate_up, chosen, inner, self.interleave, weights if on_input else None)
+        kernels.moe_gate_up(hidden, self.gate_up, chosen, inner, self.interleave, weights if on_input else None, **self._gate_options("limit"))
         kernels.moe_down(inner, self.down, chosen, None if on_input else weights, shared_out, shared_gate, out, hidden if self.identity else None)
         return out
+
+    def _gate_options(self, name: str) -> dict:
+        return {name: self.limit} if self.limit else {}
 
     def _grouped(self, hidden, chosen, weights, shared_out, shared_gate, out) -> None:
         spec = self.spec
@@ -144,7 +163,7 @@ class RoutedExperts(FeedForward):
         kernels.moe_gather(hidden, order, spec.top, gathered, weights if on_input else None)
         inner = torch.empty((pairs, spec.intermediate), dtype=hidden.dtype, device=device)
         rows = torch.empty((pairs, spec.hidden), dtype=torch.float32, device=device)
-        kernels.gemm_tc_groups(gathered, self.gate_up, inner, bounds, gated=True)
+        kernels.gemm_tc_groups(gathered, self.gate_up, inner, bounds, gated=True, **self._gate_options("gate_limit"))
         kernels.gemm_tc_groups(inner, self.down, rows, bounds)
         if self.identity:
             kernels.moe_combine(rows, position, None if on_input else weights, shared_out, shared_gate, out, chosen, hidden, spec.experts)
