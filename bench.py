@@ -387,9 +387,32 @@ def bikovik_sizes():
     }
 
 
+def tukulorn_sizes():
+    """Layer sizes that resemble a real model of Tukulorn's kind: latent attention (128 + 64 elements per head over a latent of 512, a window of
+    1,024 positions) alternates with differential attention (two 64-element maps over 128-element values, 8 key/value heads, no window); one
+    dense feed-forward four times the width, then 64 experts in 8 groups of which 4 are kept and 6 experts chosen.  Beside it the closest
+    designs that were here before, Fasesun (the same latent attention without a window, the same experts and a shared one) and Bisudra (the
+    same differential attention with a window), and a dense Qwen3, each of the same width, depth and vocabulary."""
+    def tukulorn(width, heads, expert_ff):
+        latent = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "mask": {"size": 1024}, "scale": 192 ** -0.5, "rot": {"base": 10000.0, "dims": 64}}
+        maps = {"heads": heads, "kv_heads": 8, "dim": 64, "vdim": 128, "diff": 0.5, "scale": 0.125, "q_temp": {"coef": 0.25, "every": 512}}
+        dense = {"kind": "dense", "ff": 4 * width}
+        routed = {"kind": "moe", "router": {"experts": 64, "top": 6, "groups": {"count": 8, "keep": 4}, "scale": 2.5}, "expert": {"ff": expert_ff, "limit": 7.0}}
+        layers = [{"type": "latent_attention", "mixer": latent, "mlp": dense}, {"type": "attention", "mixer": maps, "mlp": routed},
+                  {"type": "latent_attention", "mixer": latent, "mlp": routed}, {"type": "attention", "mixer": maps, "mlp": routed}]
+        return {"architecture": "Tukulorn", "layers": layers, "loop": None, "norm": {"eps": 1e-5}, "vocab": 32768, "width": width}
+
+    fasesun, bisudra = fasesun_sizes(), bisudra_sizes()
+    return {
+        "1024": (tukulorn(1024, 8, 704), fasesun["1024"][1], fasesun["1024"][0], bisudra["1024"][0]),
+        "2048": (tukulorn(2048, 16, 1408), fasesun["2048"][1], fasesun["2048"][0], bisudra["2048"][0]),
+        "4096": (tukulorn(4096, 32, 2048), fasesun["4096"][1], fasesun["4096"][0], bisudra["4096"][0]),
+    }
+
+
 def design_comparison(args) -> int:
-    """`--design fasesun|bisudra|pegurax|nugolorn|bikovik`: prefill and decode throughput of the design's layers at three real sizes beside a dense Qwen3
-    of equal width, depth and active feed-forward width (Pegurax also beside Fasesun, Nugolorn also beside Pegurax, Bikovik also beside Nugolorn), with the device time of each kernel class in one
+    """`--design fasesun|bisudra|pegurax|nugolorn|bikovik|tukulorn`: prefill and decode throughput of the design's layers at three real sizes beside a dense Qwen3
+    of equal width, depth and active feed-forward width (Pegurax also beside Fasesun, Nugolorn also beside Pegurax, Bikovik also beside Nugolorn, Tukulorn also beside Fasesun and Bisudra), with the device time of each kernel class in one
     prompt step and one decode step."""
     import numpy as np
     import torch
@@ -405,7 +428,7 @@ def design_comparison(args) -> int:
     records = []
     clocks = ClockSampler()
     clocks.start()
-    sizes = {"bisudra": bisudra_sizes, "fasesun": fasesun_sizes, "pegurax": pegurax_sizes, "nugolorn": nugolorn_sizes, "bikovik": bikovik_sizes}[args.design]()
+    sizes = {"bisudra": bisudra_sizes, "fasesun": fasesun_sizes, "pegurax": pegurax_sizes, "nugolorn": nugolorn_sizes, "bikovik": bikovik_sizes, "tukulorn": tukulorn_sizes}[args.design]()
     for size, (design_config, dense_config, *others) in sizes.items():
         if args.widths and size not in args.widths.split(","):
             continue
@@ -504,7 +527,7 @@ def main() -> int:
                         help="which measurements to run: prefill, decode, points, e2e, kernels (the counterparts of the reference arm's kernels), "
                              "classes (time per kernel class of a decode step, outside a graph)")
     parser.add_argument("--widths", default="", help="with --design: only these of the widths 1024, 2048, 4096 (comma-separated)")
-    parser.add_argument("--design", default="", choices=["", "fasesun", "bisudra", "pegurax", "nugolorn", "bikovik"],
+    parser.add_argument("--design", default="", choices=["", "fasesun", "bisudra", "pegurax", "nugolorn", "bikovik", "tukulorn"],
                         help="instead of the default workload: layers of this design at real sizes beside a dense Qwen3 of equal size")
     args = parser.parse_args()
 
