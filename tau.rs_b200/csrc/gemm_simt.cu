@@ -78,6 +78,99 @@ int launch(const void* x, const void* w, const float* bias, void* out, int M, in
     return tau_launch_status();
 }
 
+// The batched product for few rows (single tokens against one small weight per head), bound by reading the weights once: a group of
+// `kLanes` lanes takes a weight row in 16-byte pieces against up to eight rows of x, which lie in shared memory as floats.
+// grid: (ceil(N / features_per_block), batch, ceil(M / 8)).
+constexpr int kFewRows = 8;
+
+template <typename TIn> struct Piece;
+template <> struct Piece<bf16> { static constexpr int n = 8; };
+template <> struct Piece<float> { static constexpr int n = 4; };
+__device__ __forceinline__ void unpack_piece(const uint4& raw, float (&v)[8]) {
+    const unsigned words[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[2 * i] = __uint_as_float(words[i] << 16);
+        v[2 * i + 1] = __uint_as_float(words[i] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void unpack_piece(const uint4& raw, float (&v)[4]) {
+    v[0] = __uint_as_float(raw.x); v[1] = __uint_as_float(raw.y); v[2] = __uint_as_float(raw.z); v[3] = __uint_as_float(raw.w);
+}
+
+template <typename TIn, typename TOut, int kLanes>
+__global__ void __launch_bounds__(kThreads)
+gemm_few_rows_kernel(const TIn* __restrict__ x, const TIn* __restrict__ w, TOut* __restrict__ out, int M, int N, int K, long long x_stride, long long w_stride,
+                     long long out_stride, long long x_batch, long long w_batch, long long out_batch, int features_per_block) {
+    grid_dependents_launch();
+    grid_dependency_wait();
+    constexpr int n = Piece<TIn>::n;
+    extern __shared__ __align__(16) float rows[];      // [kFewRows][K]
+    const int first_row = blockIdx.z * kFewRows, count = min(kFewRows, M - first_row);
+    x += blockIdx.y * x_batch;
+    w += blockIdx.y * w_batch;
+    out += blockIdx.y * out_batch;
+    for (int item = threadIdx.x; item < kFewRows * K; item += blockDim.x) {
+        const int r = item / K;
+        rows[item] = r < count ? to_float(x[(first_row + r) * x_stride + item - r * K]) : 0.0f;
+    }
+    __syncthreads();
+    const int group = threadIdx.x / kLanes, lane = threadIdx.x % kLanes, groups = blockDim.x / kLanes;
+    const int begin = blockIdx.x * features_per_block, end = min(N, begin + features_per_block);
+    for (int base = begin; base < end; base += groups) {      // every lane of a warp takes every turn: they meet in the shuffles
+        const int feature = base + group;
+        float sums[kFewRows] = {};
+        if (feature < end) {
+            const TIn* weights = w + feature * w_stride;
+            for (int column = lane * n; column < K; column += kLanes * n) {
+                float v[n];
+                unpack_piece(*reinterpret_cast<const uint4*>(weights + column), v);
+#pragma unroll
+                for (int r = 0; r < kFewRows; ++r) {
+#pragma unroll
+                    for (int i = 0; i < n; i += 4) {
+                        const float4 a = *reinterpret_cast<const float4*>(rows + r * K + column + i);
+                        sums[r] = fmaf(v[i], a.x, fmaf(v[i + 1], a.y, fmaf(v[i + 2], a.z, fmaf(v[i + 3], a.w, sums[r]))));
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < kFewRows; ++r)
+#pragma unroll
+            for (int offset = kLanes / 2; offset > 0; offset >>= 1) sums[r] += __shfl_xor_sync(0xffffffffu, sums[r], offset);
+        if (feature < end) {
+#pragma unroll
+            for (int r = 0; r < kFewRows; ++r)
+                if (r < count && lane == r % kLanes) out[(first_row + r) * out_stride + feature] = from_float<TOut>(sums[r]);
+        }
+    }
+}
+
+template <typename TIn, typename TOut>
+int launch_few_rows(const void* x, const void* w, void* out, int M, int N, int K, long long x_stride, long long w_stride, long long out_stride, cudaStream_t stream,
+                    int batch, long long x_batch, long long w_batch, long long out_batch) {
+    const int lanes = K / Piece<TIn>::n <= 8 ? 8 : K / Piece<TIn>::n <= 16 ? 16 : 32;
+    int features = 64;                              // smaller tiles while they leave SMs without a block
+    while (features > kThreads / lanes && batch * ((N + features - 1) / features) < 2 * 148) features /= 2;
+    const dim3 grid((N + features - 1) / features, batch, (M + kFewRows - 1) / kFewRows);
+    const size_t bytes = static_cast<size_t>(kFewRows) * K * sizeof(float);
+    auto* kernel = lanes == 8 ? gemm_few_rows_kernel<TIn, TOut, 8> : lanes == 16 ? gemm_few_rows_kernel<TIn, TOut, 16> : gemm_few_rows_kernel<TIn, TOut, 32>;
+    tau_launch(kernel, grid, dim3(kThreads), bytes, stream, static_cast<const TIn*>(x), static_cast<const TIn*>(w), static_cast<TOut*>(out), M, N, K, x_stride, w_stride,
+               out_stride, x_batch, w_batch, out_batch, features);
+    return tau_launch_status();
+}
+
+template <typename TIn, typename TOut>
+int launch_batched(const void* x, const void* w, void* out, int M, int N, int K, long long x_stride, long long w_stride, long long out_stride, cudaStream_t stream,
+                   int batch, long long x_batch, long long w_batch, long long out_batch) {
+    constexpr int n = Piece<TIn>::n;
+    const bool few = M <= 2 * kFewRows && K % n == 0 && w_stride % n == 0 && w_batch % n == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0
+                     && static_cast<size_t>(kFewRows) * K * sizeof(float) <= 48 * 1024;
+    if (few) return launch_few_rows<TIn, TOut>(x, w, out, M, N, K, x_stride, w_stride, out_stride, stream, batch, x_batch, w_batch, out_batch);
+    return launch<TIn, TOut>(x, w, nullptr, out, M, N, K, x_stride, w_stride, out_stride, stream, batch, x_batch, w_batch, out_batch);
+}
+
 }  // namespace
 
 // Strides are in elements between consecutive rows.  `out_dtype` may be float32 for a bfloat16 product (logits).
@@ -100,8 +193,8 @@ TAU_EXPORT int tau_gemm_simt_batched(int in_dtype, int out_dtype, const void* x,
     if (M <= 0 || N <= 0 || batch <= 0) return 0;
     if (!x || !w || !out || K <= 0 || batch > 65535) return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    if (in_dtype == TAU_F32 && out_dtype == TAU_F32) return launch<float, float>(x, w, nullptr, out, M, N, K, x_stride, w_stride, out_stride, s, batch, x_batch, w_batch, out_batch);
-    if (in_dtype == TAU_BF16 && out_dtype == TAU_BF16) return launch<bf16, bf16>(x, w, nullptr, out, M, N, K, x_stride, w_stride, out_stride, s, batch, x_batch, w_batch, out_batch);
-    if (in_dtype == TAU_BF16 && out_dtype == TAU_F32) return launch<bf16, float>(x, w, nullptr, out, M, N, K, x_stride, w_stride, out_stride, s, batch, x_batch, w_batch, out_batch);
+    if (in_dtype == TAU_F32 && out_dtype == TAU_F32) return launch_batched<float, float>(x, w, out, M, N, K, x_stride, w_stride, out_stride, s, batch, x_batch, w_batch, out_batch);
+    if (in_dtype == TAU_BF16 && out_dtype == TAU_BF16) return launch_batched<bf16, bf16>(x, w, out, M, N, K, x_stride, w_stride, out_stride, s, batch, x_batch, w_batch, out_batch);
+    if (in_dtype == TAU_BF16 && out_dtype == TAU_F32) return launch_batched<bf16, float>(x, w, out, M, N, K, x_stride, w_stride, out_stride, s, batch, x_batch, w_batch, out_batch);
     return cudaErrorInvalidValue;
 }

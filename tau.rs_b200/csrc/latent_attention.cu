@@ -158,12 +158,12 @@ latent_attention_kernel(const T* __restrict__ queries, const T* __restrict__ row
 
 // The same attention with every cached row read once per head as 16-byte vectors and never staged: lane l of a head's warp
 // holds elements [8v, 8v + 8) (4 in 32-bit) of the query for v = l, l + 32, ..., reads the same elements of each row, and keeps
-// the weighted sums of exactly those elements, so the row that was read for the score is the row that is summed.  Two rows are
-// in flight at a time.  The context may be cut into `splits` ranges (grid.z): a range leaves (top, denominator, sums) in
+// the weighted sums of exactly those elements, so the row that was read for the score is the row that is summed.  Two rows
+// are in flight at a time (four no longer fit the registers of two blocks to an SM).  The context may be cut into `splits` ranges (grid.z): a range leaves (top, denominator, sums) in
 // `partial` and `latent_merge_kernel` joins them; with one range the warp finishes the head itself.
 template <typename T> struct RowVectors;
-template <> struct RowVectors<bf16> { static constexpr int n = 8, per_lane = 3; };
-template <> struct RowVectors<float> { static constexpr int n = 4, per_lane = 6; };
+template <> struct RowVectors<bf16> { static constexpr int n = 8, per_lane = 3, at_once = 2; };
+template <> struct RowVectors<float> { static constexpr int n = 4, per_lane = 6, at_once = 2; };
 constexpr int kVectorWidth = 768;      // 32 lanes x per_lane x n elements
 
 template <typename T> __device__ __forceinline__ void unpack_row(const uint4& raw, float (&out)[RowVectors<T>::n]);
@@ -204,7 +204,7 @@ latent_attention_vec_kernel(const T* __restrict__ queries, const T* __restrict__
                             int page_tokens, int heads, int rank, int rot, float scale, int window, int splits, float* __restrict__ partial) {
     grid_dependents_launch();
     grid_dependency_wait();
-    constexpr int n = RowVectors<T>::n, kPer = RowVectors<T>::per_lane;
+    constexpr int n = RowVectors<T>::n, kPer = RowVectors<T>::per_lane, kRows = RowVectors<T>::at_once;
     const int token = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, split = blockIdx.z;
     const int head = blockIdx.y * kMaxWarps + warp;
     if (head >= heads) return;                               // the warps of a block never meet
@@ -231,43 +231,54 @@ latent_attention_vec_kernel(const T* __restrict__ queries, const T* __restrict__
         const int page_index = key / page_tokens;
         const int stop = min(end, (page_index + 1) * page_tokens);
         const T* row = rows + (static_cast<size_t>(pages[page_index]) * page_tokens + (key - page_index * page_tokens)) * width;
-        for (; key < stop; key += 2, row += 2 * static_cast<size_t>(width)) {
-            const bool pair = key + 1 < stop;
-            uint4 a[kPer], b[kPer];
+        for (; key < stop; key += kRows, row += kRows * static_cast<size_t>(width)) {
+            uint4 held[kRows][kPer];
 #pragma unroll
-            for (int i = 0; i < kPer; ++i) {
-                const int v = lane + 32 * i;
-                a[i] = v < vectors ? *reinterpret_cast<const uint4*>(row + v * n) : zero;
-                b[i] = (pair && v < vectors) ? *reinterpret_cast<const uint4*>(row + width + v * n) : zero;
-            }
-            float dot_a = 0.0f, dot_b = 0.0f;
+            for (int r = 0; r < kRows; ++r)
 #pragma unroll
-            for (int i = 0; i < kPer; ++i) {
-                dot_a += vector_dot<T>(q[i], a[i]);
-                dot_b += vector_dot<T>(q[i], b[i]);
+                for (int i = 0; i < kPer; ++i) {
+                    const int v = lane + 32 * i;
+                    held[r][i] = (key + r < stop && v < vectors) ? *reinterpret_cast<const uint4*>(row + r * width + v * n) : zero;
+                }
+            float dots[kRows];
+#pragma unroll
+            for (int r = 0; r < kRows; ++r) {
+                dots[r] = 0.0f;
+#pragma unroll
+                for (int i = 0; i < kPer; ++i) dots[r] += vector_dot<T>(q[i], held[r][i]);
             }
 #pragma unroll
-            for (int offset = 16; offset > 0; offset >>= 1) {
-                dot_a += __shfl_xor_sync(0xffffffffu, dot_a, offset);
-                dot_b += __shfl_xor_sync(0xffffffffu, dot_b, offset);
+            for (int offset = 16; offset > 0; offset >>= 1)
+#pragma unroll
+                for (int r = 0; r < kRows; ++r) dots[r] += __shfl_xor_sync(0xffffffffu, dots[r], offset);
+            float new_top = top;
+#pragma unroll
+            for (int r = 0; r < kRows; ++r) {
+                dots[r] = key + r < stop ? dots[r] * scale : -INFINITY;
+                new_top = fmaxf(new_top, dots[r]);
             }
-            dot_a *= scale;
-            dot_b *= scale;
-            const float new_top = pair ? fmaxf(top, fmaxf(dot_a, dot_b)) : fmaxf(top, dot_a);
             const float rescale = expf(top - new_top);      // 0 the first time
-            const float weight_a = expf(dot_a - new_top), weight_b = pair ? expf(dot_b - new_top) : 0.0f;
-            denominator = denominator * rescale + weight_a + weight_b;
+            denominator *= rescale;
+#pragma unroll
+            for (int r = 0; r < kRows; ++r) {
+                dots[r] = expf(dots[r] - new_top);           // 0 behind the last row
+                denominator += dots[r];
+            }
             top = new_top;
 #pragma unroll
             for (int i = 0; i < kPer; ++i) {
-                float x[n], y[n];
-                unpack_row<T>(a[i], x);
-                unpack_row<T>(b[i], y);
 #pragma unroll
-                for (int j = 0; j < n; ++j) sums[i][j] = fmaf(weight_b, y[j], fmaf(sums[i][j], rescale, weight_a * x[j]));
+                for (int j = 0; j < n; ++j) sums[i][j] *= rescale;
+#pragma unroll
+                for (int r = 0; r < kRows; ++r) {
+                    float x[n];
+                    unpack_row<T>(held[r][i], x);
+#pragma unroll
+                    for (int j = 0; j < n; ++j) sums[i][j] = fmaf(dots[r], x[j], sums[i][j]);
+                }
             }
         }
-        key = stop;      // the step of two may have overshot by one
+        key = stop;      // the last step may have overshot
     }
     if (splits > 1) {
         float* record = partial + ((static_cast<size_t>(token) * heads + head) * splits + split) * (rank + 2);
@@ -298,29 +309,39 @@ latent_attention_vec_kernel(const T* __restrict__ queries, const T* __restrict__
         }
 }
 
-// One block per (token, head): joins the ranges of a context in their order.
+// One block per (token, head): joins the ranges of a context in their order.  A range's factor is computed once, by one thread.
+constexpr int kMaxSplits = 64;
+
 template <typename T>
 __global__ void latent_merge_kernel(const float* __restrict__ partial, const float* __restrict__ sinks, T* __restrict__ out, int heads, int rank, int splits) {
     grid_dependents_launch();
     grid_dependency_wait();
     const size_t item = blockIdx.x;
     const float* records = partial + item * splits * (rank + 2);
-    float top = -INFINITY;
-    for (int split = 0; split < splits; ++split) top = fmaxf(top, records[static_cast<size_t>(split) * (rank + 2)]);
-    const float sink = sinks ? sinks[item % heads] : -INFINITY;
-    const float all_top = fmaxf(top, sink);
-    float denominator = sinks ? expf(sink - all_top) : 0.0f;
-    for (int split = 0; split < splits; ++split) {
-        const float* record = records + static_cast<size_t>(split) * (rank + 2);
-        denominator += expf(record[0] - all_top) * record[1];
+    __shared__ float factors[kMaxSplits];
+    __shared__ float inverse;
+    if (threadIdx.x < 32) {
+        const int lane = threadIdx.x;
+        const float sink = sinks ? sinks[item % heads] : -INFINITY;
+        float top = sink;
+        for (int split = lane; split < splits; split += 32) top = fmaxf(top, records[static_cast<size_t>(split) * (rank + 2)]);
+        top = warp_max(top);
+        float denominator = 0.0f;
+        for (int split = lane; split < splits; split += 32) {
+            const float* record = records + static_cast<size_t>(split) * (rank + 2);
+            const float factor = expf(record[0] - top);
+            factors[split] = factor;
+            denominator += factor * record[1];
+        }
+        denominator = warp_sum(denominator) + (sinks ? expf(sink - top) : 0.0f);
+        if (lane == 0) inverse = 1.0f / denominator;
     }
+    __syncthreads();
     for (int column = threadIdx.x; column < rank; column += blockDim.x) {
         float sum = 0.0f;
-        for (int split = 0; split < splits; ++split) {
-            const float* record = records + static_cast<size_t>(split) * (rank + 2);
-            sum = fmaf(expf(record[0] - all_top), record[2 + column], sum);
-        }
-        out[item * rank + column] = from_float<T>(sum / denominator);
+#pragma unroll 16
+        for (int split = 0; split < splits; ++split) sum = fmaf(factors[split], records[static_cast<size_t>(split) * (rank + 2) + 2 + column], sum);
+        out[item * rank + column] = from_float<T>(sum * inverse);
     }
 }
 
@@ -366,6 +387,62 @@ latent_expand_kernel(const T* __restrict__ q, long long q_stride, const T* __res
         const size_t slot = ((page * heads + head) * page_tokens + position % page_tokens) * width + column;
         key_pages[slot] = from_float<T>(key);
         value_pages[slot] = column < value_dim ? expanded_row[heads * head_dim + head * value_dim + column] : from_float<T>(0.0f);
+    }
+}
+
+// The same for bfloat16 rows whose parts are whole 16-byte pieces: a thread moves eight neighbouring columns of a head's query, key and value at
+// a time, and the sine and cosine of the token's rotated pairs are computed once for all heads.
+constexpr int kMaxTurns = 256;
+
+__global__ void __launch_bounds__(256)
+latent_expand_vec_kernel(const bf16* __restrict__ q, long long q_stride, const bf16* __restrict__ down, long long down_stride, const bf16* __restrict__ expanded,
+                         bf16* __restrict__ queries, bf16* __restrict__ key_pages, bf16* __restrict__ value_pages, const float* __restrict__ inv_freq, int rotary,
+                         const int* __restrict__ positions, const int* __restrict__ token_seq, int pages_per_sequence, int page_tokens, int heads,
+                         int head_dim, int rot, int rank, int value_dim) {
+    grid_dependents_launch();
+    grid_dependency_wait();
+    __shared__ float2 turns[kMaxTurns];      // (cosine, sine); pairs behind the rotation stay as they are
+    const int token = blockIdx.x, position = positions[token];
+    for (int pair = threadIdx.x; pair < rot / 2; pair += blockDim.x) {
+        float sine = 0.0f, cosine = 1.0f;
+        if (2 * pair + 1 < rotary) sincosf(static_cast<float>(position) * inv_freq[pair], &sine, &cosine);
+        turns[pair] = make_float2(cosine, sine);
+    }
+    __syncthreads();
+    const int width = head_dim + rot, pieces = width / 8;
+    const size_t page = static_cast<size_t>(token_seq[token]) * pages_per_sequence + position / page_tokens;
+    const bf16* q_row = q + static_cast<size_t>(token) * q_stride;
+    const bf16* shared_key = down + static_cast<size_t>(token) * down_stride + rank;
+    const bf16* expanded_row = expanded + static_cast<size_t>(token) * heads * (head_dim + value_dim);
+    auto turned = [&](const bf16* source, int first) {      // eight elements of the rotated part from element `first` on
+        const uint4 raw = *reinterpret_cast<const uint4*>(source + first);
+        const unsigned in[4] = {raw.x, raw.y, raw.z, raw.w};
+        unsigned out[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 turn = turns[first / 2 + i];
+            const float u = __uint_as_float(in[i] << 16), w = __uint_as_float(in[i] & 0xffff0000u);
+            const __nv_bfloat162 two = __floats2bfloat162_rn(u * turn.x - w * turn.y, w * turn.x + u * turn.y);
+            out[i] = *reinterpret_cast<const unsigned*>(&two);
+        }
+        return make_uint4(out[0], out[1], out[2], out[3]);
+    };
+    for (int item = threadIdx.x; item < heads * pieces; item += blockDim.x) {
+        const int head = item / pieces, column = item % pieces * 8;
+        const bf16* q_head = q_row + head * width;
+        uint4 query, key, value = make_uint4(0u, 0u, 0u, 0u);
+        if (column < head_dim) {
+            query = *reinterpret_cast<const uint4*>(q_head + column);
+            key = *reinterpret_cast<const uint4*>(expanded_row + head * head_dim + column);
+        } else {
+            query = turned(q_head + head_dim, column - head_dim);
+            key = turned(shared_key, column - head_dim);
+        }
+        if (column < value_dim) value = *reinterpret_cast<const uint4*>(expanded_row + heads * head_dim + head * value_dim + column);
+        *reinterpret_cast<uint4*>(queries + (static_cast<size_t>(token) * heads + head) * width + column) = query;
+        const size_t slot = ((page * heads + head) * page_tokens + position % page_tokens) * width + column;
+        *reinterpret_cast<uint4*>(key_pages + slot) = key;
+        *reinterpret_cast<uint4*>(value_pages + slot) = value;
     }
 }
 
@@ -433,7 +510,7 @@ int launch_vec(const void* queries, const void* rows, void* out, const float* si
     if (splits > 1) {
         const int status = tau_launch_status();
         if (status != 0) return status;
-        tau_launch(latent_merge_kernel<T>, dim3(tokens * heads), dim3(128), 0, s, static_cast<const float*>(partial), sinks, static_cast<T*>(out), heads, rank, splits);
+        tau_launch(latent_merge_kernel<T>, dim3(tokens * heads), dim3(rank >= 512 ? 512 : (rank + 31) / 32 * 32), 0, s, static_cast<const float*>(partial), sinks, static_cast<T*>(out), heads, rank, splits);
     }
     return tau_launch_status();
 }
@@ -471,7 +548,7 @@ TAU_EXPORT int tau_latent_attention(int dtype, const void* queries, const void* 
                                     const int* token_seq, const int* page_rows, int page_stride, int page_tokens, int tokens, int heads, int rank,
                                     int rot, float scale, int window, int splits, float* partial, long long partial_floats, void* stream) {
     if (tokens <= 0) return 0;
-    if (!queries || !rows || !out || !positions || !token_seq || !page_rows || heads <= 0 || rank <= 0 || rank > 32 * kMaxOwned || rot < 0 || splits < 1)
+    if (!queries || !rows || !out || !positions || !token_seq || !page_rows || heads <= 0 || rank <= 0 || rank > 32 * kMaxOwned || rot < 0 || splits < 1 || splits > kMaxSplits)
         return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     // Rows that are whole 16-byte vectors take the kernel that reads them as such; others the one that stages tiles.
@@ -511,7 +588,14 @@ TAU_EXPORT int tau_latent_expand(int dtype, const void* q, long long q_stride, c
         || value_dim <= 0 || value_dim > head_dim + rot || rotary > rot || (rotary > 0 && !inv_freq) || pages_per_sequence <= 0)
         return cudaErrorInvalidValue;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    if (dtype == TAU_BF16)
+    const bool pieces = head_dim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && value_dim % 8 == 0 && q_stride % 8 == 0 && down_stride % 8 == 0 && rot / 2 <= kMaxTurns
+                        && ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(down) | reinterpret_cast<uintptr_t>(expanded) | reinterpret_cast<uintptr_t>(queries)
+                             | reinterpret_cast<uintptr_t>(key_pages) | reinterpret_cast<uintptr_t>(value_pages)) & 15) == 0;
+    if (dtype == TAU_BF16 && pieces)
+        tau_launch(latent_expand_vec_kernel, dim3(tokens), dim3(256), 0, s, static_cast<const bf16*>(q), q_stride, static_cast<const bf16*>(down), down_stride,
+                   static_cast<const bf16*>(expanded), static_cast<bf16*>(queries), static_cast<bf16*>(key_pages), static_cast<bf16*>(value_pages), inv_freq,
+                   rotary, positions, token_seq, pages_per_sequence, page_tokens, heads, head_dim, rot, rank, value_dim);
+    else if (dtype == TAU_BF16)
         tau_launch(latent_expand_kernel<bf16>, dim3(tokens), dim3(256), 0, s, static_cast<const bf16*>(q), q_stride, static_cast<const bf16*>(down), down_stride,
                    static_cast<const bf16*>(expanded), static_cast<bf16*>(queries), static_cast<bf16*>(key_pages), static_cast<bf16*>(value_pages), inv_freq,
                    rotary, positions, token_seq, pages_per_sequence, page_tokens, heads, head_dim, rot, rank, value_dim);

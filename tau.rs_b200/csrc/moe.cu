@@ -30,28 +30,38 @@ __device__ __forceinline__ float warp_dot(const T* __restrict__ weights, const f
     return warp_sum(sum);
 }
 
-// 32-bit rows (the router's) that start on a 16-byte boundary are read four elements at a time.
-template <>
-__device__ __forceinline__ float warp_dot<float>(const float* __restrict__ weights, const float* __restrict__ vector, int length, int lane) {
-    float sum = 0.0f;
+// Dot products of one 32-bit row (the router's) with `kRows` vectors in shared memory, `pitch` floats apart, over the warp; a row that starts
+// on a 16-byte boundary is read four elements at a time.  The order of the sums is the same for every `kRows`.
+template <int kRows>
+__device__ __forceinline__ void warp_dot_rows(const float* __restrict__ weights, const float* __restrict__ vectors, int pitch, int length, int lane, float (&sums)[kRows]) {
+    float other[kRows];
+#pragma unroll
+    for (int row = 0; row < kRows; ++row) sums[row] = other[row] = 0.0f;
     if ((reinterpret_cast<uintptr_t>(weights) & 15) == 0 && length % 4 == 0) {
-        float other = 0.0f;
+        auto add = [](float sum, const float4& w, const float4& x) { return fmaf(w.x, x.x, fmaf(w.y, x.y, fmaf(w.z, x.z, fmaf(w.w, x.w, sum)))); };
         int column = lane * 4;
         for (; column + 128 < length; column += 256) {
             const float4 w0 = *reinterpret_cast<const float4*>(weights + column), w1 = *reinterpret_cast<const float4*>(weights + column + 128);
-            const float4 x0 = *reinterpret_cast<const float4*>(vector + column), x1 = *reinterpret_cast<const float4*>(vector + column + 128);
-            sum = fmaf(w0.x, x0.x, fmaf(w0.y, x0.y, fmaf(w0.z, x0.z, fmaf(w0.w, x0.w, sum))));
-            other = fmaf(w1.x, x1.x, fmaf(w1.y, x1.y, fmaf(w1.z, x1.z, fmaf(w1.w, x1.w, other))));
+#pragma unroll
+            for (int row = 0; row < kRows; ++row) {
+                sums[row] = add(sums[row], w0, *reinterpret_cast<const float4*>(vectors + row * pitch + column));
+                other[row] = add(other[row], w1, *reinterpret_cast<const float4*>(vectors + row * pitch + column + 128));
+            }
         }
         if (column < length) {
-            const float4 w0 = *reinterpret_cast<const float4*>(weights + column), x0 = *reinterpret_cast<const float4*>(vector + column);
-            sum = fmaf(w0.x, x0.x, fmaf(w0.y, x0.y, fmaf(w0.z, x0.z, fmaf(w0.w, x0.w, sum))));
+            const float4 w0 = *reinterpret_cast<const float4*>(weights + column);
+#pragma unroll
+            for (int row = 0; row < kRows; ++row) sums[row] = add(sums[row], w0, *reinterpret_cast<const float4*>(vectors + row * pitch + column));
         }
-        sum += other;
     } else {
-        for (int column = lane; column < length; column += 32) sum = fmaf(weights[column], vector[column], sum);
+        for (int column = lane; column < length; column += 32) {
+            const float w = weights[column];
+#pragma unroll
+            for (int row = 0; row < kRows; ++row) sums[row] = fmaf(w, vectors[row * pitch + column], sums[row]);
+        }
     }
-    return warp_sum(sum);
+#pragma unroll
+    for (int row = 0; row < kRows; ++row) sums[row] = warp_sum(sums[row] + other[row]);
 }
 
 // Eight bfloat16 weights against eight floats of shared memory, which are read as two 16-byte words (lanes 32 bytes apart meet
@@ -129,31 +139,59 @@ __device__ __forceinline__ void warp_dot_pair<bf16>(const bf16* __restrict__ fir
     second_sum = warp_sum(b + d);
 }
 
+// Activation rows as floats in shared memory: `count` elements from `source` on, 16 bytes at a time where they allow it.
+__device__ __forceinline__ void unpack_eight(const uint4& raw, float* target) {
+    *reinterpret_cast<float4*>(target) = make_float4(__uint_as_float(raw.x << 16), __uint_as_float(raw.x & 0xffff0000u), __uint_as_float(raw.y << 16), __uint_as_float(raw.y & 0xffff0000u));
+    *reinterpret_cast<float4*>(target + 4) = make_float4(__uint_as_float(raw.z << 16), __uint_as_float(raw.z & 0xffff0000u), __uint_as_float(raw.w << 16), __uint_as_float(raw.w & 0xffff0000u));
+}
+
 template <typename T>
-__global__ void __launch_bounds__(kThreads)
+__device__ __forceinline__ void stage_row(const T* __restrict__ source, float* __restrict__ target, int count) {
+    if constexpr (sizeof(T) == 2) {
+        if (((reinterpret_cast<uintptr_t>(source) | reinterpret_cast<uintptr_t>(target)) & 15) == 0 && count % 8 == 0) {
+            for (int column = threadIdx.x * 8; column < count; column += blockDim.x * 8) unpack_eight(*reinterpret_cast<const uint4*>(source + column), target + column);
+            return;
+        }
+    }
+    for (int column = threadIdx.x; column < count; column += blockDim.x) target[column] = to_float(source[column]);
+}
+
+// A block scores `kRows` tokens, so that a router row is read once for all of them; a warp per token then chooses.
+template <typename T, int kRows>
+__global__ void __launch_bounds__(kRows == 1 ? 1024 : kThreads)
 moe_route_kernel(const T* __restrict__ hidden, const float* __restrict__ router, const float* __restrict__ logit_bias, const float* __restrict__ correction,
                  const float* __restrict__ shared_gate_weight, int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ shared_gate,
-                 int width, int experts, int top, int softmax, int renormalize, int groups, int keep, float scale) {
+                 int tokens, int width, int experts, int top, int softmax, int renormalize, int groups, int keep, float scale) {
     grid_dependents_launch();
     grid_dependency_wait();
     extern __shared__ __align__(16) float shared[];
-    float* row = shared;               // [width]
-    float* scores = shared + width;    // [experts]
-    float* choice = scores + experts;  // [experts]
-    float* ranks = choice + experts;   // [groups], if there are several
-    const int token = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int column = threadIdx.x; column < width; column += blockDim.x) row[column] = to_float(hidden[static_cast<size_t>(token) * width + column]);
+    const int pitch = (width + 3) & ~3, per_token = 2 * experts + groups;
+    const int first = blockIdx.x * kRows, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const int count = min(kRows, tokens - first);
+    float* numbers = shared + kRows * pitch;      // per token: scores [experts], what is chosen by [experts], the groups' ranks [groups]
+    for (int row = 0; row < kRows; ++row) stage_row(hidden + static_cast<size_t>(first + min(row, count - 1)) * width, shared + row * pitch, width);
     __syncthreads();
-    for (int expert = warp; expert < experts; expert += kWarps) {
-        const float z = warp_dot(router + static_cast<size_t>(expert) * width, row, width, lane);
-        if (lane == 0) scores[expert] = z + (logit_bias ? logit_bias[expert] : 0.0f);
+    for (int expert = warp; expert < experts; expert += warps) {
+        float z[kRows];
+        warp_dot_rows<kRows>(router + static_cast<size_t>(expert) * width, shared, pitch, width, lane, z);
+        if (lane == 0)
+#pragma unroll
+            for (int row = 0; row < kRows; ++row) numbers[row * per_token + expert] = z[row] + (logit_bias ? logit_bias[expert] : 0.0f);
     }
-    if (shared_gate_weight && warp == kWarps - 1) {
-        const float z = warp_dot(shared_gate_weight, row, width, lane);
-        if (lane == 0) shared_gate[token] = 1.0f / (1.0f + expf(-z));
+    if (shared_gate_weight && warp == warps - 1) {
+        float z[kRows];
+        warp_dot_rows<kRows>(shared_gate_weight, shared, pitch, width, lane, z);
+        if (lane == 0)
+#pragma unroll
+            for (int row = 0; row < kRows; ++row)
+                if (row < count) shared_gate[first + row] = 1.0f / (1.0f + expf(-z[row]));
     }
     __syncthreads();
-    if (warp != 0) return;
+    if (warp >= count) return;
+    const int token = first + warp;
+    float* scores = numbers + warp * per_token;
+    float* choice = scores + experts;
+    float* ranks = choice + experts;
     if (softmax) {
         float top_z = -INFINITY;
         for (int expert = lane; expert < experts; expert += 32) top_z = fmaxf(top_z, scores[expert]);
@@ -228,7 +266,7 @@ moe_gate_up_kernel(const T* __restrict__ hidden, const T* __restrict__ gate_up, 
     extern __shared__ __align__(16) float row[];
     const int pair = blockIdx.x, token = pair / top, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (chosen[pair] >= real_experts) return;      // an identity expert has no inner features
-    for (int column = threadIdx.x; column < width; column += blockDim.x) row[column] = to_float(hidden[static_cast<size_t>(token) * width + column]);
+    stage_row(hidden + static_cast<size_t>(token) * width, row, width);
     __syncthreads();
     const T* weights = gate_up + static_cast<size_t>(chosen[pair]) * 2 * inner * width;
     // A weight on the expert's input: both products are linear in the row, so the weight multiplies their 32-bit sums.
@@ -257,8 +295,13 @@ moe_down_kernel(const T* __restrict__ inner_in, const T* __restrict__ down, cons
     grid_dependency_wait();
     extern __shared__ __align__(16) float rows[];     // [top][inner]
     const int token = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int item = threadIdx.x; item < top * inner; item += blockDim.x)      // an identity expert's place was never written: nothing of it is read
-        rows[item] = chosen[static_cast<size_t>(token) * top + item / inner] < real_experts ? to_float(inner_in[static_cast<size_t>(token) * top * inner + item]) : 0.0f;
+    const T* source = inner_in + static_cast<size_t>(token) * top * inner;
+    if (!hidden) {                                   // without identity experts every place was written
+        stage_row(source, rows, top * inner);
+    } else {
+        for (int item = threadIdx.x; item < top * inner; item += blockDim.x)      // an identity expert's place was never written: nothing of it is read
+            rows[item] = chosen[static_cast<size_t>(token) * top + item / inner] < real_experts ? to_float(source[item]) : 0.0f;
+    }
     __syncthreads();
     const int begin = blockIdx.y * features_per_block, end = min(width, begin + features_per_block);
     for (int feature = begin + warp; feature < end; feature += kWarps) {
@@ -330,7 +373,11 @@ __global__ void moe_gather_kernel(const T* __restrict__ hidden, const int* __res
     const int pair = order[blockIdx.x];
     const T* source = hidden + static_cast<size_t>(pair / top) * width;
     T* target = gathered + static_cast<size_t>(blockIdx.x) * width;
-    if (input_weights) {
+    constexpr int kPiece = 16 / sizeof(T);
+    if (!input_weights && width % kPiece == 0 && ((reinterpret_cast<uintptr_t>(hidden) | reinterpret_cast<uintptr_t>(gathered)) & 15) == 0) {
+        for (int column = threadIdx.x * kPiece; column < width; column += blockDim.x * kPiece)
+            *reinterpret_cast<uint4*>(target + column) = *reinterpret_cast<const uint4*>(source + column);
+    } else if (input_weights) {
         const float weight = input_weights[pair];
         for (int column = threadIdx.x; column < width; column += blockDim.x) target[column] = from_float<T>(weight * to_float(source[column]));
     } else {
@@ -346,6 +393,20 @@ __global__ void moe_combine_kernel(const float* __restrict__ rows, const int* __
     grid_dependents_launch();
     grid_dependency_wait();
     const int token = blockIdx.x;
+    if (!chosen && !shared_out && width % 4 == 0 && ((reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+        for (int column = threadIdx.x * 4; column < width; column += blockDim.x * 4) {      // the same sums, four columns at a time
+            float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            for (int place = 0; place < top; ++place) {
+                const size_t pair = static_cast<size_t>(token) * top + place;
+                const float weight = weights ? weights[pair] : 1.0f;
+                const float4 row = *reinterpret_cast<const float4*>(rows + static_cast<size_t>(position[pair]) * width + column);
+                sum.x = fmaf(weight, row.x, sum.x); sum.y = fmaf(weight, row.y, sum.y);
+                sum.z = fmaf(weight, row.z, sum.z); sum.w = fmaf(weight, row.w, sum.w);
+            }
+            *reinterpret_cast<float4*>(out + static_cast<size_t>(token) * width + column) = sum;
+        }
+        return;
+    }
     for (int column = threadIdx.x; column < width; column += blockDim.x) {
         float sum = 0.0f;
         for (int place = 0; place < top; ++place) {
@@ -364,11 +425,14 @@ int launch_all(int what, const void* a, const void* b, const void* c, const void
                int tokens, int width, int inner, int experts, int top, int flag_a, int flag_b, cudaStream_t s, const void* g = nullptr, float constant = 1.0f,
                int groups = 1, int keep = 1) {
     if (what == 0) {
-        const size_t bytes = (static_cast<size_t>(width) + 2 * experts + groups) * sizeof(float);
-        if (bytes > 48 * 1024 && cudaFuncSetAttribute(moe_route_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)) != cudaSuccess)
-            return cudaErrorInvalidValue;
-        tau_launch(moe_route_kernel<T>, dim3(tokens), dim3(kThreads), bytes, s, static_cast<const T*>(a), static_cast<const float*>(b), static_cast<const float*>(e),
-                   static_cast<const float*>(c), static_cast<const float*>(d), static_cast<int*>(o1), static_cast<float*>(o2), static_cast<float*>(o3), width, experts, top, flag_a, flag_b,
+        // Few tokens: one to a block with many warps, since its rows of the router are a chain of loads; many: four to a block.
+        const size_t one = (static_cast<size_t>((width + 3) & ~3) + 2 * experts + groups) * sizeof(float);
+        const bool four = tokens >= 4 * 148 && 4 * one <= 200 * 1024;
+        const size_t bytes = four ? 4 * one : one;
+        auto* kernel = four ? moe_route_kernel<T, 4> : moe_route_kernel<T, 1>;
+        if (bytes > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)) != cudaSuccess) return cudaErrorInvalidValue;
+        tau_launch(kernel, dim3(four ? (tokens + 3) / 4 : tokens), dim3(tokens <= 2 * 148 ? 1024 : kThreads), bytes, s, static_cast<const T*>(a), static_cast<const float*>(b), static_cast<const float*>(e),
+                   static_cast<const float*>(c), static_cast<const float*>(d), static_cast<int*>(o1), static_cast<float*>(o2), static_cast<float*>(o3), tokens, width, experts, top, flag_a, flag_b,
                    groups, keep, constant);
     } else if (what == 1) {
         const int per_block = 64;

@@ -126,19 +126,25 @@ def test_the_gate_on_heads(heads, width, value_dim, per_head):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("experts, top, groups, keep", [(12, 3, 4, 2), (8, 2, 4, 3), (1, 1, 1, 1), (5, 2, 5, 3), (6, 6, 2, 2), (64, 6, 8, 3), (160, 4, 40, 7), (40, 1, 40, 1), (6, 2, 1, 1)])
-def test_the_router_chooses_among_the_best_groups(dtype, experts, top, groups, keep):
+@pytest.mark.parametrize("experts, top, groups, keep, tokens, width", [
+    (12, 3, 4, 2, 41, 72), (8, 2, 4, 3, 41, 72), (1, 1, 1, 1, 41, 72), (5, 2, 5, 3, 41, 72), (6, 6, 2, 2, 41, 72), (64, 6, 8, 3, 41, 72), (160, 4, 40, 7, 41, 72), (40, 1, 40, 1, 41, 72),
+    (6, 2, 1, 1, 41, 72), (12, 3, 4, 2, 601, 72), (8, 2, 4, 3, 602, 75), (10, 2, 5, 2, 594, 300), (8, 2, 4, 3, 350, 75)])      # one token to a block of many warps, of few, four to a block
+def test_the_router_chooses_among_the_best_groups(dtype, experts, top, groups, keep, tokens, width):
     from tau_rs_b200.csrc import kernels
 
     torch.manual_seed(experts + top)
-    tokens, width, scale = 41, 72, 2.3
+    scale, shared = 2.3, torch.randn(width) * 0.2
     hidden, router = torch.randn(tokens, width).to(TORCH[dtype]).float(), torch.randn(experts, width) * 0.3
     if experts >= 8:
         router[experts // 2] = router[experts // 2 + 1]                     # two experts that always tie
     hidden[0] = 0.0                                                         # a token whose experts all tie: the lowest numbers
     chosen = torch.empty((tokens, top), dtype=torch.int32, device=DEVICE)
     weights = torch.empty((tokens, top), dtype=torch.float32, device=DEVICE)
-    kernels.moe_route(on_device(hidden, TORCH[dtype]), on_device(router), None, None, chosen, weights, None, top, False, True, None, groups=groups, keep=keep, scale=scale)
+    shared_gate = torch.empty(tokens, dtype=torch.float32, device=DEVICE)
+    kernels.moe_route(on_device(hidden, TORCH[dtype]), on_device(router), None, on_device(shared), chosen, weights, shared_gate, top, False, True, None, groups=groups, keep=keep,
+                      scale=scale)
+    assert torch.allclose(shared_gate.cpu().double(), plain.sigmoid(hidden.double() @ shared.double()), atol=2e-6)
+    chosen, weights = chosen.cpu(), weights.cpu()
     scores = plain.sigmoid(hidden.double() @ router.double().T)
     kept_apart = 0
     for token in range(tokens):
@@ -146,7 +152,7 @@ def test_the_router_chooses_among_the_best_groups(dtype, experts, top, groups, k
         wanted = plain.choose_experts(row, top, groups, keep)
         assert chosen[token].tolist() == wanted, token
         picked = scores[token][wanted]
-        assert torch.allclose(weights[token].cpu().double(), picked / (picked.sum() + 1e-20) * scale, atol=2e-6)
+        assert torch.allclose(weights[token].double(), picked / (picked.sum() + 1e-20) * scale, atol=2e-6)
         kept_apart += wanted != plain.choose_experts(row, top, 1, 1)
     assert kept_apart > 0 or groups == keep or experts == groups      # groups of one expert keep the best experts anyway
 
@@ -309,6 +315,22 @@ def test_one_differential_key_that_stands_out_far_back(monkeypatch, dtype, vdim)
     assert relative_error(cold, wanted) > 0.2
     monkeypatch.setattr(plain, "visible", lambda tokens, window=None, real=plain.visible: real(tokens, 300))      # the far keys forgotten
     assert relative_error(plain.differential_attention(h.double(), doubled(values), "m", mixer, 1e-5), wanted) > 0.3
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("rows, batch, features, depth", [(1, 3, 40, 24), (8, 16, 512, 128), (9, 2, 70, 512), (16, 1, 1, 8), (17, 5, 33, 64), (3, 4, 50, 22), (2, 2, 9, 2048)])
+def test_the_batched_product_of_few_rows(dtype, rows, batch, features, depth):
+    """Views whose rows and batches lie further apart than they are long; sizes that whole 16-byte pieces serve and others."""
+    from tau_rs_b200.csrc import kernels
+
+    torch.manual_seed(rows)
+    values, weight = torch.randn(rows, batch, depth + 8), torch.randn(batch, features, depth)
+    for out_dtype in {dtype, "float32"}:
+        out = torch.full((rows, batch, features + 3), float("nan"), dtype=TORCH[out_dtype], device=DEVICE)
+        kernels.gemm_simt_batched(on_device(values, TORCH[dtype])[:, :, :depth], on_device(weight, TORCH[dtype]), out[:, :, :features])
+        wanted = torch.einsum("mbk,bnk->mbn", values[:, :, :depth].to(TORCH[dtype]).double(), weight.to(TORCH[dtype]).double())
+        assert relative_error(out[:, :, :features].float().cpu(), wanted) < (2e-6 if out_dtype == "float32" else 5e-3)
+        assert torch.isnan(out[:, :, features:].float()).all()
 
 
 # ---- whole models: cuttings, batches, reuse ----------------------------------------------------------------------------
