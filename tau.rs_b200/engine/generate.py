@@ -109,7 +109,7 @@ class GenerationMetrics:
             "decode_tokens_per_second": round(self.decode_tokens_per_second, 2),
             "prefill_tokens_per_second": round(self.prefill_tokens_per_second, 2),
             "prefill_steps": self.prefill_steps, "decode_steps": self.decode_steps, "batches": self.batches,
-            "decode_gb_per_second": self.decode_gb_per_second and round(self.decode_gb_per_second, 1),
+            "decode_gb_per_second": self.decode_gb_per_second and round(self.decode_gb_per_second, 3),
             "fraction_of_roofline": (round(self.decode_gb_per_second / self.peak_gb_per_second, 4)
                                      if self.decode_gb_per_second and self.peak_gb_per_second else None),
         }
